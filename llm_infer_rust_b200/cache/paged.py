@@ -37,7 +37,8 @@ class LayerCache:
     v: Optional[torch.Tensor] = None
     writes: bool = True                      # False: this entry reads another entry's pages
     state: Optional[torch.Tensor] = None     # the mixer's state, [slots + 1, *state_shape]; slot 0 is the sink
-    states: Dict[str, torch.Tensor] = field(default_factory=dict)   # states of the block itself, by name, same layout
+    # states of the block itself, by name, and the several states of a mixer, by "mixer.<name>"; same layout
+    states: Dict[str, torch.Tensor] = field(default_factory=dict)
 
 
 @dataclass
@@ -55,6 +56,7 @@ class CachePlan:
     group_of_entry: Dict[int, int]        # every run-list entry with a paged cache (owned or read)
     state_entries: Dict[int, object]      # run-list entry -> StateSpec of its mixer
     block_states: Dict[int, Dict[str, object]] = field(default_factory=dict)   # run-list entry -> name -> StateSpec
+    embedding_states: Dict[str, object] = field(default_factory=dict)          # name -> StateSpec of the embedding
 
 
 def plan_cache(model, page_size: int, itemsize: int) -> CachePlan:
@@ -72,6 +74,9 @@ def plan_cache(model, page_size: int, itemsize: int) -> CachePlan:
         own = getattr(block, "state_specs", None)
         if own is not None and own():
             block_states[e] = dict(own())
+        several = getattr(mixer, "state_specs", None)
+        if several is not None:
+            block_states.setdefault(e, {}).update({"mixer." + name: spec for name, spec in several().items()})
         kv = mixer.cache_spec()
         if kv is None:
             continue
@@ -87,7 +92,8 @@ def plan_cache(model, page_size: int, itemsize: int) -> CachePlan:
         value_width = 0 if kv.shared_values else (kv.v_head_dim or kv.head_dim)
         groups[g].bytes_per_page += page_size * kv.num_kv_heads * (kv.head_dim + value_width) * itemsize
         group_of_entry[e] = g
-    return CachePlan(groups, group_of_entry, state_entries, block_states)
+    kept = getattr(model.embedding, "state_specs", None)
+    return CachePlan(groups, group_of_entry, state_entries, block_states, dict(kept()) if kept is not None else {})
 
 
 def cache_budget_bytes(free: int, total: int, memory_ratio: float) -> int:
@@ -169,10 +175,13 @@ class PagedCache:
                 cache.states[name] = torch.zeros((max_requests + 1,) + tuple(spec.shape), dtype=spec.dtype,
                                                  device=device)
             self.layer_caches.append(cache)
+        self.embedding = LayerCache()
+        for name, spec in plan.embedding_states.items():
+            self.embedding.states[name] = torch.zeros((max_requests + 1,) + tuple(spec.shape), dtype=spec.dtype, device=device)
 
     def bytes(self) -> int:
         total = 0
-        for c in self.layer_caches:
+        for c in self.layer_caches + [self.embedding]:
             if c.writes and c.k is not None:
                 total += (c.k.numel() + (c.v.numel() if c.v is not None else 0)) * c.k.element_size()
             if c.state is not None:

@@ -6,7 +6,8 @@ from .kefetar import KefetarConfig
 from .mukenex import MukenexConfig
 from .torinex import TorinexConfig
 from .lufizen import LufizenConfig
+from .sigudra import SigudraConfig
 
 __all__ = ["ConfigError", "LayerSpec", "ModelSpec", "PartSpec", "RunEntry", "Architecture",
            "register_architecture", "registered_architectures", "resolve_architecture",
-           "Qwen3Config", "KefetarConfig", "MukenexConfig", "TorinexConfig", "LufizenConfig"]
+           "Qwen3Config", "KefetarConfig", "MukenexConfig", "TorinexConfig", "LufizenConfig", "SigudraConfig"]

@@ -8,7 +8,7 @@ run time: ``register_architecture`` is all that a new architecture needs.
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import Any, Callable, Dict, List, Optional, Sequence
+from typing import Any, Callable, Dict, List, Mapping, Optional, Sequence
 
 from .spec import ConfigError, ModelSpec
 
@@ -24,6 +24,9 @@ class Architecture:
     checkpoint_dtype: Callable[[Any], str] = lambda config: "bfloat16"
     # typed configuration -> token ids that end a generation
     stop_ids: Callable[[Any], Sequence[int]] = lambda config: ()
+    # (raw config.json, checkpoint tensor name -> shape) -> the raw configuration with the sizes that the file leaves to
+    # the tensors' shapes (None: the file gives every size)
+    sizes_from_shapes: Optional[Callable[[dict, Mapping[str, tuple]], dict]] = None
 
 
 _ARCHITECTURES: Dict[str, Architecture] = {}

@@ -151,7 +151,7 @@ static int launch(const void* x, int in_stride, const float* w, int taps, float*
                   void* v_cache, const float* inv_freq, int rot_dim, const int* positions, const int* slots, int nh,
                   int nkv, int d, int dv, int page_size, long long cache_slots, const float* vmix, float* v_first,
                   int v_mode, int tokens, int num_rows, int all_single, int* err, cudaStream_t stream) {
-  TapsInput<T> in;
+  TapsInput<T> in = {};
   in.x = static_cast<const T*>(x); in.in_stride = in_stride; in.scale = nullptr; in.w = w; in.taps = w ? taps : 1;
   in.channels = nh * d + nkv * d + nkv * dv; in.state = state; in.row_of_token = row_of_token; in.cu_q = cu_q;
   in.prefix_len = prefix_len; in.state_slots = state_slots;

@@ -23,6 +23,39 @@ __global__ void embedding_kernel(TA* __restrict__ out, const TW* __restrict__ ta
     dst[i] = ok ? from_f32<TA>(to_f32<TW>(src[i]) * scale) : from_f32<TA>(0.0f);      // scale 1: the row as stored
 }
 
+// out[t] = table[id_t] + pairs[(id_(t-1) * mul_prev + id_t * mul_cur) mod buckets], the sum in float; a sequence's first
+// token takes the last row (`buckets`) of `pairs`.  The token before a row's first token of this step is the row's state
+// (last_token [slots + 1]), which the block of that first token reads and then brings up to date: no other block touches
+// it.  Two's-complement products of 32-bit ids and multipliers fit 64 bits.
+template <typename TA, typename TW>
+__global__ void __launch_bounds__(256)
+pair_embedding_kernel(TA* __restrict__ out, const TW* __restrict__ table, const TW* __restrict__ pairs,
+                      const int* __restrict__ ids, const int* __restrict__ row_of_token, const int* __restrict__ cu_q,
+                      const int* __restrict__ prefix_len, const int* __restrict__ state_slots, int* __restrict__ last_token,
+                      int width, int vocab, int buckets, long long mul_prev, long long mul_cur, int* err) {
+  __shared__ int pair_row;
+  const int t = blockIdx.x;
+  const int id = ids[t];
+  const bool ok = id >= 0 && id < vocab;
+  if (threadIdx.x == 0) {
+    if (!ok) atomicOr(err, B200_ERR_TOKEN_RANGE);
+    const int r = row_of_token[t], first = cu_q[r];
+    int at = buckets;
+    if (t > first || prefix_len[r] > 0) {
+      const long long before = t > first ? ids[t - 1] : last_token[state_slots[r]];
+      const long long m = (before * mul_prev + static_cast<long long>(id) * mul_cur) % buckets;
+      at = static_cast<int>(m < 0 ? m + buckets : m);
+    }
+    if (t == first) last_token[state_slots[r]] = ids[cu_q[r + 1] - 1];
+    pair_row = at;
+  }
+  __syncthreads();
+  const TW* src = table + static_cast<size_t>(ok ? id : 0) * width;
+  const TW* add = pairs + static_cast<size_t>(pair_row) * width;
+  TA* dst = out + static_cast<size_t>(t) * width;
+  for (int i = threadIdx.x; i < width; i += blockDim.x) dst[i] = from_f32<TA>(ok ? to_f32<TW>(src[i]) + to_f32<TW>(add[i]) : 0.0f);
+}
+
 // ------------------------------------------------------------------ norms
 // out[r] = rms_norm(x[src(r)] (+ residual[src(r)])) * w, src(r) = rows ? rows[r] : r.
 // With ADD the rounded sum is written back to residual[src(r)] when write_residual != 0.
@@ -175,6 +208,20 @@ B200_EXPORT int b200_embedding(void* out, const void* table, const int* ids, int
   if (width <= 0 || vocab <= 0) return B200_BAD_SIZE;
 #define CALL(TA, TW) embedding_kernel<TA, TW><<<tokens, 256, 0, stream>>>( \
     static_cast<TA*>(out), static_cast<const TW*>(table), ids, width, vocab, scale, err)
+  DISPATCH2(act_dtype, table_dtype, CALL)
+#undef CALL
+  return b200_check_launch();
+}
+
+B200_EXPORT int b200_pair_embedding(void* out, const void* table, const void* pairs, const int* ids, const int* row_of_token,
+                                    const int* cu_q, const int* prefix_len, const int* state_slots, int* last_token, int tokens,
+                                    int width, int vocab, int buckets, long long mul_prev, long long mul_cur, int act_dtype,
+                                    int table_dtype, int* err, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (width <= 0 || vocab <= 0 || buckets <= 0) return B200_BAD_SIZE;
+#define CALL(TA, TW) pair_embedding_kernel<TA, TW><<<tokens, 256, 0, stream>>>( \
+    static_cast<TA*>(out), static_cast<const TW*>(table), static_cast<const TW*>(pairs), ids, row_of_token, cu_q, prefix_len, \
+    state_slots, last_token, width, vocab, buckets, mul_prev, mul_cur, err)
   DISPATCH2(act_dtype, table_dtype, CALL)
 #undef CALL
   return b200_check_launch();

@@ -5,6 +5,8 @@
 //
 //   expert e:  y = W_down[e] glu(W_gate[e] x, W_up[e] x)          out[t] = sum_k weight_(t, k) y_(t, k) [+ add[t]]
 //   glu(g, u) = silu(g) u,  or  g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit), u' = clamp(u, -limit, limit)
+// or, with the weights on the experts' INPUTS:  y = W_down[e] glu(W_gate[e] (weight x), W_up[e] (weight x)),
+// out[t] = sum_k y_(t, k): the weight is one number a pair, so it multiplies the two sums before glu, in float.
 //
 // Four kernels behind the choice, nothing goes through the host (a step can be captured in a graph):
 //   expert_route       (token, choice) pairs sorted by expert: sorted_token[pos], pos_of_pair[pair], the experts'
@@ -39,7 +41,8 @@ __global__ void __launch_bounds__(1024)
 expert_route_kernel(const int* __restrict__ token_ids, const int* __restrict__ table, int vocab, int top, int experts,
                     const int* __restrict__ choice, int tokens, int* __restrict__ sorted_token, int* __restrict__ pos_of_pair,
                     int* __restrict__ expert_start, int* __restrict__ tile_expert, int* __restrict__ tile_first,
-                    int* __restrict__ num_tiles, int tile_rows, int* err) {
+                    int* __restrict__ num_tiles, int tile_rows, const float* __restrict__ weight,
+                    float* __restrict__ sorted_gain, int* err) {
   pdl_launch_dependents();                          // the kernel after this one may be scheduled; it waits before it reads
   pdl_wait();                                        // what this kernel reads belongs to the kernels before it
   extern __shared__ int sm[];
@@ -75,6 +78,7 @@ expert_route_kernel(const int* __restrict__ token_ids, const int* __restrict__ t
     const int pos = start[e] + atomicAdd(&count[e], 1);
     sorted_token[pos] = i / top;
     pos_of_pair[i] = pos;
+    if (sorted_gain != nullptr) sorted_gain[pos] = weight[i];
   }
 }
 
@@ -82,9 +86,11 @@ __device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z));
 
 // What joins an expert's gate and up projections.  kind 0: silu(g) u.  kind 1: g' sigmoid(alpha g') (u' + 1) with
 // g' = min(g, limit), u' = clamp(u, -limit, limit).
+// gain (null: none): one number a sorted pair, which multiplies both projections of its row.
 struct GluAct {
   int kind;
   float limit, alpha;
+  const float* gain;
 };
 __device__ __forceinline__ float glu_f(float g, float u, const GluAct a) {
   if (a.kind == 0) return silu_f(g) * u;
@@ -92,6 +98,7 @@ __device__ __forceinline__ float glu_f(float g, float u, const GluAct a) {
   u = fminf(fmaxf(u, -a.limit), a.limit);
   return g / (1.0f + expf(-a.alpha * g)) * (u + 1.0f);
 }
+__device__ __forceinline__ float row_gain(const GluAct a, int row) { return a.gain != nullptr ? a.gain[row] : 1.0f; }
 
 // ------------------------------------------------------------------ float32 products
 // GATED: C[pos][n] = silu(A . Wg[n]) * (A . Wu[n]) with A rows gathered by sorted_token; else C[pos][n] = A[pos] . W[n].
@@ -161,11 +168,12 @@ expert_gemm_f32_kernel(const float* __restrict__ A, int lda, const int* __restri
   for (int i = 0; i < 4; ++i) {
     const int r = r0 + ty * 4 + i;
     if (r >= r_end) continue;
+    const float w = GATED ? row_gain(act, r) : 1.0f;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
       if (n >= N) continue;
-      if constexpr (GATED) C[static_cast<size_t>(r) * N + n] = glu_f(acc[0][i][j], acc[1][i][j], act);
+      if constexpr (GATED) C[static_cast<size_t>(r) * N + n] = glu_f(w * acc[0][i][j], w * acc[1][i][j], act);
       else C[static_cast<size_t>(r) * N + n] = acc[0][i][j];
     }
   }
@@ -260,6 +268,24 @@ expert_gemm_bf16_kernel(const __nv_bfloat16* __restrict__ A, int lda, const int*
         }
     }
   }
+  if constexpr (GATED) {
+    if (act.gain != nullptr) {      // a matrix whose rows hold the rows' gains, in the accumulators' layout
+      wmma::fragment<wmma::accumulator, 16, 16, 16, float> fg;
+      for (int i = lane; i < 16 * 16; i += 32) {
+        const int r = r0 + wr * 16 + (i >> 4);
+        Cs[warp][i >> 4][i & 15] = r < r_end ? act.gain[r] : 0.0f;
+      }
+      __syncwarp();
+      wmma::load_matrix_sync(fg, &Cs[warp][0][0], 32 + 4, wmma::mem_row_major);
+#pragma unroll
+      for (int g = 0; g < G; ++g)
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int i = 0; i < fg.num_elements; ++i) acc[g][j].x[i] *= fg.x[i];
+      __syncwarp();
+    }
+  }
 #pragma unroll
   for (int j = 0; j < 2; ++j) {
     if constexpr (GATED) {          // both accumulators have one layout: element i of one meets element i of the other
@@ -332,8 +358,10 @@ expert_rows_few_kernel(const __nv_bfloat16* __restrict__ A, int lda, const int* 
     for (int i = 0; i < FEW_ROWS; ++i) {
       const float s0 = warp_sum(acc0[i]);
       const float s1 = GATED ? warp_sum(acc1[i]) : 0.0f;
-      if (lane == 0 && i < nr)
-        C[static_cast<size_t>(r0 + i) * ldc + n] = from_f32<TO>(GATED ? glu_f(s0, s1, act) : s0);
+      if (lane == 0 && i < nr) {
+        const float w = GATED ? row_gain(act, r0 + i) : 1.0f;
+        C[static_cast<size_t>(r0 + i) * ldc + n] = from_f32<TO>(GATED ? glu_f(w * s0, w * s1, act) : s0);
+      }
     }
   }
 }
@@ -614,12 +642,13 @@ expert_router_kernel(const TX* __restrict__ x, const TW* __restrict__ W, int tok
 B200_EXPORT long long b200_expert_route_ints(int tokens, int top, int experts) {
   const long long pairs = static_cast<long long>(tokens) * top;
   const long long tiles = (pairs + TM - 1) / TM + experts;
-  return 2 * pairs + (experts + 1) + 2 * tiles + 1;
+  return 3 * pairs + (experts + 1) + 2 * tiles + 1;
 }
 
 // Where the parts of the routing scratch lie.
 struct RouteLayout {
   int *sorted_token, *pos_of_pair, *expert_start, *tile_expert, *tile_first, *num_tiles;
+  float* sorted_gain;          // used when the weights multiply the experts' inputs
   int tiles;
 };
 static RouteLayout route_layout(int* route, int pairs, int experts) {
@@ -631,6 +660,7 @@ static RouteLayout route_layout(int* route, int pairs, int experts) {
   r.tile_expert = r.expert_start + experts + 1;
   r.tile_first = r.tile_expert + r.tiles;
   r.num_tiles = r.tile_first + r.tiles;
+  r.sorted_gain = reinterpret_cast<float*>(r.num_tiles + 1);
   return r;
 }
 
@@ -644,23 +674,25 @@ struct ExpertChoice {
   const void* add;
   int add_dtype;
   const float* add_scale;      // null, or one factor a token for `add`
+  bool weight_on_input;        // the weights multiply the experts' inputs; the outputs are summed as they are
 };
 
 static int launch_combine(float* out, const float* y, const int* pos_of_pair, int tokens, int top, int width,
                           const ExpertChoice& c, cudaStream_t stream) {
-  const float uniform = 1.0f / static_cast<float>(top);
+  const float uniform = c.weight_on_input ? 1.0f : 1.0f / static_cast<float>(top);
+  const float* weight = c.weight_on_input ? nullptr : c.weight;
   const dim3 combine_grid(tokens, (width + 1023) / 1024);
   if (c.add != nullptr && c.add_dtype == B200_BF16)
     return b200_launch(expert_combine_kernel<__nv_bfloat16>, combine_grid, dim3(256), 0, stream, 0, out, y, pos_of_pair,
-                       top, width, uniform, c.weight, static_cast<const __nv_bfloat16*>(c.add), c.add_scale);
+                       top, width, uniform, weight, static_cast<const __nv_bfloat16*>(c.add), c.add_scale);
   return b200_launch(expert_combine_kernel<float>, combine_grid, dim3(256), 0, stream, 0, out, y, pos_of_pair, top, width,
-                     uniform, c.weight, static_cast<const float*>(c.add), c.add_scale);
+                     uniform, weight, static_cast<const float*>(c.add), c.add_scale);
 }
 
 // x [tokens, width] -> out [tokens, width] float32.  `h` holds pairs * ff elements of x's dtype, `y` pairs * width
 // floats, `route` b200_expert_route_ints(...) ints.
 static int run_experts(const void* x, int dtype, const ExpertChoice& c, int top, int experts, const void* gate_up,
-                       const void* down, int tokens, int width, int ff, const GluAct act, void* h, float* y, int* route,
+                       const void* down, int tokens, int width, int ff, GluAct act, void* h, float* y, int* route,
                        float* out, int* err, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (top <= 0 || experts <= 0 || width <= 0 || ff <= 0 || (c.choice == nullptr && c.vocab <= 0)) return B200_BAD_SIZE;
@@ -669,12 +701,14 @@ static int run_experts(const void* x, int dtype, const ExpertChoice& c, int top,
   const int pairs = static_cast<int>(pairs_ll);
   const RouteLayout rl = route_layout(route, pairs, experts);
   const int tiles = rl.tiles;
+  act.gain = c.weight_on_input ? rl.sorted_gain : nullptr;
   if (tiles > 65535) return B200_BAD_SIZE;
   int *sorted_token = rl.sorted_token, *pos_of_pair = rl.pos_of_pair, *expert_start = rl.expert_start;
   int *tile_expert = rl.tile_expert, *tile_first = rl.tile_first, *num_tiles = rl.num_tiles;
   int rc = b200_launch(expert_route_kernel, dim3(1), dim3(1024), (2 * experts + 1) * sizeof(int), stream, 0,
                        c.token_ids, c.table, c.vocab, top, experts, c.choice, tokens, sorted_token, pos_of_pair,
-                       expert_start, tile_expert, tile_first, num_tiles, TM, err);
+                       expert_start, tile_expert, tile_first, num_tiles, TM, c.weight,
+                       c.weight_on_input ? rl.sorted_gain : static_cast<float*>(nullptr), err);
   if (rc != 0) return rc;
   const dim3 g1((ff + TN - 1) / TN, tiles), g2((width + TN - 1) / TN, tiles);
   const long long gu_stride = 2ll * ff * width, dn_stride = static_cast<long long>(width) * ff;
@@ -713,8 +747,8 @@ static int run_experts(const void* x, int dtype, const ExpertChoice& c, int top,
 B200_EXPORT int b200_table_experts(const void* x, int dtype, const int* token_ids, const int* table, int vocab, int top,
                                    int experts, const void* gate_up, const void* down, int tokens, int width, int ff,
                                    void* h, float* y, int* route, float* out, int* err, cudaStream_t stream) {
-  const ExpertChoice c = {token_ids, table, vocab, nullptr, nullptr, nullptr, B200_F32, nullptr};
-  return run_experts(x, dtype, c, top, experts, gate_up, down, tokens, width, ff, GluAct{0, 0.0f, 0.0f}, h, y, route,
+  const ExpertChoice c = {token_ids, table, vocab, nullptr, nullptr, nullptr, B200_F32, nullptr, false};
+  return run_experts(x, dtype, c, top, experts, gate_up, down, tokens, width, ff, GluAct{0, 0.0f, 0.0f, nullptr}, h, y, route,
                      out, err, stream);
 }
 
@@ -756,14 +790,15 @@ B200_EXPORT int b200_expert_router(const void* x, int x_dtype, const void* w, in
 
 // Experts chosen by a router: choice and weight [tokens, top] (b200_expert_router), glu kind `act_kind` with `limit`
 // and `alpha`, `add` (null, or [tokens, width] of add_dtype: what every token gets besides, e.g. a shared expert),
-// `add_scale` (null, or one float a token that multiplies its row of `add`).
+// `add_scale` (null, or one float a token that multiplies its row of `add`), `weight_on_input` (the weights multiply the
+// experts' inputs instead of their outputs).
 B200_EXPORT int b200_routed_experts(const void* x, int dtype, const int* choice, const float* weight, int top,
                                     int experts, const void* gate_up, const void* down, int tokens, int width, int ff,
                                     int act_kind, float limit, float alpha, const void* add, int add_dtype,
-                                    const float* add_scale, void* h, float* y, int* route, float* out, int* err,
-                                    cudaStream_t stream) {
+                                    const float* add_scale, int weight_on_input, void* h, float* y, int* route, float* out,
+                                    int* err, cudaStream_t stream) {
   if (choice == nullptr || weight == nullptr || act_kind < 0 || act_kind > 1) return B200_BAD_SIZE;
-  const ExpertChoice c = {nullptr, nullptr, 0, choice, weight, add, add_dtype, add_scale};
-  return run_experts(x, dtype, c, top, experts, gate_up, down, tokens, width, ff, GluAct{act_kind, limit, alpha}, h, y,
+  const ExpertChoice c = {nullptr, nullptr, 0, choice, weight, add, add_dtype, add_scale, weight_on_input != 0};
+  return run_experts(x, dtype, c, top, experts, gate_up, down, tokens, width, ff, GluAct{act_kind, limit, alpha, nullptr}, h, y,
                      route, out, err, stream);
 }

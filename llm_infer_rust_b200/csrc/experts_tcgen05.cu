@@ -144,8 +144,9 @@ expert_gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap amap, const __gri
           if (row_ok && col0 < cols) {
             TO* dst = out + static_cast<size_t>(row) * cols + col0;
             __align__(16) bf16 r[32];
+            const float w = row_gain(act, row);
 #pragma unroll
-            for (int e = 0; e < 32; ++e) r[e] = __float2bfloat16_rn(glu_f(g[e], u[e], act));
+            for (int e = 0; e < 32; ++e) r[e] = __float2bfloat16_rn(glu_f(w * g[e], w * u[e], act));
             if (col0 + 32 <= cols && (cols % 8) == 0) {
 #pragma unroll
               for (int q = 0; q < 4; ++q) *reinterpret_cast<uint4*>(dst + q * 8) = *reinterpret_cast<const uint4*>(r + q * 8);
@@ -171,7 +172,7 @@ expert_gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap amap, const __gri
 // The same as run_experts for bfloat16 with width and ff multiples of 8; `xs` holds pairs * width more elements (the
 // gathered rows).  gate_up [experts * 2 ff, width] and down [experts * width, ff] as stacked matrices.
 static int run_experts_tcgen05(const void* x, const ExpertChoice& c, int top, int experts, const void* gate_up,
-                               const void* down, int tokens, int width, int ff, const GluAct act, void* xs, void* h,
+                               const void* down, int tokens, int width, int ff, GluAct act, void* xs, void* h,
                                float* y, int* route, float* out, int* err, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (top <= 0 || experts <= 0 || width <= 0 || ff <= 0 || (c.choice == nullptr && c.vocab <= 0) || width % 8 || ff % 8)
@@ -180,9 +181,11 @@ static int run_experts_tcgen05(const void* x, const ExpertChoice& c, int top, in
   if (pairs_ll > (1ll << 30) || (2 * experts + 1) * sizeof(int) > 48 * 1024) return B200_BAD_SIZE;
   const int pairs = static_cast<int>(pairs_ll);
   const RouteLayout rl = route_layout(route, pairs, experts);
+  act.gain = c.weight_on_input ? rl.sorted_gain : nullptr;
   expert_route_kernel<<<1, 1024, (2 * experts + 1) * sizeof(int), stream>>>(
       c.token_ids, c.table, c.vocab, top, experts, c.choice, tokens, rl.sorted_token, rl.pos_of_pair, rl.expert_start,
-      rl.tile_expert, rl.tile_first, rl.num_tiles, TC_ROWS, err);
+      rl.tile_expert, rl.tile_first, rl.num_tiles, TC_ROWS, c.weight,
+      c.weight_on_input ? rl.sorted_gain : nullptr, err);
   int rc = b200_check_launch();
   if (rc != 0) return rc;
   gather_rows_kernel<<<pairs, 256, 0, stream>>>(static_cast<bf16*>(xs), static_cast<const bf16*>(x), rl.sorted_token, width);
@@ -219,8 +222,8 @@ B200_EXPORT int b200_table_experts_tcgen05(const void* x, const int* token_ids, 
                                            int experts, const void* gate_up, const void* down, int tokens, int width,
                                            int ff, void* xs, void* h, float* y, int* route, float* out, int* err,
                                            cudaStream_t stream) {
-  const ExpertChoice c = {token_ids, table, vocab, nullptr, nullptr, nullptr, B200_F32, nullptr};
-  return run_experts_tcgen05(x, c, top, experts, gate_up, down, tokens, width, ff, GluAct{0, 0.0f, 0.0f}, xs, h, y,
+  const ExpertChoice c = {token_ids, table, vocab, nullptr, nullptr, nullptr, B200_F32, nullptr, false};
+  return run_experts_tcgen05(x, c, top, experts, gate_up, down, tokens, width, ff, GluAct{0, 0.0f, 0.0f, nullptr}, xs, h, y,
                              route, out, err, stream);
 }
 
@@ -228,10 +231,10 @@ B200_EXPORT int b200_table_experts_tcgen05(const void* x, const int* token_ids, 
 B200_EXPORT int b200_routed_experts_tcgen05(const void* x, const int* choice, const float* weight, int top, int experts,
                                             const void* gate_up, const void* down, int tokens, int width, int ff,
                                             int act_kind, float limit, float alpha, const void* add, int add_dtype,
-                                            const float* add_scale, void* xs, void* h, float* y, int* route, float* out, int* err,
-                                            cudaStream_t stream) {
+                                            const float* add_scale, int weight_on_input, void* xs, void* h, float* y,
+                                            int* route, float* out, int* err, cudaStream_t stream) {
   if (choice == nullptr || weight == nullptr || act_kind < 0 || act_kind > 1) return B200_BAD_SIZE;
-  const ExpertChoice c = {nullptr, nullptr, 0, choice, weight, add, add_dtype, add_scale};
-  return run_experts_tcgen05(x, c, top, experts, gate_up, down, tokens, width, ff, GluAct{act_kind, limit, alpha}, xs,
+  const ExpertChoice c = {nullptr, nullptr, 0, choice, weight, add, add_dtype, add_scale, weight_on_input != 0};
+  return run_experts_tcgen05(x, c, top, experts, gate_up, down, tokens, width, ff, GluAct{act_kind, limit, alpha, nullptr}, xs,
                              h, y, route, out, err, stream);
 }

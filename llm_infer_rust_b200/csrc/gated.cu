@@ -113,7 +113,7 @@ poly_norm_vec_kernel(T* __restrict__ out, const T* __restrict__ z, const float* 
 template <typename T>
 __global__ void __launch_bounds__(128)
 head_unit_norm_gate_kernel(T* __restrict__ out, const float* __restrict__ o, const T* __restrict__ g, int g_stride,
-                           int heads, int dv, float eps, long long vectors) {
+                           int heads, int dv, float eps, const float* __restrict__ w, int sigmoid_gate, long long vectors) {
   const long long vec = static_cast<long long>(blockIdx.x) * 4 + (threadIdx.x >> 5);
   if (vec >= vectors) return;
   const int lane = threadIdx.x & 31;
@@ -128,7 +128,8 @@ head_unit_norm_gate_kernel(T* __restrict__ out, const float* __restrict__ o, con
   T* dst = out + (t * heads + h) * dv;
   for (int j = lane; j < dv; j += 32) {
     const float x = to_f32<T>(gate[j]);
-    dst[j] = from_f32<T>(src[j] * r * (x / (1.0f + expf(-x))));
+    const float gain = w != nullptr ? w[j] : 1.0f;
+    dst[j] = from_f32<T>(src[j] * r * gain * ((sigmoid_gate ? 1.0f : x) / (1.0f + expf(-x))));
   }
 }
 
@@ -170,18 +171,19 @@ B200_EXPORT int b200_poly_norm(void* out, const void* z, const float* coef, floa
 }
 
 B200_EXPORT int b200_head_unit_norm_gate(void* out, const float* o, const void* g, int g_stride, int tokens, int heads,
-                                         int dv, float eps, int dtype, cudaStream_t stream) {
+                                         int dv, float eps, const float* w, int sigmoid_gate, int dtype, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (heads <= 0 || dv <= 0) return B200_BAD_SIZE;
   const long long vectors = static_cast<long long>(tokens) * heads;
   const unsigned blocks = static_cast<unsigned>((vectors + 3) / 4);
   if (dtype == B200_F32)
     head_unit_norm_gate_kernel<float><<<blocks, 128, 0, stream>>>(static_cast<float*>(out), o,
-                                                                   static_cast<const float*>(g), g_stride, heads, dv, eps,
-                                                                   vectors);
+                                                                   static_cast<const float*>(g), g_stride, heads, dv, eps, w,
+                                                                   sigmoid_gate, vectors);
   else if (dtype == B200_BF16)
     head_unit_norm_gate_kernel<__nv_bfloat16><<<blocks, 128, 0, stream>>>(
-        static_cast<__nv_bfloat16*>(out), o, static_cast<const __nv_bfloat16*>(g), g_stride, heads, dv, eps, vectors);
+        static_cast<__nv_bfloat16*>(out), o, static_cast<const __nv_bfloat16*>(g), g_stride, heads, dv, eps, w,
+        sigmoid_gate, vectors);
   else
     return B200_BAD_DTYPE;
   return b200_check_launch();
@@ -324,9 +326,10 @@ B200_EXPORT int b200_tanh_cap(float* z, long long n, float cap, cudaStream_t str
 
 // ------------------------------------------------------------------ gate and up joined; an activation times a table row
 // out[t][c] = glu(gate_up[t][c], gate_up[t][ff + c]).  kind 0: silu(g) u.  kind 1: g' sigmoid(alpha g') (u' + 1) with
-// g' = min(g, limit), u' = clamp(u, -limit, limit).  Computed in float, rounded once.
+// g' = min(g, limit), u' = clamp(u, -limit, limit).  kind 2: gelu_tanh(g) u.  Computed in float, rounded once.
 __device__ __forceinline__ float glu_join(float g, float u, int kind, float limit, float alpha) {
   if (kind == 0) return g / (1.0f + expf(-g)) * u;
+  if (kind == 2) return activate(g, ACT_GELU_TANH) * u;
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
   return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
@@ -394,7 +397,7 @@ B200_EXPORT int b200_glu_columns(void* out, const void* gate_up, int tokens, int
                                  int dtype, cudaStream_t stream) {
   int launch_rc = 0;
   if (tokens <= 0 || ff <= 0) return 0;
-  if (kind < 0 || kind > 1) return B200_BAD_SIZE;
+  if (kind < 0 || kind > 2) return B200_BAD_SIZE;
   if (ff % 8 == 0) {
     const dim3 wide(tokens, (ff / 8 + 255) / 256);
     if (dtype == B200_F32)

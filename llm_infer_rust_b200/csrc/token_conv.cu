@@ -4,7 +4,7 @@
 //   residual_scale   x[t] += y[t] (optional, the sum in float), s[t] = gain / sqrt(mean(x[t]^2) + eps)
 //   scaled_rows      out[r] = x[rows[r]] * s[rows[r]]                       (the norm itself, for chosen rows)
 //   causal_taps      y[t][c] = (identity ? u[t][c] : 0) + sum_j w[c][j] * u[t - taps + 1 + j][c],
-//                    u[t][c] = in[t][c] * (s ? s[t] : 1)
+//                    u[t][c] = in[t][c] * (s ? s[t] : 1) (+ a bias per channel), y (+ a bias per channel)
 //   taps_state_update   the last taps - 1 inputs u of every row become the row's state
 //   add_norm_taps_single   the first, the third and the fourth in one kernel, for steps whose rows have one token
 //
@@ -53,12 +53,12 @@ scaled_rows_kernel(TO* __restrict__ out, const float* __restrict__ x, const floa
 // grid (tokens, channel tiles of 256)
 template <typename TI, typename TO>
 __global__ void __launch_bounds__(256)
-causal_taps_kernel(TapsInput<TI> in, TO* __restrict__ out, int out_stride, int identity) {
+causal_taps_kernel(TapsInput<TI> in, TO* __restrict__ out, int out_stride, int identity, const float* __restrict__ out_bias) {
   const int t = blockIdx.x;
   const int c = blockIdx.y * blockDim.x + threadIdx.x;
   if (c >= in.channels) return;
   const TapsRow row = taps_row(in, t);
-  const float y = taps_value(in, row, t, c, identity != 0);
+  const float y = taps_value(in, row, t, c, identity != 0) + (out_bias ? out_bias[c] : 0.0f);
   out[static_cast<size_t>(t) * out_stride + c] = from_f32<TO>(y);
 }
 
@@ -66,13 +66,19 @@ causal_taps_kernel(TapsInput<TI> in, TO* __restrict__ out, int out_stride, int i
 // also brings the row's state up to date (see taps_value8)
 template <typename TI, typename TO>
 __global__ void __launch_bounds__(128)
-causal_taps_vec_kernel(TapsInput<TI> in, TO* __restrict__ out, int out_stride, int identity) {
+causal_taps_vec_kernel(TapsInput<TI> in, TO* __restrict__ out, int out_stride, int identity, const float* __restrict__ out_bias) {
   const int t = blockIdx.x;
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 8;
   if (c >= in.channels) return;
   const TapsRow row = taps_row(in, t);
   float y[8];
   taps_value8(in, row, t, c, identity != 0, taps_single(in, t), y);
+  if (out_bias != nullptr) {
+    float b[8];
+    load_floats<float, 8>(out_bias + c, b);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) y[i] += b[i];
+  }
   store8<TO>(out + static_cast<size_t>(t) * out_stride + c, y);
 }
 
@@ -143,18 +149,19 @@ B200_EXPORT int b200_scaled_rows(void* out, int out_dtype, const float* x, const
 
 template <typename TI>
 static int launch_taps(const TapsInput<TI>& in, void* out, int out_dtype, int out_stride, int identity, int tokens,
-                       int num_rows, int update_state, int all_single, cudaStream_t stream) {
+                       int num_rows, int update_state, int all_single, const float* out_bias, cudaStream_t stream) {
   const dim3 grid(tokens, (in.channels + 255) / 256);
   const bool vec = update_state && in.channels % 8 == 0 && in.in_stride % 8 == 0 && out_stride % 8 == 0 &&
                    (reinterpret_cast<uintptr_t>(in.x) | reinterpret_cast<uintptr_t>(out) |
-                    reinterpret_cast<uintptr_t>(in.state)) % 16 == 0;
+                    reinterpret_cast<uintptr_t>(in.state) | reinterpret_cast<uintptr_t>(in.bias) |
+                    reinterpret_cast<uintptr_t>(out_bias)) % 16 == 0;
   if (vec) {
     const dim3 vgrid(tokens, (in.channels / 8 + 127) / 128);
     if (out_dtype == B200_F32)
-      causal_taps_vec_kernel<TI, float><<<vgrid, 128, 0, stream>>>(in, static_cast<float*>(out), out_stride, identity);
+      causal_taps_vec_kernel<TI, float><<<vgrid, 128, 0, stream>>>(in, static_cast<float*>(out), out_stride, identity, out_bias);
     else if (out_dtype == B200_BF16)
       causal_taps_vec_kernel<TI, __nv_bfloat16><<<vgrid, 128, 0, stream>>>(in, static_cast<__nv_bfloat16*>(out),
-                                                                          out_stride, identity);
+                                                                          out_stride, identity, out_bias);
     else
       return B200_BAD_DTYPE;
     int rc = b200_check_launch();
@@ -164,10 +171,10 @@ static int launch_taps(const TapsInput<TI>& in, void* out, int out_dtype, int ou
     return b200_check_launch();
   }
   if (out_dtype == B200_F32)
-    causal_taps_kernel<TI, float><<<grid, 256, 0, stream>>>(in, static_cast<float*>(out), out_stride, identity);
+    causal_taps_kernel<TI, float><<<grid, 256, 0, stream>>>(in, static_cast<float*>(out), out_stride, identity, out_bias);
   else if (out_dtype == B200_BF16)
     causal_taps_kernel<TI, __nv_bfloat16><<<grid, 256, 0, stream>>>(in, static_cast<__nv_bfloat16*>(out), out_stride,
-                                                                    identity);
+                                                                    identity, out_bias);
   else
     return B200_BAD_DTYPE;
   int rc = b200_check_launch();
@@ -180,8 +187,9 @@ static int launch_taps(const TapsInput<TI>& in, void* out, int out_dtype, int ou
 template <typename TI>
 static TapsInput<TI> taps_input(const void* x, int in_stride, const float* scale, const float* w, int taps,
                                 int channels, float* state, const int* row_of_token, const int* cu_q,
-                                const int* prefix_len, const int* state_slots) {
+                                const int* prefix_len, const int* state_slots, const float* bias = nullptr) {
   TapsInput<TI> in;
+  in.bias = bias;
   in.x = static_cast<const TI*>(x); in.in_stride = in_stride; in.scale = scale; in.w = w; in.taps = taps;
   in.channels = channels; in.state = state; in.row_of_token = row_of_token; in.cu_q = cu_q;
   in.prefix_len = prefix_len; in.state_slots = state_slots;
@@ -195,18 +203,18 @@ B200_EXPORT int b200_causal_taps(const void* x, int in_dtype, int in_stride, con
                                  int taps, int channels, float* state, const int* row_of_token, const int* cu_q,
                                  const int* prefix_len, const int* state_slots, void* out, int out_dtype,
                                  int out_stride, int identity, int tokens, int num_rows, int update_state,
-                                 int all_single, cudaStream_t stream) {
+                                 int all_single, const float* in_bias, const float* out_bias, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (channels <= 0 || taps < 1 || taps > TAPS_MAX || num_rows <= 0) return B200_BAD_SIZE;
   if ((channels + 255) / 256 > 65535) return B200_BAD_SIZE;
   if (in_dtype == B200_F32)
     return launch_taps<float>(taps_input<float>(x, in_stride, scale, w, taps, channels, state, row_of_token, cu_q,
-                                                prefix_len, state_slots),
-                              out, out_dtype, out_stride, identity, tokens, num_rows, update_state, all_single, stream);
+                                                prefix_len, state_slots, in_bias),
+                              out, out_dtype, out_stride, identity, tokens, num_rows, update_state, all_single, out_bias, stream);
   if (in_dtype == B200_BF16)
     return launch_taps<__nv_bfloat16>(taps_input<__nv_bfloat16>(x, in_stride, scale, w, taps, channels, state,
-                                                                row_of_token, cu_q, prefix_len, state_slots),
-                                      out, out_dtype, out_stride, identity, tokens, num_rows, update_state, all_single, stream);
+                                                                row_of_token, cu_q, prefix_len, state_slots, in_bias),
+                                      out, out_dtype, out_stride, identity, tokens, num_rows, update_state, all_single, out_bias, stream);
   return B200_BAD_DTYPE;
 }
 

@@ -10,6 +10,7 @@ struct TapsInput {
   const TI* x;               // [tokens, in_stride]; channel c of token t at x[t * in_stride + c]
   int in_stride;
   const float* scale;        // per token, or null
+  const float* bias;         // per channel, or null: the input is x * scale + bias (zeros before the start all the same)
   const float* w;            // [channels, taps]
   int taps;
   int channels;
@@ -41,7 +42,8 @@ template <typename TI>
 __device__ __forceinline__ float taps_past(const TapsInput<TI>& in, const TapsRow& row, int t, int c, int back) {
   if (back <= row.local) {
     const int s = t - back;
-    return to_f32<TI>(in.x[static_cast<size_t>(s) * in.in_stride + c]) * (in.scale ? in.scale[s] : 1.0f);
+    return to_f32<TI>(in.x[static_cast<size_t>(s) * in.in_stride + c]) * (in.scale ? in.scale[s] : 1.0f) +
+           (in.bias ? in.bias[c] : 0.0f);
   }
   if (!row.has_past) return 0.0f;
   const int k = in.taps - 1 - (back - row.local);       // state k holds the input (taps - 1 - k) before the row's first token
@@ -95,6 +97,12 @@ __device__ __forceinline__ void taps_value8_n(const TapsInput<T>& in, const Taps
 #pragma unroll
     for (int i = 0; i < 8; ++i) now[i] *= s;
   }
+  float shift[8];
+  if (in.bias != nullptr) {
+    load_floats<float, 8>(in.bias + c, shift);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) now[i] += shift[i];
+  }
 #pragma unroll
   for (int i = 0; i < 8; ++i) y[i] = identity ? now[i] : 0.0f;
   if (in.w == nullptr) {
@@ -120,6 +128,10 @@ __device__ __forceinline__ void taps_value8_n(const TapsInput<T>& in, const Taps
         const float s = in.scale[t - back];
 #pragma unroll
         for (int i = 0; i < 8; ++i) u[i] *= s;
+      }
+      if (in.bias != nullptr) {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) u[i] += shift[i];
       }
     } else if (row.has_past) {
       load_floats<float, 8>(st + static_cast<size_t>(hist - (back - row.local)) * in.channels + c, u);
@@ -179,7 +191,8 @@ taps_state_update_kernel(TapsInput<TI> in, int num_rows, int skip_single) {
     float v = 0.0f;
     if (pos >= prefix) {
       const int t = first + (pos - prefix);
-      v = to_f32<TI>(in.x[static_cast<size_t>(t) * in.in_stride + c]) * (in.scale ? in.scale[t] : 1.0f);
+      v = to_f32<TI>(in.x[static_cast<size_t>(t) * in.in_stride + c]) * (in.scale ? in.scale[t] : 1.0f) +
+          (in.bias ? in.bias[c] : 0.0f);
     } else if (pos >= 0 && prefix > 0) {
       v = st[static_cast<size_t>(pos - prefix + hist) * in.channels + c];
     }

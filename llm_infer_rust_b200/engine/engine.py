@@ -28,7 +28,7 @@ from ..kernels import ops
 from ..kernels.build import load_host_runtime
 from ..parts import DecoderModel
 from ..sampling import Sampler, SamplingParams
-from ..weights.loader import load_weights, read_config_json
+from ..weights.loader import load_weights, read_model_config
 from ..weights.random_init import bind_random_weights
 from .context import StepContext, context_from_layout
 
@@ -157,8 +157,11 @@ class Engine:
             log.addHandler(handler)
         if model_path is None and random_weights_config is None:
             raise ConfigError("a model folder (or random_weights_config) is needed")
-        raw = dict(random_weights_config) if model_path is None else read_config_json(model_path)
-        self.arch = resolve_architecture(raw)
+        if model_path is None:
+            raw = dict(random_weights_config)
+            self.arch = resolve_architecture(raw)
+        else:
+            self.arch, raw = read_model_config(model_path)
         self.config = self.arch.parse_config(raw)
         self.raw_config = raw
         spec = self.arch.model_spec(self.config)
@@ -368,7 +371,7 @@ class Engine:
             dev[layout.off_tokens:layout.off_tokens + layout.num_tokens].copy_(device_tokens, non_blocking=True)
         ctx = self._context(layout, dev, host, layout.max_kv_len)
         self._launched = True
-        return self.model.forward(ctx, self.cache.layer_caches)
+        return self.model.forward(ctx, self.cache.layer_caches, self.cache.embedding)
 
     def _shape_graph(self, key: tuple) -> Optional[_DecodeGraph]:
         g = self._shape_graphs.get(key)
@@ -424,12 +427,12 @@ class Engine:
             side.wait_stream(torch.cuda.current_stream())
             before = ops.launch_count()
             with torch.cuda.stream(side):
-                self.model.forward(g.ctx, self.cache.layer_caches)
+                self.model.forward(g.ctx, self.cache.layer_caches, self.cache.embedding)
             torch.cuda.current_stream().wait_stream(side)
             torch.cuda.synchronize(self.device)
             graph = torch.cuda.CUDAGraph()
             with ops.graph_capture(graph):
-                g.logits = self.model.forward(g.ctx, self.cache.layer_caches)
+                g.logits = self.model.forward(g.ctx, self.cache.layer_caches, self.cache.embedding)
             g.launches = (ops.launch_count() - before) // 2
             ops.add_launches(-2 * g.launches)    # a warm-up on throw-away rows and a capture: not the model's work
             g.graph = graph

@@ -186,6 +186,26 @@ def embedding(ids: torch.Tensor, table: torch.Tensor, out_dtype: torch.dtype, sc
     return out
 
 
+def pair_embedding(ids: torch.Tensor, table: torch.Tensor, pairs: torch.Tensor, last_token: torch.Tensor, ctx,
+                   buckets: int, mul_prev: int, mul_cur: int, out_dtype: torch.dtype) -> torch.Tensor:
+    """out[t] = table[id_t] + pairs[(id_(t-1) * mul_prev + id_t * mul_cur) mod buckets], the sum in float; a sequence's
+    first token takes row ``buckets`` (the last) of ``pairs``.  ``last_token`` (int32 [slots + 1, 1]): the token before a
+    row's first one of this step is read there, and the row's last one left there."""
+    _cuda(ids, table, pairs, last_token)
+    _contig(ids, table, pairs, last_token)
+    _i32(ids, last_token)
+    if table.dtype != pairs.dtype or tuple(pairs.shape) != (buckets + 1, table.shape[1]) or last_token[0].numel() != 1:
+        raise KernelError("pair_embedding: the second table must be [buckets + 1, width] in the first one's dtype")
+    out = torch.empty((ids.numel(), table.shape[1]), dtype=out_dtype, device=table.device)
+    rc = _elementwise().b200_pair_embedding(
+        _p(out), _p(table), _p(pairs), _p(ids), _p(ctx.row_of_token), _p(ctx.cu_q), _p(ctx.prefix_len),
+        _p(ctx.state_slots), _p(last_token), ids.numel(), table.shape[1], table.shape[0], int(buckets),
+        ctypes.c_longlong(mul_prev), ctypes.c_longlong(mul_cur), _code(out), _code(table),
+        _p(error_word(table.device)), _stream())
+    _ok(rc, "pair_embedding")
+    return out
+
+
 def rms_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: Optional[torch.Tensor] = None,
              rows: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[r] = rms_norm(x[rows[r]]) * weight (rows None: every row, in place allowed)."""
@@ -1315,6 +1335,36 @@ def head_products(x: torch.Tensor, weight: torch.Tensor, out: Optional[torch.Ten
     return out
 
 
+def linear_columns(packed: torch.Tensor, column: int, weight: torch.Tensor, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    """A product whose input is the column range [column, column + K) of a wider contiguous matrix (the second half of a
+    low-rank projection whose first half is part of a packed one): [tokens, N] in ``out_dtype``."""
+    _cuda(packed, weight)
+    _contig(packed, weight)
+    tokens, (n, k) = packed.shape[0], weight.shape
+    out_dtype = out_dtype or packed.dtype
+    if packed.dtype != weight.dtype or column < 0 or column + k > packed.shape[1]:
+        raise KernelError("linear_columns: columns or dtypes do not fit")
+    x = packed[:, column:column + k]
+    if packed.dtype == torch.float32:
+        return cast(head_products(x.unsqueeze(0), weight.unsqueeze(0))[0], out_dtype)
+    flush_chain()
+    return torch.mm(x, weight.t(), out_dtype=out_dtype) if out_dtype != packed.dtype else torch.mm(x, weight.t())
+
+
+def block_products(u: torch.Tensor, gates: torch.Tensor) -> torch.Tensor:
+    """u [tokens, blocks * size] in equal parts, part b times gates[b] ([n, size]): float32 [blocks, tokens, n]."""
+    _cuda(u, gates)
+    _contig(u, gates)
+    blocks, _, size = gates.shape
+    if u.shape[1] != blocks * size or u.dtype != gates.dtype:
+        raise KernelError("block_products: the parts do not fit the matrices")
+    x = u.view(u.shape[0], blocks, size).transpose(0, 1)
+    if u.dtype == torch.float32:
+        return head_products(x, gates)
+    flush_chain()
+    return torch.bmm(x, gates.transpose(1, 2), out_dtype=torch.float32)
+
+
 def linear(x: torch.Tensor, weight: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
            lazy: bool = False) -> torch.Tensor:
     """x[M, K] . weight[N, K]^T, no bias.  ``lazy``: see ``few_row_linear``.
@@ -1422,28 +1472,34 @@ def _all_single(ctx) -> int:
 
 def causal_taps(x: torch.Tensor, weight: Optional[torch.Tensor], state: Optional[torch.Tensor], ctx,
                 out_dtype: torch.dtype, scale: Optional[torch.Tensor] = None, identity: bool = False,
-                channels: Optional[int] = None, update_state: bool = True) -> torch.Tensor:
+                channels: Optional[int] = None, update_state: bool = True, column: int = 0,
+                bias: Optional[torch.Tensor] = None, out_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """A short causal convolution over time on every channel, for a step's rows:
 
         y[t] = (u[t] if identity) + sum_j weight[:, j] * u[t - taps + 1 + j],   u[t] = x[t] * scale[t]
 
     with the inputs before a row's first token taken from ``state[slot]`` ([taps - 1, channels] float32, oldest
     first; zeros for a row that starts its sequence), and the rows' states brought up to date afterwards.
-    ``channels``: only the first so many columns of ``x`` pass through.  ``ctx`` gives the step's index arrays."""
-    _cuda(x, weight, state, scale)
-    _contig(x, weight, state, scale)
-    _f32(weight, state, scale)
-    c = int(channels or x.shape[1])
+    ``channels``: only so many columns of ``x``, from ``column`` on, pass through.  ``bias`` (float32, per channel):
+    u[t] = x[t] * scale[t] + bias (the zeros before the start stay zeros); ``out_bias``: y[t] + out_bias.  ``ctx`` gives
+    the step's index arrays."""
+    _cuda(x, weight, state, scale, bias, out_bias)
+    _contig(x, weight, state, scale, bias, out_bias)
+    _f32(weight, state, scale, bias, out_bias)
+    c = int(channels or x.shape[1] - column)
+    if column < 0 or column + c > x.shape[1] or any(b is not None and b.numel() != c for b in (bias, out_bias)):
+        raise KernelError("causal_taps: the columns or the biases do not fit")
     taps = 1 if weight is None else weight.shape[1]
     if weight is not None and weight.shape[0] != c:
         raise KernelError("the taps must be [channels, taps]")
     if taps > 1 and (state is None or tuple(state.shape[1:]) != (taps - 1, c)):
         raise KernelError("the state of a convolution must be [slots + 1, taps - 1, channels]")
     out = torch.empty((x.shape[0], c), dtype=out_dtype, device=x.device)
+    src = ctypes.c_void_p(x.data_ptr() + column * x.element_size())
     rc = _token_conv().b200_causal_taps(
-        _p(x), _code(x), x.shape[1], _p(scale), _p(weight), taps, c, _p(state), _p(ctx.row_of_token), _p(ctx.cu_q),
+        src, _code(x), x.shape[1], _p(scale), _p(weight), taps, c, _p(state), _p(ctx.row_of_token), _p(ctx.cu_q),
         _p(ctx.prefix_len), _p(ctx.state_slots), _p(out), _code(out), c, int(bool(identity)), x.shape[0],
-        ctx.num_rows, int(bool(update_state)), _all_single(ctx), _stream())
+        ctx.num_rows, int(bool(update_state)), _all_single(ctx), _p(bias), _p(out_bias), _stream())
     _ok(rc, "causal_taps", 2 if update_state and taps > 1 and not _all_single(ctx) else 1)
     return out
 
@@ -1566,6 +1622,185 @@ def retention(x: torch.Tensor, state: torch.Tensor, decay: torch.Tensor, inv_fre
     return o
 
 
+# --------------------------------------------------------------------------- a state that decays per key channel
+class _LinearStateShape(ctypes.Structure):
+    """Mirror of ``LinearStateShape`` in csrc/linear_state.cu (same order, native alignment)."""
+    _fields_ = [("heads", ctypes.c_int), ("kv_heads", ctypes.c_int), ("d", ctypes.c_int), ("dv", ctypes.c_int),
+                ("beta_column", ctypes.c_int), ("silu", ctypes.c_int), ("unit_eps", ctypes.c_float),
+                ("q_scale", ctypes.c_float), ("decay_kind", ctypes.c_int), ("inv_tau", ctypes.c_float),
+                ("decay_bias", ctypes.c_void_p), ("a_log", ctypes.c_void_p)]
+
+
+class _StateDecodeParams(ctypes.Structure):
+    """Mirror of ``StateDecodeParams`` in csrc/linear_state.cu."""
+    _fields_ = [("a2", ctypes.c_void_p), ("g2", ctypes.c_void_p), ("a_column", ctypes.c_int), ("a_rank", ctypes.c_int),
+                ("g_column", ctypes.c_int), ("g_rank", ctypes.c_int), ("gate_kind", ctypes.c_int),
+                ("norm_w", ctypes.c_void_p), ("eps", ctypes.c_float), ("own_conv", ctypes.c_int)]
+
+
+def _linear_state():
+    lib = load_cuda_library("linear_state.cu")
+    if not getattr(lib, "_checked", False):
+        if lib.b200_linear_state_shape_size() != ctypes.sizeof(_LinearStateShape) or \
+                lib.b200_state_decode_params_size() != ctypes.sizeof(_StateDecodeParams):
+            raise KernelError("the parameter blocks of linear_state.cu and their Python mirrors differ")
+        lib._checked = True
+    return lib
+
+
+class LinearStateForm:
+    """What a linear-attention layer with per-channel decays does between its projections (csrc/linear_state.cu):
+
+    ``decay`` "logistic": sigmoid(z + bias)^(1 / tau); "softplus": exp(-exp(a_log) softplus(z + bias)).
+    ``beta_column``: column of the packed row where one number a head begins whose sigmoid is the delta rule's step (None:
+    no delta rule).  ``silu``: on q, k, v behind the convolution.  ``unit_eps``: q and k become unit vectors (None: not).
+    """
+
+    def __init__(self, heads: int, kv_heads: int, head_dim: int, v_head_dim: int, q_scale: float = 1.0,
+                 decay: str = "logistic", tau: float = 1.0, decay_bias: Optional[torch.Tensor] = None,
+                 a_log: Optional[torch.Tensor] = None, beta_column: Optional[int] = None, silu: bool = False,
+                 unit_eps: Optional[float] = None):
+        if decay not in ("logistic", "softplus"):
+            raise KernelError(f"decay {decay!r} is refused: logistic or softplus")
+        _cuda(decay_bias, a_log)
+        _contig(decay_bias, a_log)
+        _f32(decay_bias, a_log)
+        if (decay_bias is not None and decay_bias.numel() != heads * head_dim) or (a_log is not None and a_log.numel() != heads) \
+                or (decay == "softplus") != (a_log is not None):
+            raise KernelError("the decay's bias [heads * head_dim] or rates [heads] do not fit")
+        self.heads, self.kv_heads, self.d, self.dv = heads, kv_heads, head_dim, v_head_dim
+        self.channels = 2 * kv_heads * head_dim + heads * v_head_dim
+        self.delta = beta_column is not None
+        self.keep = (decay_bias, a_log)
+        self.shape = _LinearStateShape(heads, kv_heads, head_dim, v_head_dim, -1 if beta_column is None else int(beta_column),
+                                       int(bool(silu)), float(unit_eps or 0.0), float(q_scale),
+                                       int(decay == "softplus"), 1.0 / float(tau),
+                                       decay_bias.data_ptr() if decay_bias is not None else None,
+                                       a_log.data_ptr() if a_log is not None else None)
+
+
+def _state_checks(form: LinearStateForm, x, conv, conv_state, state) -> int:
+    _cuda(x, conv, conv_state, state)
+    _contig(x, conv, conv_state, state)
+    _f32(conv, conv_state, state)
+    taps = 0 if conv is None else conv.shape[1]
+    if x.shape[1] < form.channels or (form.delta and form.shape.beta_column + form.heads > x.shape[1]) or \
+            tuple(state.shape[1:]) != (form.heads, form.d, form.dv) or \
+            (conv is not None and conv.shape[0] != form.channels) or \
+            (taps > 1 and (conv_state is None or tuple(conv_state.shape[1:]) != (taps - 1, form.channels))):
+        raise KernelError("linear state: sizes of the projection, the convolution or the states do not fit")
+    return taps
+
+
+def state_decode(form: LinearStateForm, x: torch.Tensor, conv: Optional[torch.Tensor], conv_state: Optional[torch.Tensor],
+                 state: torch.Tensor, ctx, a2: torch.Tensor, a_column: int, norm: torch.Tensor, eps: float,
+                 gate_column: int, g2: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """A step whose rows all bring one token: the layer between its packed projection ``x`` and its output projection in one
+    kernel (convolution, decay, recurrence, per-head norm, gate), [tokens, heads * v_head_dim] in x's dtype; the states are
+    brought up to date.  ``a2`` [heads * d, rank] meets x's columns from ``a_column`` on.  Gate: with ``g2``
+    sigmoid(g2 x[gate_column ..]), else silu of the columns from ``gate_column`` on.  None: the step has longer rows or the
+    sizes do not fit the kernel; the caller then runs the parts one by one."""
+    if not _all_single(ctx):
+        return None
+    taps = _state_checks(form, x, conv, conv_state, state)
+    _cuda(a2, g2, norm)
+    _contig(a2, g2, norm)
+    _f32(norm)
+    if a2.dtype != x.dtype or a2.shape[0] != form.heads * form.d or a_column + a2.shape[1] > x.shape[1] or \
+            norm.numel() != form.dv or (g2 is not None and (g2.dtype != x.dtype or g2.shape[0] != form.heads * form.dv)) or \
+            gate_column + (g2.shape[1] if g2 is not None else form.heads * form.dv) > x.shape[1]:
+        raise KernelError("state_decode: the low-rank products, the norm or the gate do not fit")
+    out = torch.empty((x.shape[0], form.heads * form.dv), dtype=x.dtype, device=x.device)
+    own = form.heads == form.kv_heads
+    params = _StateDecodeParams(a2.data_ptr(), g2.data_ptr() if g2 is not None else None, int(a_column), a2.shape[1],
+                                int(gate_column), g2.shape[1] if g2 is not None else 0, int(g2 is None), norm.data_ptr(),
+                                float(eps), int(own))
+    rc = _linear_state().b200_state_decode(
+        _p(x), _code(x), x.shape[1], _p(conv), taps, _p(conv_state), _p(ctx.row_of_token), _p(ctx.cu_q), _p(ctx.prefix_len),
+        _p(ctx.state_slots), ctypes.byref(form.shape), ctypes.byref(params), _p(out), _p(state), x.shape[0], _stream())
+    if rc == -2:
+        return None
+    _ok(rc, "state_decode")
+    if taps > 1 and not own:
+        taps_state_update(x, taps, form.channels, conv_state, ctx)
+    return out
+
+
+def state_recurrence(form: LinearStateForm, x: torch.Tensor, z: torch.Tensor, conv: Optional[torch.Tensor],
+                     conv_state: Optional[torch.Tensor], state: torch.Tensor, ctx) -> torch.Tensor:
+    """The recurrence over a step's rows of any length: o [tokens, heads * v_head_dim] float32, the states brought up to
+    date.  ``z`` (float32 [tokens, heads * d]): the decays' pre-activations without bias."""
+    taps = _state_checks(form, x, conv, conv_state, state)
+    _cuda(z)
+    _contig(z)
+    _f32(z)
+    tokens, dev = x.shape[0], x.device
+    if tuple(z.shape) != (tokens, form.heads * form.d):
+        raise KernelError("state_recurrence: one pre-activation for every head and key channel is needed")
+    qf = torch.empty((2, tokens, form.kv_heads * form.d), dtype=torch.float32, device=dev)
+    vf = torch.empty((tokens, form.heads * form.dv), dtype=torch.float32, device=dev)
+    gf = torch.empty((tokens, form.heads * form.d), dtype=torch.float32, device=dev)
+    beta = torch.empty((tokens, form.heads), dtype=torch.float32, device=dev) if form.delta else None
+    lib = _linear_state()
+    rc = lib.b200_state_prepare(
+        _p(x), _code(x), x.shape[1], _p(conv), taps, _p(conv_state), _p(ctx.row_of_token), _p(ctx.cu_q), _p(ctx.prefix_len),
+        _p(ctx.state_slots), ctypes.byref(form.shape), _p(z), _p(qf[0]), _p(qf[1]), _p(vf), _p(gf), _p(beta), tokens, _stream())
+    _ok(rc, "state_prepare")
+    if taps > 1:
+        taps_state_update(x, taps, form.channels, conv_state, ctx)
+    o = torch.empty((tokens, form.heads * form.dv), dtype=torch.float32, device=dev)
+    rc = lib.b200_state_scan(_p(qf[0]), _p(qf[1]), _p(vf), _p(gf), _p(beta), _p(o), _p(state), _p(ctx.cu_q),
+                             _p(ctx.prefix_len), _p(ctx.state_slots), ctx.num_rows, form.heads, form.kv_heads, form.d,
+                             form.dv, _stream())
+    _ok(rc, "state_scan")
+    return o
+
+
+# --------------------------------------------------------------------------- a gated linear recurrent unit
+LRU_FEW_ROWS = 16      # a step of at most this many one-token rows takes the kernel that does the block products itself
+
+
+def gated_lru(u: torch.Tensor, packed: torch.Tensor, y_column: int, gates: torch.Tensor, r_bias: torch.Tensor,
+              i_bias: torch.Tensor, lam: torch.Tensor, y_bias: torch.Tensor, state: torch.Tensor, ctx) -> torch.Tensor:
+    """out = S * gelu_tanh(y + y_bias), S <- a S + sqrt(1 - a^2) i u with log a = -8 r softplus(lam), r and i the sigmoids
+    of u's parts times ``gates`` [blocks, 2 size, size] (a part's r rows, then its i rows) plus biases.  u [tokens, width];
+    y lies in ``packed`` from ``y_column`` on; ``state`` [slots + 1, width] float32 is read (rows with a prefix) and
+    written.  The result has u's dtype."""
+    _cuda(u, packed, gates, r_bias, i_bias, lam, y_bias, state)
+    _contig(u, packed, gates, r_bias, i_bias, lam, y_bias, state)
+    _f32(r_bias, i_bias, lam, y_bias, state)
+    tokens, width = u.shape
+    blocks = gates.shape[0]
+    if gates.dtype != u.dtype or packed.dtype != u.dtype or tuple(gates.shape) != (blocks, 2 * (width // blocks), width // blocks) \
+            or any(t.numel() != width for t in (r_bias, i_bias, lam, y_bias)) or tuple(state.shape[1:]) != (width,) or \
+            packed.shape[0] != tokens or y_column + width > packed.shape[1]:
+        raise KernelError("gated_lru: sizes or dtypes do not fit")
+    lib = load_cuda_library("gated_lru.cu")
+    out = torch.empty_like(u)
+    y = ctypes.c_void_p(packed.data_ptr() + y_column * packed.element_size())
+    single = _all_single(ctx)
+    common = (_p(r_bias), _p(i_bias), _p(lam), _p(y_bias), width, blocks, _p(state))
+    if single and tokens <= LRU_FEW_ROWS:
+        rc = lib.b200_lru_few(_p(u), y, _code(u), packed.shape[1], _p(gates), *common, _p(ctx.prefix_len),
+                              _p(ctx.state_slots), _p(out), tokens, _stream())
+        _ok(rc, "lru_few")
+        return out
+    pre = block_products(u, gates)
+    if single:
+        rc = lib.b200_lru_rows(_p(u), y, _code(u), packed.shape[1], _p(pre), *common, _p(ctx.prefix_len),
+                               _p(ctx.state_slots), _p(out), tokens, _stream())
+        _ok(rc, "lru_rows")
+        return out
+    windows = -(-tokens // int(lib.b200_lru_window()))
+    win = torch.empty((3, windows, width), dtype=torch.float32, device=u.device)
+    start = torch.empty((ctx.num_rows, width), dtype=torch.float32, device=u.device)
+    rc = lib.b200_lru_scan(_p(u), y, _code(u), packed.shape[1], _p(pre), *common, _p(ctx.row_of_token), _p(ctx.cu_q),
+                           _p(ctx.prefix_len), _p(ctx.state_slots), _p(win[0]), _p(win[1]), _p(win[2]), _p(start), _p(out),
+                           tokens, ctx.num_rows, _stream())
+    _ok(rc, "lru_scan", 3)
+    return out
+
+
 # --------------------------------------------------------------------------- gates and PolyNorm
 def _gated():
     return load_cuda_library("gated.cu")
@@ -1586,18 +1821,22 @@ def poly_norm(z: torch.Tensor, coef: torch.Tensor, eps: float) -> torch.Tensor:
 
 
 def head_unit_norm_gate(o: torch.Tensor, packed: torch.Tensor, gate_column: int, heads: int, v_head_dim: int,
-                        eps: float) -> torch.Tensor:
-    """Every head's vector of ``o`` (float32) divided by its root mean square, times silu of the gate that lies
-    in ``packed`` from column ``gate_column`` on; the result has ``packed``'s dtype."""
-    _cuda(o, packed)
-    _contig(o, packed)
-    _f32(o)
+                        eps: float, weight: Optional[torch.Tensor] = None, gate: str = "silu") -> torch.Tensor:
+    """Every head's vector of ``o`` (float32) divided by its root mean square, times ``weight`` (float32
+    [v_head_dim], shared by the heads; None: none), times silu (``gate`` "sigmoid": sigmoid) of the gate that lies in
+    ``packed`` from column ``gate_column`` on; the result has ``packed``'s dtype."""
+    _cuda(o, packed, weight)
+    _contig(o, packed, weight)
+    _f32(o, weight)
+    if gate not in ("silu", "sigmoid") or (weight is not None and weight.numel() != v_head_dim):
+        raise KernelError("head_unit_norm_gate: an unknown gate, or a weight that is not a head's size")
     if packed.shape[1] < gate_column + heads * v_head_dim or o.shape[1] != heads * v_head_dim:
         raise KernelError("head_unit_norm_gate: the gate's columns do not fit")
     out = torch.empty((o.shape[0], o.shape[1]), dtype=packed.dtype, device=o.device)
-    gate = packed.view(-1)[gate_column:]
-    rc = _gated().b200_head_unit_norm_gate(_p(out), _p(o), ctypes.c_void_p(gate.data_ptr()), packed.shape[1],
-                                           o.shape[0], heads, v_head_dim, ctypes.c_float(eps), _code(packed), _stream())
+    at = ctypes.c_void_p(packed.data_ptr() + gate_column * packed.element_size())
+    rc = _gated().b200_head_unit_norm_gate(_p(out), _p(o), at, packed.shape[1], o.shape[0], heads, v_head_dim,
+                                           ctypes.c_float(eps), _p(weight), int(gate == "sigmoid"), _code(packed),
+                                           _stream())
     _ok(rc, "head_unit_norm_gate")
     return out
 
@@ -1832,7 +2071,8 @@ def columns_rms_norm(x: torch.Tensor, width: int, weight: torch.Tensor, eps: flo
 
 # --------------------------------------------------------------------------- experts chosen by a table or a router
 EXPERTS_TCGEN05_FROM_PAIRS = 512      # steps with this many (token, expert) pairs take the tcgen05 products
-GLU_KINDS = {"silu": 0, "clamped_swish": 1}
+GLU_KINDS = {"silu": 0, "clamped_swish": 1}          # of the experts' products
+GLU_COLUMN_KINDS = dict(GLU_KINDS, gelu_tanh=2)      # of glu_columns
 
 
 def _experts_buffers(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, top: int, what: str):
@@ -1920,11 +2160,12 @@ def expert_router(x: torch.Tensor, weight: torch.Tensor, top: int, groups: int =
 def routed_experts(x: torch.Tensor, choice: torch.Tensor, gains: torch.Tensor, gate_up: torch.Tensor,
                    down: torch.Tensor, glu: str = "silu", limit: float = 0.0, alpha: float = 1.0,
                    add: Optional[torch.Tensor] = None, tensor_memory: Optional[bool] = None,
-                   add_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   add_scale: Optional[torch.Tensor] = None, gains_on_input: bool = False) -> torch.Tensor:
     """out[t] = sum_k gains[t, k] down[e] glu(gate[e] x_t, up[e] x_t) (+ add_scale[t] * add[t]), e = choice[t, k]; float32
     [tokens, width].  ``glu``: "silu" (silu(g) u) or "clamped_swish" (g' sigmoid(alpha g') (u' + 1), g' = min(g, limit),
     u' = clamp(u, -limit, limit)).  ``add`` [tokens, width] (float32 or x's dtype) joins the sum in float: what every
-    token gets besides its experts, times ``add_scale`` (float32 [tokens]; None: 1).  Weights and the choice of product
+    token gets besides its experts, times ``add_scale`` (float32 [tokens]; None: 1).  ``gains_on_input``: the gains
+    multiply the experts' inputs instead, out[t] = sum_k down[e] glu(gate[e] (gains x_t), up[e] (gains x_t)).  Weights and the choice of product
     kernels as in ``table_experts``."""
     _cuda(x, choice, gains, gate_up, down, add, add_scale)
     _contig(x, choice, gains, gate_up, down, add, add_scale)
@@ -1943,28 +2184,30 @@ def routed_experts(x: torch.Tensor, choice: torch.Tensor, gains: torch.Tensor, g
         xs = torch.empty((pairs, width), dtype=x.dtype, device=x.device)
         rc = load_cuda_library("experts_tcgen05.cu").b200_routed_experts_tcgen05(
             _p(x), _p(choice), _p(gains), top, experts, _p(gate_up), _p(down), tokens, width, ff, GLU_KINDS[glu],
-            ctypes.c_float(limit), ctypes.c_float(alpha), _p(add), add_code, _p(add_scale), _p(xs), _p(h), _p(y),
-            _p(route), _p(out),
+            ctypes.c_float(limit), ctypes.c_float(alpha), _p(add), add_code, _p(add_scale), int(bool(gains_on_input)), _p(xs),
+            _p(h), _p(y), _p(route), _p(out),
             _p(error_word(x.device)), _stream())
         _ok(rc, "routed_experts_tcgen05", 5)
         return out
     rc = lib.b200_routed_experts(_p(x), _code(x), _p(choice), _p(gains), top, experts, _p(gate_up), _p(down), tokens,
                                  width, ff, GLU_KINDS[glu], ctypes.c_float(limit), ctypes.c_float(alpha), _p(add),
-                                 add_code, _p(add_scale), _p(h), _p(y), _p(route), _p(out), _p(error_word(x.device)),
+                                 add_code, _p(add_scale), int(bool(gains_on_input)), _p(h), _p(y), _p(route), _p(out),
+                                 _p(error_word(x.device)),
                                  _stream())
     _ok(rc, "routed_experts", 4)
     return out
 
 
 def glu_columns(gate_up: torch.Tensor, glu: str = "silu", limit: float = 0.0, alpha: float = 1.0) -> torch.Tensor:
-    """out = glu(gate_up[:, :F], gate_up[:, F:]) with the forms of ``routed_experts``; computed in float, rounded once."""
+    """out = glu(gate_up[:, :F], gate_up[:, F:]) with the forms of ``routed_experts`` or "gelu_tanh" (gelu_tanh(g) u);
+    computed in float, rounded once."""
     _cuda(gate_up)
     _contig(gate_up)
     tokens, width2 = gate_up.shape
-    if width2 % 2 or glu not in GLU_KINDS:
+    if width2 % 2 or glu not in GLU_COLUMN_KINDS:
         raise KernelError("glu_columns needs an even width and a known form")
     out = torch.empty((tokens, width2 // 2), dtype=gate_up.dtype, device=gate_up.device)
-    rc = _gated().b200_glu_columns(_p(out), _p(gate_up), tokens, width2 // 2, GLU_KINDS[glu], ctypes.c_float(limit),
+    rc = _gated().b200_glu_columns(_p(out), _p(gate_up), tokens, width2 // 2, GLU_COLUMN_KINDS[glu], ctypes.c_float(limit),
                                    ctypes.c_float(alpha), _code(gate_up), _stream())
     _ok(rc, "glu_columns")
     return out
@@ -2033,10 +2276,10 @@ def token_side_few(stream: torch.Tensor, x: torch.Tensor, gate: torch.Tensor, ta
 
 # --------------------------------------------------------------------------- a float stream with norms on the outputs
 def norm_add(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: float, bias: Optional[torch.Tensor] = None,
-             cast_to: Optional[torch.dtype] = None) -> Optional[torch.Tensor]:
+             cast_to: Optional[torch.dtype] = None, center: bool = False) -> Optional[torch.Tensor]:
     """x <- x + (y + bias) / sqrt(mean((y + bias)^2) + eps) * weight, in place on the float32 stream x [tokens, width];
     y float32 or bfloat16, weight and bias float32.  With ``cast_to`` the new x is also returned rounded once to that
-    dtype (float32: x itself is returned)."""
+    dtype (float32: x itself is returned).  ``center``: a layer norm, the row's mean is taken off y + bias first."""
     _cuda(x, y, weight, bias)
     _contig(x, y, weight, bias)
     _f32(x, weight, bias)
@@ -2047,7 +2290,7 @@ def norm_add(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: float,
     if cast_to is not None and cast_to != torch.float32:
         out = torch.empty((tokens, width), dtype=cast_to, device=x.device)
     rc = load_cuda_library("post_norm.cu").b200_norm_add(
-        _p(x), _p(y), _code(y), _p(bias), _p(weight), ctypes.c_float(eps), _p(out),
+        _p(x), _p(y), _code(y), _p(bias), _p(weight), ctypes.c_float(eps), int(bool(center)), _p(out),
         _code(out) if out is not None else F32, tokens, width, _stream())
     _ok(rc, "norm_add")
     if cast_to is None:
@@ -2055,10 +2298,42 @@ def norm_add(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: float,
     return out if out is not None else x
 
 
+class NormedPair:
+    """The mean of two branches, each RMS-normed with its own weights (float32), that has not been formed: a norm that
+    adds into the stream takes it in the same kernel."""
+
+    def __init__(self, a: torch.Tensor, b: torch.Tensor, a_weight: torch.Tensor, b_weight: torch.Tensor, eps: float):
+        self.a, self.b, self.a_weight, self.b_weight, self.eps = a, b, a_weight, b_weight, float(eps)
+        self.shape, self.dtype, self.device = a.shape, a.dtype, a.device
+
+
+def norm_add_pair(x: torch.Tensor, pair: NormedPair, weight: torch.Tensor, eps: float,
+                  cast_to: Optional[torch.dtype] = None, center: bool = False) -> Optional[torch.Tensor]:
+    """``norm_add`` of y = (R(a) + R(b)) / 2, R the pair's RMS norms, everything in float and in one kernel."""
+    a, b = pair.a, pair.b
+    _cuda(x, a, b, pair.a_weight, pair.b_weight, weight)
+    _contig(x, a, b, pair.a_weight, pair.b_weight, weight)
+    _f32(x, pair.a_weight, pair.b_weight, weight)
+    tokens, width = x.shape
+    if tuple(a.shape) != (tokens, width) or a.shape != b.shape or a.dtype != b.dtype or eps != pair.eps or \
+            any(w.numel() != width for w in (pair.a_weight, pair.b_weight, weight)):
+        raise KernelError("norm_add_pair: the branches, the weights or their eps do not fit")
+    out = None
+    if cast_to is not None and cast_to != torch.float32:
+        out = torch.empty((tokens, width), dtype=cast_to, device=x.device)
+    rc = load_cuda_library("post_norm.cu").b200_norm_add_pair(
+        _p(x), _p(a), _p(b), _code(a), _p(pair.a_weight), _p(pair.b_weight), _p(weight), ctypes.c_float(eps),
+        int(bool(center)), _p(out), _code(out) if out is not None else F32, tokens, width, _stream())
+    _ok(rc, "norm_add_pair")
+    if cast_to is None:
+        return None
+    return out if out is not None else x
+
+
 def norm_rows(x: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype: torch.dtype,
-              rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+              rows: Optional[torch.Tensor] = None, center: bool = False) -> torch.Tensor:
     """out[r] = x[rows[r]] / sqrt(mean(x[rows[r]]^2) + eps) * weight for the float32 stream x (every row without
-    ``rows``), rounded once to ``out_dtype``."""
+    ``rows``), rounded once to ``out_dtype``; ``center``: of x less its row's mean (a layer norm)."""
     _cuda(x, weight, rows)
     _contig(x, weight, rows)
     _f32(x, weight)
@@ -2069,6 +2344,6 @@ def norm_rows(x: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype: torc
     n = x.shape[0] if rows is None else rows.numel()
     out = torch.empty((n, width), dtype=out_dtype, device=x.device)
     rc = load_cuda_library("post_norm.cu").b200_norm_rows(_p(out), _code(out), _p(x), _p(rows), _p(weight),
-                                                          ctypes.c_float(eps), n, width, _stream())
+                                                          ctypes.c_float(eps), int(bool(center)), n, width, _stream())
     _ok(rc, "norm_rows")
     return out

@@ -302,7 +302,7 @@ class GroupedAttention(Part):
         not scaled); "zero": the number is 0 for every head and no parameter (one is added to the denominator);
       * ``own_kv`` False: the layer has no key and value projections (the packed matrix and bias hold q alone) and
         reads the cache of the run-list entry that its own entry names, with its own queries, masks and scale;
-      * ``gate``: the heads' outputs are multiplied by sigmoid(g) before the output projection.
+      * ``gate``: the heads' outputs are multiplied by sigmoid(g) before the output projection; "head": one gate a head.
     Softmax weights stay floats."""
     category = "mixer"
 
@@ -321,6 +321,7 @@ class GroupedAttention(Part):
         self.zero_sink = spec.get("sink") == "zero"
         self.sink = bool(spec.get("sink", False)) and not self.zero_sink
         self.gate = bool(spec.get("gate", False))
+        self.gate_per_head = spec.get("gate") == "head"
         self.out_bias = bool(spec.get("out_bias", False))
         self.norm_scope = str(spec.get("qk_norm_scope", "head"))
         self.own_kv = bool(spec.get("own_kv", True))
@@ -356,7 +357,7 @@ class GroupedAttention(Part):
         self.zero_sinks = torch.zeros(self.nh, dtype=torch.float32, device=env.device) if self.zero_sink else None
 
     def param_decls(self):
-        rows = self.qkv_channels + (self.nh * self.dv if self.gate else 0)
+        rows = self.qkv_channels + ((self.nh if self.gate_per_head else self.nh * self.dv) if self.gate else 0)
         decls = {"qkv_proj": ParamDecl((rows, self.hidden)), "o_proj": ParamDecl((self.hidden, self.nh * self.dv))}
         if self.bias:
             decls["qkv_bias"] = ParamDecl((self.qkv_channels,), "vector")
@@ -423,7 +424,18 @@ class GroupedAttention(Part):
             if self.out_bias and not self.bias_deferred:
                 ops.add_row_bias(y, p["o_bias"])
             return y
-        packed = ops.linear(x, p["qkv_proj"])
+        return self.forward_packed(ops.linear(x, p["qkv_proj"]), 0, ctx, cache)
+
+    def in_proj_name(self) -> str:
+        return "qkv_proj"
+
+    def forward_packed(self, packed, column, ctx, cache):
+        """From the packed projection on: its columns are the first of ``packed`` (``column`` 0), others may follow."""
+        if column != 0:
+            raise ValueError("this part's columns come first in a packed projection")
+        p = self.params
+        tokens = packed.shape[0]
+        rope = self.rope
         q = torch.empty((tokens, self.nh * self.d), dtype=packed.dtype, device=packed.device)
         slots = ctx.slots[cache.group] if cache.writes else None
         prepare = ops.joint_heads_prepare if self.norm_scope == "projection" else ops.heads_prepare
@@ -439,7 +451,7 @@ class GroupedAttention(Part):
         _masked_attention(self, q, out, ctx, cache, self.nh, self.nkv, self.d, self.dv,
                           self.zero_sinks if self.zero_sink else p.get("sink"))
         if self.gate:
-            ops.sigmoid_gate_mul(out, packed, self.qkv_channels)
+            ops.sigmoid_gate_mul(out, packed, self.qkv_channels, per=self.dv if self.gate_per_head else 1)
         y = ops.linear(out, p["o_proj"])
         if self.out_bias and not self.bias_deferred:
             ops.add_row_bias(y, p["o_bias"])

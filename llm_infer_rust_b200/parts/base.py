@@ -13,7 +13,9 @@ Categories and the interface each must have:
                       (``half_split_rope``: ``cos``, ``sin``, ``rot_dim``)
 ``mixer``             ``forward(x, ctx, cache) -> y``; ``cache_spec()`` (paged keys and
                       values it needs, or None); ``state_spec()`` (fixed-size
-                      per-request state it needs, or None)
+                      per-request state it needs, or None); optionally ``state_specs()`` (several, by name:
+                      ``mixer_state(cache, name)`` gives the tensor) and ``children()`` (parts inside the part, by
+                      name: their parameters' paths continue the part's own)
 ``feed_forward``      ``forward(x) -> y``
 ``token_conv``        ``forward(x, scale, ctx, state, out_dtype) -> y`` (a convolution over time whose last
                       inputs are per-request state); ``state_spec()``
@@ -23,12 +25,13 @@ returns the add + norm unrun (``ops.PendingNorm``); a mixer, feed-forward or hea
 ``takes_pending(tokens) -> bool`` and answers True is then given that object as ``x`` and runs it
 as the prologue of its first product.  Parts without these methods get plain tensors.
 ``block``             built from a ``LayerSpec``; ``forward(h, residual, ctx, cache) -> (h, residual)``
-``embedding``         ``forward(token_ids) -> h``
+``embedding``         ``forward(token_ids) -> h``; one that says ``needs_context`` (it keeps per-request state,
+                      ``state_specs()``): ``forward(token_ids, ctx, cache) -> h``
 ``head``              ``forward(x) -> float32 logits``
 """
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, replace
 from typing import Dict, Optional, Tuple
 
 import torch
@@ -66,6 +69,25 @@ class BuildEnv:
     dtype: torch.dtype                # the engine's activation dtype
     device: torch.device
     position_encodings: Dict[str, "Part"]
+
+
+def mixer_state(cache, name: str) -> Optional[torch.Tensor]:
+    """The named state of a mixer that has several (``state_specs()``), [slots + 1, *shape]; None if it has none of it."""
+    return cache.states.get("mixer." + name)
+
+
+def sub_cache(cache, child: str):
+    """What the mixer ``child`` inside a mixer sees of its cache: the same pages, and its own states."""
+    lead = f"mixer.{child}."
+    return replace(cache, states={"mixer." + name[len(lead):]: t for name, t in cache.states.items() if name.startswith(lead)})
+
+
+def padded_rows(weight: torch.Tensor, multiple: int = 8) -> torch.Tensor:
+    """A projection's matrix with zero rows behind it up to a multiple: its results' rows are whole 16-byte pieces."""
+    extra = -weight.shape[0] % multiple
+    if not extra:
+        return weight
+    return torch.cat([weight, weight.new_zeros((extra,) + tuple(weight.shape[1:]))])
 
 
 class Part:

@@ -4,7 +4,7 @@ from __future__ import annotations
 import torch
 
 from ..kernels import ops
-from .base import ParamDecl, Part
+from .base import ParamDecl, Part, StateSpec
 from .registry import register_part
 
 
@@ -26,6 +26,33 @@ class TokenEmbedding(Part):
 
     def forward(self, token_ids):
         return ops.embedding(token_ids, self.params["weight"], self.out_dtype, self.scale)
+
+
+class PairEmbedding(Part):
+    """h[t] = table[id_t] + pairs[row(id_(t-1), id_t)], row(a, b) = (a * ``mul_prev`` + b * ``mul_cur``) mod ``buckets``;
+    a sequence's first token takes the last row (``buckets``) of ``pairs``.  The sum is taken in float.  The previous
+    token is the request's state, so a step may begin anywhere in a sequence."""
+    category = "embedding"
+    needs_context = True
+
+    def __init__(self, spec, env):
+        super().__init__(spec, env)
+        self.vocab = int(spec["vocab_size"])
+        self.hidden = int(spec["hidden_size"])
+        self.buckets = int(spec["buckets"])
+        self.mul_prev = int(spec["mul_prev"])
+        self.mul_cur = int(spec["mul_cur"])
+        self.out_dtype = torch.float32 if spec.get("out_dtype") == "float32" else env.dtype
+
+    def param_decls(self):
+        return {"weight": ParamDecl((self.vocab, self.hidden)), "pairs": ParamDecl((self.buckets + 1, self.hidden))}
+
+    def state_specs(self):
+        return {"last_token": StateSpec((1,), torch.int32)}
+
+    def forward(self, token_ids, ctx, cache):
+        return ops.pair_embedding(token_ids, self.params["weight"], self.params["pairs"], cache.states["last_token"], ctx,
+                                  self.buckets, self.mul_prev, self.mul_cur, self.out_dtype)
 
 
 class LinearHead(Part):
@@ -63,4 +90,5 @@ class LinearHead(Part):
 
 
 register_part("embedding", "token_embedding", TokenEmbedding)
+register_part("embedding", "pair_embedding", PairEmbedding)
 register_part("head", "linear_head", LinearHead)

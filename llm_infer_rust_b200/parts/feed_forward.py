@@ -90,6 +90,29 @@ class DenseActFF(Part):
         return ops.linear(ops.activate(z, self.activation, in_place=True), self.params["down_proj"])
 
 
+class GatedActFF(Part):
+    """down(act(gate(x)) * up(x)), no bias, gate and up packed into one matrix (gate rows first); ``activation``:
+    gelu_tanh or silu, computed in float on the rounded projections and rounded once."""
+    category = "feed_forward"
+    _GLU = {"gelu_tanh": "gelu_tanh", "silu": "silu"}
+
+    def __init__(self, spec, env):
+        super().__init__(spec, env)
+        self.hidden = int(spec["hidden_size"])
+        self.inter = int(spec["intermediate_size"])
+        self.activation = str(spec["activation"])
+        if self.activation not in self._GLU:
+            raise ValueError(f"activation {self.activation!r} is refused: {sorted(self._GLU)}")
+
+    def param_decls(self):
+        return {"gate_up_proj": ParamDecl((2 * self.inter, self.hidden)),
+                "down_proj": ParamDecl((self.hidden, self.inter))}
+
+    def forward(self, x):
+        gate_up = ops.linear(x, self.params["gate_up_proj"])
+        return ops.linear(ops.glu_columns(gate_up, self._GLU[self.activation]), self.params["down_proj"])
+
+
 class TableExperts(Part):
     """A mixture of gated experts without a router: row ``token id`` of an integer ``table`` [vocab, top] names the
     token's experts (the entries of a row differ), and each counts 1 / top:
@@ -131,7 +154,8 @@ class RoutedExperts(Part):
         experts form ``groups`` equal groups of neighbours; a group's score is the sum of its ``group_members``
         largest c (1, the default: its largest); only experts of the ``keep_groups`` best groups can be chosen; the
         ``top`` largest c of those are, with weights s (divided by their sum if ``renormalize``) times ``weight_scale``
-        y = sum_k s_k down[e_k] glu(gate[e_k] x, up[e_k] x)  +  a shared_down glu(shared_gate x, shared_up x)
+        y = sum_k s_k down[e_k] glu(gate[e_k] x, up[e_k] x)   (``weights_on`` "input":
+            sum_k down[e_k] glu(gate[e_k] (s_k x), up[e_k] (s_k x)))  +  a shared_down glu(shared_gate x, shared_up x)
         a = 1, or with ``shared_gated`` sigmoid(shared_gate_row x): one number a token (``shared_gate_row`` [1, hidden])
 
     ``activation``: "swiglu" (silu(g) u) or "clamped_swish_glu" (g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit),
@@ -162,6 +186,9 @@ class RoutedExperts(Part):
         self.group_members = int(spec.get("group_members") or 1)
         self.weight_scale = float(spec.get("weight_scale", 1.0))
         self.shared_gated = bool(spec.get("shared_gated", False)) and self.shared_inter > 0
+        self.weights_on = str(spec.get("weights_on", "output"))
+        if self.weights_on not in ("output", "input"):
+            raise ValueError(f"weights_on {self.weights_on!r} is refused: output or input")
         if self.activation not in self._GLU:
             raise ValueError(f"activation {self.activation!r} is refused: {sorted(self._GLU)}")
         if self.experts % self.groups or not 1 <= self.keep <= self.groups or \
@@ -211,10 +238,12 @@ class RoutedExperts(Part):
         shared = self._shared_expert(x, glu) if self.shared_inter else None
         return ops.routed_experts(x, choice, gains, p["gate_up_proj"].view(self.experts, 2 * self.inter, self.hidden),
                                   p["down_proj"].view(self.experts, self.hidden, self.inter), glu, self.limit,
-                                  self.alpha, add=shared, add_scale=shared_scale)
+                                  self.alpha, add=shared, add_scale=shared_scale,
+                                  gains_on_input=self.weights_on == "input")
 
 
 register_part("feed_forward", "swiglu", SwiGLU)
+register_part("feed_forward", "gated_act", GatedActFF)
 register_part("feed_forward", "routed_experts", RoutedExperts)
 register_part("feed_forward", "dense_act", DenseActFF)
 register_part("feed_forward", "table_experts", TableExperts)

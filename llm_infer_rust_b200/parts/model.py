@@ -15,7 +15,7 @@ class DecoderModel:
     """Built from a ``ModelSpec`` alone; knows no architecture.
 
     Parameter paths: ``embedding.weight``, ``layers.<i>.<child>.<name>`` (children as
-    the block names them), ``final_norm.weight``, ``lm_head.weight``.
+    the block names them; ``layers.<i>.<child>.<inner>.<name>`` for a part inside a part), ``final_norm.weight``, ``lm_head.weight``.
     """
 
     def __init__(self, spec: ModelSpec, dtype: torch.dtype, device: torch.device):
@@ -45,8 +45,15 @@ class DecoderModel:
         owners = {"embedding": self.embedding, "final_norm": self.final_norm, "lm_head": self.lm_head}
         for i, block in enumerate(self.blocks):
             for child, part in block.children().items():
-                owners[f"layers.{i}.{child}"] = part
+                self._own(owners, f"layers.{i}.{child}", part)
         return owners
+
+    @staticmethod
+    def _own(owners: Dict[str, Part], path: str, part) -> None:
+        owners[path] = part
+        inner = getattr(part, "children", None)
+        for child, sub in (inner() if inner is not None else {}).items():
+            DecoderModel._own(owners, f"{path}.{child}", sub)
 
     def parameter_shapes(self) -> Dict[str, tuple]:
         return {f"{prefix}.{name}": decl.shape
@@ -77,9 +84,13 @@ class DecoderModel:
         return total
 
     # ------------------------------------------------------------------ one step
-    def forward(self, ctx, caches) -> torch.Tensor:
-        """Run the step's tokens; float32 logits [ctx.num_logits, vocab] at ``ctx.logit_rows``."""
-        h = self.embedding.forward(ctx.token_ids)
+    def forward(self, ctx, caches, embedding_cache=None) -> torch.Tensor:
+        """Run the step's tokens; float32 logits [ctx.num_logits, vocab] at ``ctx.logit_rows``.  ``embedding_cache``:
+        the states of an embedding that keeps some."""
+        if getattr(self.embedding, "needs_context", False):
+            h = self.embedding.forward(ctx.token_ids, ctx, embedding_cache)
+        else:
+            h = self.embedding.forward(ctx.token_ids)
         residual = None
         for e, entry in enumerate(self.run_list):
             h, residual = self.blocks[entry.layer].forward(h, residual, ctx, caches[e])

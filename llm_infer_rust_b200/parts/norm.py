@@ -143,11 +143,14 @@ class OutputRMSNorm(Part):
         ``add_into(stream, y)``:  stream <- stream + (y + bias) / sqrt(mean((y + bias)^2) + eps) * weight
 
     in float and in place, one kernel; it returns the new stream rounded once to the engine's dtype (the stream itself
-    in a float32 engine), which is what the next sublayer's first product reads.  ``bias`` (float32, per column) is an
+    in a float32 engine), which is what the next sublayer's first product reads.  ``y`` may be the mean of two
+    normed branches that has not been formed (``ops.NormedPair``).  ``bias`` (float32, per column) is an
     output projection's bias that its owner left to this kernel.  ``forward`` / ``forward_add`` are the plain norm of
     the stream itself at chosen rows (a model's last norm); ``forward_add`` is handed the rounded copy that the blocks
     pass on as ``residual`` and does not need it."""
     category = "norm"
+
+    center = False
 
     def __init__(self, spec, env):
         super().__init__(spec, env)
@@ -162,16 +165,28 @@ class OutputRMSNorm(Part):
         self.params[name] = tensor.to(torch.float32).contiguous()
 
     def add_into(self, stream, y, bias=None):
-        return ops.norm_add(stream, y, self.params["weight"], self.eps, bias=bias, cast_to=self.env.dtype)
+        if isinstance(y, ops.NormedPair):
+            if bias is not None:
+                raise ValueError("a mean of two branches has no bias")
+            return ops.norm_add_pair(stream, y, self.params["weight"], self.eps, cast_to=self.env.dtype, center=self.center)
+        return ops.norm_add(stream, y, self.params["weight"], self.eps, bias=bias, cast_to=self.env.dtype,
+                            center=self.center)
 
     def forward(self, x, out=None, rows=None):
-        return ops.norm_rows(x, self.params["weight"], self.eps, self.env.dtype, rows=rows)
+        return ops.norm_rows(x, self.params["weight"], self.eps, self.env.dtype, rows=rows, center=self.center)
 
     def forward_add(self, x, residual, out=None, rows=None, write_residual=True):
-        return ops.norm_rows(x, self.params["weight"], self.eps, self.env.dtype, rows=rows)
+        return ops.norm_rows(x, self.params["weight"], self.eps, self.env.dtype, rows=rows, center=self.center)
+
+
+class OutputLayerNorm(OutputRMSNorm):
+    """The same with a layer norm without bias: the row's mean is taken off first,
+    (y - mean) / sqrt(mean((y - mean)^2) + eps) * weight."""
+    center = True
 
 
 register_part("norm", "rms_norm", RMSNorm)
 register_part("norm", "output_rms_norm", OutputRMSNorm)
+register_part("norm", "output_layer_norm", OutputLayerNorm)
 register_part("norm", "stream_rms_norm", StreamRMSNorm)
 register_part("norm", "scalar_rms_norm", ScalarRMSNorm)

@@ -33,16 +33,14 @@ def main(argv: Optional[List[str]] = None) -> int:
     args = ap.parse_args(argv)
     os.makedirs(args.out, exist_ok=True)
 
-    from .config.registry import resolve_architecture
     from .engine import Engine, StepEntry
-    from .weights.loader import read_config_json
+    from .weights.loader import read_model_config
     page = args.page_size
     # Each live request's count is rounded up to a multiple of 64 (or of the page, if larger).
     unit = _round_up(64, page)
     pool_tokens = _round_up(max(args.max_tokens, unit), unit)
     # A request may be as long as the pool (and the model) allows.
-    raw = read_config_json(args.model)
-    arch = resolve_architecture(raw)
+    arch, raw = read_model_config(args.model)
     longest = min(arch.model_spec(arch.parse_config(raw)).max_positions, max(8192, pool_tokens))
     engine = Engine(args.model, dtype=args.dtype, max_running_req=args.max_requests, page_size=page,
                     max_total_tokens=pool_tokens, max_seq_len=longest, cuda_graph_bs=0,

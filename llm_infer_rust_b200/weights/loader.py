@@ -22,10 +22,11 @@ from __future__ import annotations
 import json
 import logging
 import os
-from typing import Dict, List, Optional, Sequence
+from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
 
+from ..config.registry import Architecture, resolve_architecture
 from .plan import WeightBinding
 from .safetensors_io import Checkpoint
 
@@ -69,6 +70,20 @@ def read_config_json(model_dir: str) -> dict:
         if "eos_token_id" in generation:
             config["eos_token_id"] = generation["eos_token_id"]
     return config
+
+
+def read_model_config(model_dir: str) -> Tuple[Architecture, dict]:
+    """The architecture of a model folder and its config.json, completed with the sizes that only the checkpoint's
+    tensor shapes tell (``Architecture.sizes_from_shapes``)."""
+    raw = read_config_json(model_dir)
+    arch = resolve_architecture(raw)
+    if arch.sizes_from_shapes is not None:
+        ckpt = Checkpoint(model_dir)
+        try:
+            raw = arch.sizes_from_shapes(raw, {name: tuple(ckpt.info(name)[1]) for name in ckpt.names()})
+        finally:
+            ckpt.close()
+    return arch, raw
 
 
 def kept_dtype(stored: torch.dtype, engine_dtype: torch.dtype, keep_float32: bool = False) -> torch.dtype:
