@@ -44,6 +44,10 @@ a stretched rotation and learned sinks; latent attention with queries through a 
 with a choice correction and groups ranked by their two best members; a gated shared expert), beside Torinex, the
 closest earlier design, and Qwen3.
 
+``--design sigudra`` does the same for Sigudra (states that decay per key channel with and without the delta rule,
+attention over a window beside a gated linear recurrent unit, experts weighted on their input, layer norms on the
+outputs), beside Kefetar, the closest earlier design, and Qwen3; its kernels also stand beside Torinex's.
+
 Peaks come from MEASURED_PEAKS.json beside this file when it is there.  Weights are random
 (drawn on the device), token ids are synthetic.  One GPU only.
 """
@@ -1094,10 +1098,226 @@ def lufizen_kernel_table(size, peak):
     return out
 
 
+# ----------------------------------------------------------------------------- --design sigudra
+SIGUDRA_EXPERTS = dict(experts=16, top=4)
+
+
+def sigudra_sizes(size):
+    """What the design has beside DESIGN_SIZES: the window, the recurrent unit's blocks, the low-rank projections' ranks
+    and the linear attention's key size (half a head, which with values of a whole head is its usual ratio)."""
+    z = DESIGN_SIZES[size]
+    return dict(window=1024, blocks=z["heads"], taps=4, rank=z["head_dim"], gla_rank=16, gla_dim=z["head_dim"] // 2, tau=16.0)
+
+
+def sigudra_config(size, layers):
+    """Layers in turn: the delta rule, attention over a window beside a gated recurrent unit as wide as the model, the
+    delta rule, gated linear attention; each second feed-forward is dense (gated, as wide as Qwen3's), the others 16 routed
+    experts, four a token, which together take a token through as many parameters."""
+    z, s = DESIGN_SIZES[size], sigudra_sizes(size)
+    d, I, r = z["head_dim"], z["inter"], SIGUDRA_EXPERTS
+
+    def layer(i):
+        mlp = {"kind": "dense", "ff": I} if i % 2 == 0 else {
+            "kind": "moe", "expert": {"ff": I // r["top"]}, "router": {"experts": r["experts"], "top": r["top"]}}
+        if i % 4 == 1:
+            return {"type": "parallel", "mlp": mlp, "mixer": {
+                "left": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": d, "vdim": d, "scale": d ** -0.5,
+                         "mask": {"size": s["window"]}},
+                "right": {"width": z["width"], "blocks": s["blocks"], "conv": s["taps"]}}}
+        if i % 4 == 3:
+            return {"type": "gla", "mlp": mlp, "mixer": {"heads": z["heads"], "dim": s["gla_dim"], "vdim": d, "tau": s["tau"],
+                                                         "decay_rank": s["gla_rank"]}}
+        return {"type": "channel_delta", "mlp": mlp, "mixer": {
+            "heads": z["heads"], "kv_heads": z["heads"], "dim": d, "vdim": d, "conv": s["taps"], "decay_rank": s["rank"],
+            "gate_rank": s["rank"]}}
+
+    return {"architecture": "Sigudra", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5},
+            "embedding": {"bigram": {"buckets": 4099, "mul_prev": 8191, "mul_cur": 31}},
+            "layers": [layer(i) for i in range(layers)]}
+
+
+def sigudra_kernel_table(size, peak):
+    """Every kernel of Sigudra alone, beside the like kernel of the closest designs (Kefetar's retention, convolution and
+    per-head norm, Torinex's norms, prepare kernel and experts, Qwen3's activation and embedding), at one layer's sizes: a
+    prompt portion of 2,048 tokens and a decode step of 8 rows at 2,048 tokens.  ``frac`` as in ``kernel_table``; of the
+    recurrences' FLOPs: 4 d dv a token and head for retention and gated linear attention (the read-out and the update, two
+    each), 8 d dv for the delta rule with its decay per channel (decay, read of the past, update, read-out)."""
+    import types
+    import torch
+    from llm_infer_rust_b200.kernels import ops
+    from llm_infer_rust_b200.parts.attention import decode_splits
+    z, s, r = DESIGN_SIZES[size], sigudra_sizes(size), SIGUDRA_EXPERTS
+    W, nh, nkv, d, I = z["width"], z["heads"], z["kv_heads"], z["head_dim"], z["inter"]
+    E, top, ffe, window = r["experts"], r["top"], I // r["top"], s["window"]
+    dev, bf = torch.device("cuda"), torch.bfloat16
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    page, ctx_len, rows_dec = 16, 2048, 8
+    out = {}
+
+    def put(name, us, nbytes=None, flops=None, of="bf16"):
+        rec = {"us": round(us, 2)}
+        if nbytes is not None:
+            rec["gb_s"] = round(nbytes / us / 1e3, 1)
+            rec["frac"] = round(nbytes / us / 1e3 / peak["hbm_gbs"], 3)
+        if flops is not None:
+            rec["tflops"] = round(flops / us / 1e6, 2)
+            rec["frac"] = round(flops / us / 1e6 / {"bf16": peak["bf16_tflops"], "fp32": peak["fp32_tflops"]}[of], 3)
+            rec["of"] = of
+        out[name] = rec
+
+    def step(rows):
+        cu, row_of, pos = [0], [], []
+        for i, (prefix, n) in enumerate(rows):
+            cu.append(cu[-1] + n)
+            row_of += [i] * n
+            pos += list(range(prefix, prefix + n))
+        R = len(rows)
+        width = -(-max(p + n for p, n in rows) // page)
+        table = torch.arange(1, R * width + 1, dtype=torch.int32, device=dev).view(R, width).contiguous()
+        slots = [int(table[i, (p + j) // page]) * page + (p + j) % page for i, (p, n) in enumerate(rows) for j in range(n)]
+        return types.SimpleNamespace(
+            num_rows=R, row_of_token=i32(row_of), cu_q=i32(cu), positions=i32(pos), prefix_len=i32([p for p, _ in rows]),
+            kv_len=i32([p + n for p, n in rows]), state_slots=i32(list(range(1, R + 1))), slots=i32(slots), table=table,
+            rows=i32(list(range(R))), tokens=cu[-1], pages=R * width + 1, max_q_len=max(n for _, n in rows),
+            num_prefill=sum(n > 1 for _, n in rows))
+
+    for phase, c in (("prefill", step([(0, ctx_len)])), ("decode", step([(ctx_len - 1, 1)] * rows_dec))):
+        T = c.tokens
+        rnd = lambda *shape, f=1.0: (torch.randn(*shape, device=dev) * f).to(bf)
+        few = 3 if phase == "prefill" else 7
+        # --- embedding and norms
+        ids, tbl, pairs = torch.randint(0, 4096, (T,), device=dev, dtype=torch.int32), rnd(32768, W), rnd(4100, W)
+        last = torch.zeros(rows_dec + 1, 1, dtype=torch.int32, device=dev)
+        put(f"{phase}.sigudra.pair_embedding", timed_alone(
+            lambda: ops.pair_embedding(ids, tbl, pairs, last, c, 4099, 8191, 31, torch.float32), flush), T * W * 8)
+        put(f"{phase}.torinex.embedding", timed_alone(lambda: ops.embedding(ids, tbl, torch.float32), flush), T * W * 6)
+        stream, y, y2, wn = torch.randn(T, W, device=dev), rnd(T, W), rnd(T, W), torch.ones(W, device=dev)
+        pair = ops.NormedPair(y, y2, wn, wn, 1e-5)
+        put(f"{phase}.sigudra.layer_norm_add", timed_alone(
+            lambda: ops.norm_add(stream, y, wn, 1e-5, cast_to=bf, center=True), flush), T * W * 12)
+        put(f"{phase}.sigudra.layer_norm_add_pair", timed_alone(
+            lambda: ops.norm_add_pair(stream, pair, wn, 1e-5, cast_to=bf, center=True), flush), T * W * 14)
+        put(f"{phase}.torinex.norm_add", timed_alone(lambda: ops.norm_add(stream, y, wn, 1e-5, cast_to=bf), flush), T * W * 12)
+        # --- states that decay per channel beside retention
+        rp = rnd(T, nh * 4 * d, f=0.3)
+        rstate = torch.zeros(rows_dec + 1, nh, d, d, device=dev)
+        decay = torch.full((nh,), 0.99, device=dev)
+        us = timed_alone(lambda: ops.retention(rp, rstate, decay, None, 0, d ** -0.5, c, nh, d, d), flush, repeats=few)
+        if phase == "prefill":
+            put("prefill.kefetar.retention", us, flops=4.0 * T * nh * d * d, of="fp32")
+        else:
+            put("decode.kefetar.retention", us, rows_dec * nh * d * d * 8)
+        ro, hw = torch.randn(T, nh * d, device=dev), torch.ones(d, device=dev)
+        put(f"{phase}.kefetar.head_unit_norm_gate", timed_alone(
+            lambda: ops.head_unit_norm_gate(ro, rp, nh * 3 * d, nh, d, 1e-5), flush), T * nh * d * 8)
+        for name, dk, rank, low in (("delta", d, s["rank"], True), ("gla", s["gla_dim"], s["gla_rank"], False)):
+            channels = nh * (2 * dk + d)
+            a_col = channels + (0 if low else nh * d)
+            g_col = a_col + rank if low else channels
+            beta = g_col + rank if low else None
+            packed = rnd(T, a_col + rank + (rank + nh if low else 0), f=0.5)
+            packed = torch.nn.functional.pad(packed, (0, -packed.shape[1] % 8)).contiguous()
+            bias = torch.full((nh * dk,), -3.0 if low else 3.0, device=dev)
+            form = ops.LinearStateForm(nh, nh, dk, d, q_scale=dk ** -0.5, decay="softplus" if low else "logistic", tau=s["tau"],
+                                       decay_bias=bias, a_log=torch.zeros(nh, device=dev) if low else None, beta_column=beta,
+                                       silu=low, unit_eps=1e-6 if low else None)
+            conv = torch.randn(channels, s["taps"], device=dev) * 0.3 if low else None
+            cstate = torch.zeros(rows_dec + 1, s["taps"] - 1, channels, device=dev) if low else None
+            state = torch.zeros(rows_dec + 1, nh, dk, d, device=dev)
+            a2, g2 = rnd(nh * dk, rank, f=rank ** -0.5), rnd(nh * d, rank, f=rank ** -0.5) if low else None
+            if phase == "prefill":
+                zf = ops.linear_columns(packed, a_col, a2, out_dtype=torch.float32)
+                us = timed_alone(lambda: ops.state_recurrence(form, packed, zf, conv, cstate, state, c), flush, repeats=few)
+                put(f"prefill.sigudra.{name}_recurrence", us, flops=(8.0 if low else 4.0) * T * nh * dk * d, of="fp32")
+                o = torch.randn(T, nh * d, device=dev)
+                gz = ops.linear_columns(packed, g_col, g2) if low else packed
+                put(f"prefill.sigudra.{name}_head_norm_gate", timed_alone(
+                    lambda: ops.head_unit_norm_gate(o, gz, 0 if low else g_col, nh, d, 1e-5, weight=hw,
+                                                    gate="sigmoid" if low else "silu"), flush), T * nh * d * 8)
+                put(f"prefill.sigudra.{name}_low_rank", timed_alone(
+                    lambda: ops.linear_columns(packed, a_col, a2, out_dtype=torch.float32), flush), T * (nh * dk * 4 + rank * 2))
+            else:
+                put(f"decode.sigudra.{name}_state_decode", timed_alone(
+                    lambda: ops.state_decode(form, packed, conv, cstate, state, c, a2, a_col, hw, 1e-5, g_col, g2), flush),
+                    rows_dec * nh * dk * d * 8)
+        # --- the gated recurrent unit and its convolution beside Kefetar's convolution
+        px, cw = rnd(T, 2 * W), torch.randn(W, s["taps"], device=dev) * 0.3
+        cst, wb = torch.zeros(rows_dec + 1, s["taps"] - 1, W, device=dev), torch.zeros(W, device=dev)
+        put(f"{phase}.sigudra.convolution", timed_alone(
+            lambda: ops.causal_taps(px, cw, cst, c, bf, channels=W, column=W, bias=wb, out_bias=wb), flush), T * W * 4)
+        put(f"{phase}.kefetar.causal_taps", timed_alone(
+            lambda: ops.causal_taps(y, cw, cst, c, bf, identity=True), flush), T * W * 4)
+        B = s["blocks"]
+        gates = rnd(B, 2 * (W // B), W // B, f=(W // B) ** -0.5)
+        lst, lam = torch.zeros(rows_dec + 1, W, device=dev), torch.full((W,), -4.0, device=dev)
+        us = timed_alone(lambda: ops.gated_lru(y, px, 0, gates, wb, wb, lam, wb, lst, c), flush)
+        put(f"{phase}.sigudra.gated_lru", us, T * W * 6 + gates.numel() * 2 + (rows_dec * W * 8 if phase == "decode" else 0))
+        if phase == "prefill":
+            put("prefill.sigudra.gated_lru_block_products", timed_alone(lambda: ops.block_products(y, gates), flush),
+                T * W * 10 + gates.numel() * 2)
+        # --- attention over a window: the prepare kernel without a rotation, scores, one gate a head
+        cq = (nh + 2 * nkv) * d
+        qkvg = rnd(T, cq + nh, f=0.5)
+        k_cache, v_cache = (torch.zeros(c.pages, nkv, page, d, dtype=bf, device=dev).normal_() for _ in range(2))
+        q, o = torch.empty(T, nh * d, dtype=bf, device=dev), torch.empty(T, nh * d, dtype=bf, device=dev)
+        qw, kw = torch.ones(nh * d, device=dev), torch.ones(nkv * d, device=dev)
+        inv_freq = torch.pow(torch.tensor(1e6), -torch.arange(0, d, 2) / d).to(dev)
+        prepare = lambda **more: ops.joint_heads_prepare(qkvg, q, k_cache, v_cache, c.positions, c.slots, nh, nkv, d, d,
+                                                         q_weight=qw, k_weight=kw, eps=1e-5, **more)
+        put(f"{phase}.sigudra.joint_heads_prepare", timed_alone(prepare, flush), T * cq * 4)
+        put(f"{phase}.torinex.joint_heads_prepare", timed_alone(
+            lambda: prepare(inv_freq=inv_freq, rot_dims=d, interleaved=True), flush), T * cq * 4)
+        put(f"{phase}.sigudra.gate_per_head", timed_alone(lambda: ops.sigmoid_gate_mul(o, qkvg, cq, per=d), flush), T * nh * d * 4)
+        put(f"{phase}.kefetar.sigmoid_gate_mul", timed_alone(lambda: ops.sigmoid_gate_mul(o, rp, 0), flush), T * nh * d * 6)
+        for name, kwargs in (("sigudra.attention_window", dict(window=window)), ("torinex.attention_blocks", dict(chunk=window))):
+            win, more = kwargs.get("window"), dict(v_head_dim=d, precise_weights=True, chunk=kwargs.get("chunk"))
+            if phase == "prefill":
+                seen = sum(min(p + 1, window) if win else p % window + 1 for p in range(T))
+                put(f"prefill.{name}", timed_alone(lambda: ops.prefill_attention(
+                    q, k_cache, v_cache, o, c.table, c.cu_q, c.kv_len, c.prefix_len, c.rows, 1, T, nh, nkv, d, page, win,
+                    d ** -0.5, **more), flush, repeats=few), flops=4.0 * nh * d * seen)
+            else:
+                splits = decode_splits(ops.decode_ctas_per_split(bf, rows_dec, nh, nkv, d, page, True), window, 148)
+                scratch = torch.empty(max(ops.decode_scratch_floats(rows_dec, nh, d, splits), 1), device=dev)
+                put(f"decode.{name}", timed_alone(lambda: ops.decode_attention(
+                    q, k_cache, v_cache, o, scratch, c.table, c.cu_q, c.kv_len, c.rows, rows_dec, nh, nkv, d, page, win,
+                    d ** -0.5, splits, **more), flush), rows_dec * window * nkv * d * 4)
+        # --- feed-forwards
+        xe = rnd(T, W)
+        wgu, wdn = rnd(2 * I, W, f=W ** -0.5), rnd(W, I, f=I ** -0.5)
+        from llm_infer_rust_b200.config.spec import PartSpec
+        from llm_infer_rust_b200.parts import BuildEnv, build_part
+        for name, kind, extra in (("sigudra.gelu_feed_forward", "gated_act", {"activation": "gelu_tanh"}), ("qwen3.feed_forward", "swiglu", {})):
+            ff = build_part("feed_forward", PartSpec(kind, dict(hidden_size=W, intermediate_size=I, **extra)), BuildEnv(bf, dev, {}))
+            ff.bind("gate_up_proj", wgu)
+            ff.bind("down_proj", wdn)
+            us = timed_alone(lambda: (ff.forward(xe), ops.flush_chain()), flush)
+            if phase == "prefill":
+                put(f"prefill.{name}", us, flops=6.0 * T * W * I)
+            else:
+                put(f"decode.{name}", us, 3 * W * I * 2)
+        wr = rnd(E, W, f=W ** -0.5)
+        for name, scores in (("sigudra.expert_router", "sigmoid"), ("torinex.expert_router", "softmax")):
+            put(f"{phase}.{name}", timed_alone(lambda: ops.expert_router(xe, wr, top, scores=scores), flush),
+                T * W * 2 + E * W * 2 + T * top * 8)
+        choice, gains = ops.expert_router(xe, wr, top, scores="sigmoid")
+        gate_up, down = rnd(E, 2 * ffe, W, f=W ** -0.5), rnd(E, W, ffe, f=ffe ** -0.5)
+        used = int(torch.unique(choice).numel())
+        for name, on_input in (("sigudra.routed_experts", True), ("torinex.routed_experts", False)):
+            us = timed_alone(lambda: ops.routed_experts(xe, choice, gains, gate_up, down, "silu", gains_on_input=on_input), flush)
+            if phase == "prefill":
+                put(f"prefill.{name}", us, flops=6.0 * T * top * W * ffe)
+            else:
+                put(f"decode.{name}", us, used * 3 * W * ffe * 2)
+    return out
+
+
 DESIGNS = {"kefetar": (kefetar_config, kernel_table), "mukenex": (mukenex_config, mukenex_kernel_table),
-           "torinex": (torinex_config, torinex_kernel_table), "lufizen": (lufizen_config, lufizen_kernel_table)}
+           "torinex": (torinex_config, torinex_kernel_table), "lufizen": (lufizen_config, lufizen_kernel_table),
+           "sigudra": (sigudra_config, sigudra_kernel_table)}
 # The closest earlier design, which stands beside the new one and Qwen3 at equal sizes.
-BESIDE = {"lufizen": ("torinex", torinex_config)}
+BESIDE = {"lufizen": ("torinex", torinex_config), "sigudra": ("kefetar", kefetar_config)}
 
 
 def design_main(args) -> int:
@@ -1153,9 +1373,9 @@ def main() -> int:
                     help="other shapes measured into `points` (decode at batch 1 / 8 / 64, prefill), comma separated")
     ap.add_argument("--only", choices=["decode", "prefill"], default=None,
                     help="run one phase alone and print a short line (for profiling)")
-    ap.add_argument("--design", choices=["qwen3", "kefetar", "mukenex", "torinex", "lufizen"], default="qwen3",
-                    help="kefetar, mukenex, torinex, lufizen: that design beside Qwen3 at equal sizes, and its kernels alone (another line)")
-    ap.add_argument("--design-sizes", default="1k,4k", help="layer sizes of --design kefetar / mukenex / torinex / lufizen, comma separated")
+    ap.add_argument("--design", choices=["qwen3", "kefetar", "mukenex", "torinex", "lufizen", "sigudra"], default="qwen3",
+                    help="kefetar, mukenex, torinex, lufizen, sigudra: that design beside Qwen3 at equal sizes, and its kernels alone (another line)")
+    ap.add_argument("--design-sizes", default="1k,4k", help="layer sizes of the other designs, comma separated")
     ap.add_argument("--no-kernels", action="store_true", help="--design ... without the table of single kernels")
     args = ap.parse_args()
     if args.design in DESIGNS and args.impl == "ours":

@@ -41,6 +41,16 @@ __device__ __forceinline__ float warp_max(float v) {
   return v;
 }
 
+// What joins a gate projection to its up projection in the products that do it as their epilogue: silu(g), or
+// gelu_tanh(g) in a build with GLU_GELU_TANH.
+__device__ __forceinline__ float glu_gate(float g) {
+#ifdef GLU_GELU_TANH
+  return 0.5f * g * (1.0f + tanhf(0.79788456080286535588f * (g + 0.044715f * g * g * g)));
+#else
+  return g / (1.0f + expf(-g));
+#endif
+}
+
 // Sum over a block of up to 1024 threads; every thread gets the result.
 // `scratch` holds 33 floats of shared memory.  The order of the additions is
 // fixed by the thread layout, so a row's sum does not depend on other rows.
@@ -107,6 +117,9 @@ __device__ __forceinline__ void cp_async16(void* smem, const void* gmem, bool va
   uint32_t dst = static_cast<uint32_t>(__cvta_generic_to_shared(smem));
   int bytes = valid ? 16 : 0;
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(dst), "l"(gmem), "r"(bytes));
+}
+__device__ __forceinline__ void cp_async4(void* smem, const void* gmem) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(static_cast<uint32_t>(__cvta_generic_to_shared(smem))), "l"(gmem));
 }
 __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;\n" ::); }
 template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N)); }

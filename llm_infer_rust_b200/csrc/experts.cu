@@ -419,7 +419,8 @@ expert_combine_kernel(float* __restrict__ out, const float* __restrict__ Y, cons
 // ------------------------------------------------------------------ the router
 // z[t][e] = W[e] . x[t] in float (FFMA, whatever the dtype of x and W), scores s = softmax over all experts (or a
 // sigmoid of each).  The CHOICE looks at c = s + correction (one float an expert; null: c = s): experts in `groups`
-// equal groups of neighbours, a group's score the sum of its `group_members` largest c (1: its largest), only experts
+// equal groups of neighbours (sigmoids without a correction are ranked by their logits, which are not rounded to 1), a
+// group's score the sum of its `group_members` largest c (1: its largest), only experts
 // of the `keep` best groups can be chosen (the others are shut out whatever their c, which may be negative), the `top`
 // largest c of them are.  The WEIGHTS are the chosen experts' s (without the correction), divided by their sum if
 // `renormalize`, times `gain_scale`.  Ties go to the lower index.
@@ -547,8 +548,14 @@ expert_router_kernel(const TX* __restrict__ x, const TW* __restrict__ W, int tok
     for (int w = 0; w < ROUTER_WARPS; ++w) g += gate_part[warp][w];
     gate_out[t] = 1.0f / (1.0f + expf(-g));
   }
+  // Where the choice only ranks sigmoids it ranks their logits: a sigmoid in float is exactly 1 from about 17 on.
+  const bool by_logit = sigmoid_scores && correction == nullptr && (groups <= 1 || group_members <= 1);
   if (sigmoid_scores) {
-    for (int e = lane; e < experts; e += 32) s[e] = 1.0f / (1.0f + expf(-s[e]));
+    for (int e = lane; e < experts; e += 32) {
+      const float logit = s[e];
+      if (by_logit) c[e] = logit;
+      s[e] = 1.0f / (1.0f + expf(-logit));
+    }
   } else {
     float m = -INFINITY;
     for (int e = lane; e < experts; e += 32) m = fmaxf(m, s[e]);
@@ -560,7 +567,7 @@ expert_router_kernel(const TX* __restrict__ x, const TW* __restrict__ W, int tok
   }
   for (int e = lane; e < experts; e += 32) {
     can[e] = groups <= 1 ? 1 : 0;
-    c[e] = correction != nullptr ? s[e] + correction[e] : s[e];
+    if (!by_logit) c[e] = correction != nullptr ? s[e] + correction[e] : s[e];
   }
   __syncwarp();
   const int per = experts / max(groups, 1);

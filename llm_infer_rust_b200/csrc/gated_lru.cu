@@ -8,9 +8,10 @@
 //
 //   lru_few      a step of few rows of one token each: the block products, the recurrence and the gate in one kernel
 //   lru_rows     rows of one token each, the block products `pre` given
-//   lru_scan     rows of any length, `pre` given, in windows of 32 tokens: (1) every window's own contribution, (2) the
-//                windows of a row folded in order, (3) the recurrence of every window again from the state it starts with.
-//                Inside a window the recurrence runs token by token.
+//   lru_scan     rows of any length, `pre` given, in windows of 32 tokens: (1) a and the added term of every token, left in
+//                place of their pre-activations, and every window's own contribution, (2) the windows of a row folded in
+//                order, (3) the recurrence of every window from the state it starts with.  Inside a window the recurrence
+//                runs token by token.
 // pre [blocks, tokens, 2 * size] float: R_b u_b, then I_b u_b.  state [slots + 1, width]; a row whose prefix_len is 0
 // starts from zeros; slot 0 takes padding rows.
 #include "common.cuh"
@@ -134,25 +135,42 @@ lru_rows_kernel(const T* __restrict__ u, const T* __restrict__ y, const float* _
       from_f32<T>(S * gelu_tanh_of(to_f32<T>(y[static_cast<size_t>(m) * p.y_stride + c]) + p.y_bias[c]));
 }
 
-// (1) grid (windows, channel tiles of 128).  The segment of the window's LAST row: the product of its a and the state it
-// leaves when it starts from zero.  (The rows that end inside the window leave nothing to a later window.)
+// (1) grid (windows, channel tiles of 128).  Besides every token's terms, the segment of the window's LAST row: the product
+// of its a and the state it leaves when it starts from zero.  (Rows that end inside the window leave nothing to a later
+// one.)  Four tokens' loads are in flight at a time.
 template <typename T>
 __global__ void __launch_bounds__(128)
-lru_window_kernel(const T* __restrict__ u, const float* __restrict__ pre, LruParams p, const int* __restrict__ row_of_token,
+lru_window_kernel(const T* __restrict__ u, float* __restrict__ pre, LruParams p, const int* __restrict__ row_of_token,
                   const int* __restrict__ cu_q, float* __restrict__ win_a, float* __restrict__ win_s, int tokens) {
   const int w = blockIdx.x, c = blockIdx.y * 128 + threadIdx.x;
   if (c >= p.width) return;
-  const int last = min((w + 1) * LRU_WINDOW, tokens) - 1;
-  const int begin = max(w * LRU_WINDOW, cu_q[row_of_token[last]]);
-  const float rate = 8.0f * softplus_of(p.lam[c]);
+  const int t0 = w * LRU_WINDOW, end = min(t0 + LRU_WINDOW, tokens);
+  const int begin = cu_q[row_of_token[end - 1]];
+  const float rate = 8.0f * softplus_of(p.lam[c]), rb = p.r_bias[c], ib = p.i_bias[c];
+  const int b = c / p.size, j = c - b * p.size;
+  float* at = pre + static_cast<size_t>(b) * tokens * 2 * p.size + j;
   float A = 1.0f, S = 0.0f;
-#pragma unroll 4
-  for (int t = begin; t <= last; ++t) {
-    float r, i, a, add;
-    pre_of(pre, p, tokens, t, c, r, i);
-    lru_terms(r, i, to_f32<T>(u[static_cast<size_t>(t) * p.width + c]), rate, a, add);
-    A *= a;
-    S = fmaf(a, S, add);
+  for (int t = t0; t < end; t += 4) {
+    float r[4], i[4], x[4];
+#pragma unroll
+    for (int m = 0; m < 4; ++m) {
+      const int s = min(t + m, end - 1);
+      r[m] = at[static_cast<size_t>(s) * 2 * p.size];
+      i[m] = at[static_cast<size_t>(s) * 2 * p.size + p.size];
+      x[m] = to_f32<T>(u[static_cast<size_t>(s) * p.width + c]);
+    }
+#pragma unroll
+    for (int m = 0; m < 4; ++m) {
+      if (t + m >= end) break;
+      float a, add;
+      lru_terms(r[m] + rb, i[m] + ib, x[m], rate, a, add);
+      at[static_cast<size_t>(t + m) * 2 * p.size] = a;
+      at[static_cast<size_t>(t + m) * 2 * p.size + p.size] = add;
+      if (t + m >= begin) {
+        A *= a;
+        S = fmaf(a, S, add);
+      }
+    }
   }
   win_a[static_cast<size_t>(w) * p.width + c] = A;
   win_s[static_cast<size_t>(w) * p.width + c] = S;
@@ -182,13 +200,14 @@ lru_fold_kernel(LruParams p, const float* __restrict__ state, const int* __restr
 // (3) grid (windows, channel tiles of 128)
 template <typename T>
 __global__ void __launch_bounds__(128)
-lru_output_kernel(const T* __restrict__ u, const T* __restrict__ y, const float* __restrict__ pre, LruParams p,
-                  const int* __restrict__ row_of_token, const int* __restrict__ cu_q, const int* __restrict__ state_slots,
-                  const float* __restrict__ carry, const float* __restrict__ start, float* __restrict__ state,
-                  T* __restrict__ out, int tokens) {
+lru_output_kernel(const T* __restrict__ y, const float* __restrict__ terms, LruParams p, const int* __restrict__ row_of_token,
+                  const int* __restrict__ cu_q, const int* __restrict__ state_slots, const float* __restrict__ carry,
+                  const float* __restrict__ start, float* __restrict__ state, T* __restrict__ out, int tokens) {
   const int w = blockIdx.x, c = blockIdx.y * 128 + threadIdx.x;
   if (c >= p.width) return;
-  const float rate = 8.0f * softplus_of(p.lam[c]), yb = p.y_bias[c];
+  const float yb = p.y_bias[c];
+  const int b = c / p.size, j = c - b * p.size;
+  const float* at = terms + static_cast<size_t>(b) * tokens * 2 * p.size + j;
   const int end = min((w + 1) * LRU_WINDOW, tokens);
   int t = w * LRU_WINDOW;
   while (t < end) {
@@ -197,10 +216,7 @@ lru_output_kernel(const T* __restrict__ u, const T* __restrict__ y, const float*
     float S = t == cu_q[r] ? start[static_cast<size_t>(r) * p.width + c] : carry[static_cast<size_t>(w) * p.width + c];
 #pragma unroll 4
     for (; t < stop; ++t) {
-      float rp, ip, a, add;
-      pre_of(pre, p, tokens, t, c, rp, ip);
-      lru_terms(rp, ip, to_f32<T>(u[static_cast<size_t>(t) * p.width + c]), rate, a, add);
-      S = fmaf(a, S, add);
+      S = fmaf(at[static_cast<size_t>(t) * 2 * p.size], S, at[static_cast<size_t>(t) * 2 * p.size + p.size]);
       out[static_cast<size_t>(t) * p.width + c] =
           from_f32<T>(S * gelu_tanh_of(to_f32<T>(y[static_cast<size_t>(t) * p.y_stride + c]) + yb));
     }
@@ -253,10 +269,10 @@ B200_EXPORT int b200_lru_rows(const void* u, const void* y, int dtype, int y_str
   return B200_BAD_DTYPE;
 }
 
-// Scratch: win_a, win_s, carry [ceil(tokens / 32), width] floats each, start [num_rows, width] floats.
+// `pre` is overwritten.  Scratch: win_a, win_s, carry [ceil(tokens / 32), width] floats each, start [num_rows, width] floats.
 B200_EXPORT int b200_lru_window() { return LRU_WINDOW; }
 
-B200_EXPORT int b200_lru_scan(const void* u, const void* y, int dtype, int y_stride, const float* pre, const float* r_bias,
+B200_EXPORT int b200_lru_scan(const void* u, const void* y, int dtype, int y_stride, float* pre, const float* r_bias,
                               const float* i_bias, const float* lam, const float* y_bias, int width, int blocks, float* state,
                               const int* row_of_token, const int* cu_q, const int* prefix_len, const int* state_slots,
                               float* win_a, float* win_s, float* carry, float* start, void* out, int tokens, int num_rows,
@@ -268,12 +284,10 @@ B200_EXPORT int b200_lru_scan(const void* u, const void* y, int dtype, int y_str
   const dim3 wgrid(windows, (width + 127) / 128), rgrid(num_rows, (width + 127) / 128);
 #define B200_LRU_SCAN(T)                                                                                                  \
   do {                                                                                                                    \
-    if (windows > 1)                                                                                                      \
-      lru_window_kernel<T><<<wgrid, 128, 0, stream>>>(static_cast<const T*>(u), pre, p, row_of_token, cu_q, win_a, win_s, tokens); \
+    lru_window_kernel<T><<<wgrid, 128, 0, stream>>>(static_cast<const T*>(u), pre, p, row_of_token, cu_q, win_a, win_s, tokens); \
     lru_fold_kernel<<<rgrid, 128, 0, stream>>>(p, state, cu_q, prefix_len, state_slots, win_a, win_s, carry, start);      \
-    lru_output_kernel<T><<<wgrid, 128, 0, stream>>>(static_cast<const T*>(u), static_cast<const T*>(y), pre, p,           \
-                                                    row_of_token, cu_q, state_slots, carry, start, state,                 \
-                                                    static_cast<T*>(out), tokens);                                        \
+    lru_output_kernel<T><<<wgrid, 128, 0, stream>>>(static_cast<const T*>(y), pre, p, row_of_token, cu_q, state_slots,     \
+                                                    carry, start, state, static_cast<T*>(out), tokens);                   \
     return b200_check_launch();                                                                                           \
   } while (0)
   if (dtype == B200_F32) B200_LRU_SCAN(float);

@@ -214,7 +214,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap amap, const __grid_const
             for (int e = 0; e < 32; ++e) {
               const float gate = __bfloat162float(__float2bfloat16_rn(g[e]));
               const float up = __bfloat162float(__float2bfloat16_rn(u[e]));
-              r[e] = __float2bfloat16_rn(gate / (1.0f + expf(-gate)) * up);
+              r[e] = __float2bfloat16_rn(glu_gate(gate) * up);
             }
             if (col0 + 32 <= half && (half % 8) == 0) {
 #pragma unroll

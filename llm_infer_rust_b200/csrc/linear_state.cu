@@ -14,8 +14,7 @@
 //
 //   state_prepare   the four inputs of every token in float (qf, kf [tokens, kv_heads * d], vf [tokens, heads * dv],
 //                   gf [tokens, heads * d], beta [tokens, heads])
-//   state_scan      the recurrence, token by token in the sequence's order whatever the step's cut: a position's
-//                   result has the same bits however the prompt was cut and whatever else is in the step
+//   state_scan      the recurrence, token by token in the sequence's order whatever the step's cut
 //   state_decode    a step whose rows bring one token each: inputs, recurrence, per-head norm and output gate in one
 //                   kernel, a block a (row, head)
 //
@@ -113,160 +112,412 @@ state_prepare_kernel(TapsInput<T> in, LinearStateShape s, const float* __restric
   for (int e = lane; e < s.d; e += 32) dst[e] = value(c0 + e) * f;
 }
 
-// ------------------------------------------------------------------ the recurrence, token by token
-// grid (rows, heads, column tiles of 32).  A block owns 32 columns of one head's state; a column belongs to eight
-// neighbouring lanes, lane l of them holding the rows 32 n + 4 l .. + 3 in registers (DI = 4 ceil(d / 32) of them).
-// A column's products with k and q are sums over its eight lanes (three shuffles), so a token needs no barrier: the
-// block meets only when the next eight tokens have been fetched into shared memory (copies in flight beside the
-// recurrence, two buffers).
-constexpr int LS_TOKENS = 8;
-constexpr int LS_COLS = 32;
-constexpr int LS_LANES = 8;
+// The same with four channels a thread and LS_PREP_TOKENS consecutive tokens a warp, for head sizes and rows of whole
+// 16-byte pieces (d a multiple of 4 up to 128): a channel's taps stay in registers and its last inputs move along with the
+// tokens, so that a token costs one load of its projection.  grid (token groups, units / 4).
+constexpr int LS_PREP_TOKENS = 8;
 
-template <int DI, bool DELTA>
-__global__ void __launch_bounds__(256)
+template <typename T, int TAPS>            // TAPS 0: no convolution
+__global__ void __launch_bounds__(LS_PREP_WARPS * 32)
+state_prepare_vec_kernel(TapsInput<T> in, LinearStateShape s, const float* __restrict__ z, float* __restrict__ qf,
+                         float* __restrict__ kf, float* __restrict__ vf, float* __restrict__ gf, float* __restrict__ beta,
+                         int tokens) {
+  const int t0 = blockIdx.x * LS_PREP_TOKENS, t1 = min(t0 + LS_PREP_TOKENS, tokens);
+  const int lane = threadIdx.x & 31;
+  const int unit = blockIdx.y * LS_PREP_WARPS + (threadIdx.x >> 5);
+  if (unit >= 2 * s.kv_heads + 2 * s.heads) return;
+  if (unit >= 2 * s.kv_heads + s.heads) {                            // a head's decays
+    const int h = unit - 2 * s.kv_heads - s.heads;
+    const float rate = s.decay_kind == DECAY_SOFTPLUS ? expf(s.a_log[h]) : 0.0f;
+    const int e = 4 * lane;
+    if (e < s.d) {
+      float4 b = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+      if (s.decay_bias != nullptr) b = *reinterpret_cast<const float4*>(s.decay_bias + h * s.d + e);
+#pragma unroll 4
+      for (int t = t0; t < t1; ++t) {
+        const size_t at = static_cast<size_t>(t) * s.heads * s.d + h * s.d + e;
+        const float4 v = *reinterpret_cast<const float4*>(z + at);
+        *reinterpret_cast<float4*>(gf + at) = make_float4(decay_of(v.x + b.x, s, rate), decay_of(v.y + b.y, s, rate),
+                                                          decay_of(v.z + b.z, s, rate), decay_of(v.w + b.w, s, rate));
+      }
+    }
+    if (s.beta_column >= 0 && t0 + lane < t1)
+      beta[static_cast<size_t>(t0 + lane) * s.heads + h] =
+          sigmoid_of(to_f32<T>(in.x[static_cast<size_t>(t0 + lane) * in.in_stride + s.beta_column + h]));
+    return;
+  }
+  const bool is_v = unit >= 2 * s.kv_heads, is_k = !is_v && unit >= s.kv_heads;
+  const int h = is_v ? unit - 2 * s.kv_heads : is_k ? unit - s.kv_heads : unit;
+  const int size = is_v ? s.dv : s.d;
+  const int c0 = is_v ? 2 * s.kv_heads * s.d + h * s.dv : (is_k ? s.kv_heads * s.d : 0) + h * s.d;
+  const int out_stride = is_v ? s.heads * s.dv : s.kv_heads * s.d;
+  float* out = (is_v ? vf : is_k ? kf : qf) + static_cast<size_t>(h) * size;
+  const bool unit_norm = !is_v && s.unit_eps > 0.0f;
+  const float f = (is_v || is_k) ? 1.0f : s.q_scale;
+  constexpr int HIST = TAPS > 1 ? TAPS - 1 : 0;
+  for (int e0 = 0; e0 < size; e0 += 128) {                           // (once for q and k)
+    const int e = e0 + 4 * lane;
+    const bool on = e < size;
+    const int c = c0 + (on ? e : 0);
+    float w[4][TAPS > 0 ? TAPS : 1];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) w[i][j] = in.w[static_cast<size_t>(c + i) * TAPS + j];
+    float past[HIST > 0 ? HIST : 1][4];                              // oldest first
+    for (int t = t0; t < t1; ++t) {
+      if constexpr (HIST > 0) {
+        const int r = in.row_of_token[t];
+        if (t == t0 || t == in.cu_q[r]) {                            // the inputs before this token, from x, the state or nowhere
+          const TapsRow row = taps_row(in, t);
+#pragma unroll
+          for (int j = 0; j < HIST; ++j)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) past[j][i] = taps_past(in, row, t, c + i, HIST - j);
+        }
+      }
+      float now[4], y[4];
+      load_floats<T, 4>(in.x + static_cast<size_t>(t) * in.in_stride + c, now);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        if constexpr (TAPS > 0) {
+          y[i] = 0.0f;
+#pragma unroll
+          for (int j = 0; j < HIST; ++j) y[i] = fmaf(w[i][j], past[j][i], y[i]);
+          y[i] = fmaf(w[i][TAPS - 1], now[i], y[i]);
+        } else {
+          y[i] = now[i];
+        }
+        if (s.silu) y[i] = silu_of(y[i]);
+      }
+      if constexpr (HIST > 0) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+#pragma unroll
+          for (int j = 0; j + 1 < HIST; ++j) past[j][i] = past[j + 1][i];
+          past[HIST - 1][i] = now[i];
+        }
+      }
+      float g = f;
+      if (unit_norm) {
+        float ss = 0.0f;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) ss = on ? fmaf(y[i], y[i], ss) : 0.0f;
+        g *= 1.0f / sqrtf(warp_sum(ss) + s.unit_eps);
+      }
+      if (on)
+        *reinterpret_cast<float4*>(out + static_cast<size_t>(t) * out_stride + e) = make_float4(y[0] * g, y[1] * g, y[2] * g, y[3] * g);
+    }
+  }
+}
+
+// ------------------------------------------------------------------ the recurrence, token by token
+// grid (rows, heads, column tiles of 16 CPT).  A block of four warps owns 16 CPT columns of one head's state; CPT neighbouring
+// columns belong to eight neighbouring lanes, lane l of them holding the rows 32 n + 4 l .. + 3 in registers (DI =
+// 4 ceil(d / 32) a column).  Two columns a thread fetch a token's q, k and decays from shared memory, whose bandwidth a
+// scan runs into, half as often; one a thread spreads a small grid over more warps.
+// A column's products with k and q are sums over its eight lanes (three shuffles), so a token needs no barrier.  Eight
+// tokens at a time come through a ring of LS_STAGES buffers in shared memory (the copies of three more groups are in
+// flight beside the recurrence); a whole group is unrolled, so that a token's read-out overlaps the next token's update.
+constexpr int LS_TOKENS = 8;
+constexpr int LS_STAGES = 4;
+constexpr int LS_LANES = 8;
+constexpr int LS_THREADS = 128;
+
+__device__ __forceinline__ float over_lanes(float v) {
+  v += __shfl_xor_sync(0xffffffffu, v, 4);
+  v += __shfl_xor_sync(0xffffffffu, v, 2);
+  v += __shfl_xor_sync(0xffffffffu, v, 1);
+  return v;
+}
+
+// Eight values a lane, summed over the eight lanes: lane l gets the sum of value l.  The same additions as over_lanes
+// makes, in seven shuffles.
+__device__ __forceinline__ float eight_over_lanes(const float (&v)[8], int l) {
+  float a[4], b[2];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) a[i] = ((l & 4) ? v[i + 4] : v[i]) + __shfl_xor_sync(0xffffffffu, (l & 4) ? v[i] : v[i + 4], 4);
+#pragma unroll
+  for (int i = 0; i < 2; ++i) b[i] = ((l & 2) ? a[i + 2] : a[i]) + __shfl_xor_sync(0xffffffffu, (l & 2) ? a[i] : a[i + 2], 2);
+  return ((l & 1) ? b[1] : b[0]) + __shfl_xor_sync(0xffffffffu, (l & 1) ? b[0] : b[1], 1);
+}
+
+// A token's inputs on this lane's rows.
+template <int DI, int CPT>
+struct LaneInputs {
+  float q[DI], k[DI], g[DI], v[CPT], beta;
+
+  // tk: the token's buffer (q, k, g of dp floats each, COLS values, the step); pieces of a lane are 32 floats apart
+  __device__ __forceinline__ void load(const float* tk, int dp, int l, int cj, int cols, bool delta) {
+    const float4* q4 = reinterpret_cast<const float4*>(tk) + l;
+    const float4* k4 = reinterpret_cast<const float4*>(tk + dp) + l;
+    const float4* g4 = reinterpret_cast<const float4*>(tk + 2 * dp) + l;
+#pragma unroll
+    for (int i = 0; i < DI / 4; ++i) {
+      const float4 a = g4[8 * i], b = k4[8 * i], c = q4[8 * i];
+      g[4 * i] = a.x; g[4 * i + 1] = a.y; g[4 * i + 2] = a.z; g[4 * i + 3] = a.w;
+      k[4 * i] = b.x; k[4 * i + 1] = b.y; k[4 * i + 2] = b.z; k[4 * i + 3] = b.w;
+      q[4 * i] = c.x; q[4 * i + 1] = c.y; q[4 * i + 2] = c.z; q[4 * i + 3] = c.w;
+    }
+#pragma unroll
+    for (int j = 0; j < CPT; ++j) v[j] = tk[3 * dp + cj + j];
+    beta = delta ? tk[3 * dp + cols] : 0.0f;
+  }
+};
+
+// One token; out: this lane's parts of the read-outs of its columns.
+template <int DI, int CPT, bool DELTA>
+__device__ __forceinline__ void state_token(float (&S)[CPT][DI], const LaneInputs<DI, CPT>& x, float (&out)[CPT]) {
+  float u[CPT];
+  if constexpr (DELTA) {
+    float dot[CPT][4] = {};
+#pragma unroll
+    for (int i = 0; i < DI; ++i)
+#pragma unroll
+      for (int j = 0; j < CPT; ++j) {
+        S[j][i] *= x.g[i];
+        dot[j][i & 3] = fmaf(S[j][i], x.k[i], dot[j][i & 3]);
+      }
+#pragma unroll
+    for (int j = 0; j < CPT; ++j) u[j] = x.beta * (x.v[j] - over_lanes((dot[j][0] + dot[j][1]) + (dot[j][2] + dot[j][3])));
+  }
+  float acc[CPT][4] = {};
+#pragma unroll
+  for (int i = 0; i < DI; ++i)
+#pragma unroll
+    for (int j = 0; j < CPT; ++j) {
+      if constexpr (DELTA) S[j][i] = fmaf(x.k[i], u[j], S[j][i]);
+      else S[j][i] = fmaf(x.g[i], S[j][i], x.k[i] * x.v[j]);
+      acc[j][i & 3] = fmaf(S[j][i], x.q[i], acc[j][i & 3]);
+    }
+#pragma unroll
+  for (int j = 0; j < CPT; ++j) out[j] = (acc[j][0] + acc[j][1]) + (acc[j][2] + acc[j][3]);
+}
+
+// The delta rule over a group of LS_TOKENS tokens, what a token reads of the past being begun one token ahead, so that
+// its sum over the lanes is on its way while the token before it updates the state and is read out.  With D = diag(g_t) S
+// (the state of token t before its update) and the next token's k' and g':
+//     S_t^T (g' k') = D^T (g' k') + u_t (k_t . (g' k'))
+// and neither sum needs u_t.  The group's first token is read directly.
+template <int DI, int CPT>
+__device__ __forceinline__ void delta_group(float (&S)[CPT][DI], const float* cur, int tok, int dp, int l, int cj, int cols,
+                                            float (&part)[CPT][LS_TOKENS]) {
+  LaneInputs<DI, CPT> x[3];                          // this token's, the next one's, and the one's after that on their way
+  x[0].load(cur, dp, l, cj, cols, true);
+  x[1].load(cur + tok, dp, l, cj, cols, true);
+  float past[CPT], mix = 0.0f, u[CPT] = {};
+#pragma unroll
+  for (int tb = 0; tb < LS_TOKENS; ++tb) {
+    const LaneInputs<DI, CPT>&now = x[tb % 3], &next = x[(tb + 1) % 3];
+    if (tb + 2 < LS_TOKENS) x[(tb + 2) % 3].load(cur + (tb + 2) * tok, dp, l, cj, cols, true);
+#pragma unroll
+    for (int i = 0; i < DI; ++i)
+#pragma unroll
+      for (int j = 0; j < CPT; ++j) S[j][i] *= now.g[i];
+    if (tb == 0) {
+#pragma unroll
+      for (int j = 0; j < CPT; ++j) {
+        float dot[4] = {};
+#pragma unroll
+        for (int i = 0; i < DI; ++i) dot[i & 3] = fmaf(S[j][i], now.k[i], dot[i & 3]);
+        past[j] = over_lanes((dot[0] + dot[1]) + (dot[2] + dot[3]));
+      }
+    }
+    float ahead[CPT], ahead_mix = 0.0f;
+    if (tb + 1 < LS_TOKENS) {
+      float dot[CPT][4] = {}, m[4] = {};
+#pragma unroll
+      for (int i = 0; i < DI; ++i) {
+        const float kg = next.k[i] * next.g[i];
+        m[i & 3] = fmaf(kg, now.k[i], m[i & 3]);
+#pragma unroll
+        for (int j = 0; j < CPT; ++j) dot[j][i & 3] = fmaf(kg, S[j][i], dot[j][i & 3]);
+      }
+#pragma unroll
+      for (int j = 0; j < CPT; ++j) ahead[j] = over_lanes((dot[j][0] + dot[j][1]) + (dot[j][2] + dot[j][3]));
+      ahead_mix = over_lanes((m[0] + m[1]) + (m[2] + m[3]));
+    }
+#pragma unroll
+    for (int j = 0; j < CPT; ++j) u[j] = now.beta * (now.v[j] - fmaf(mix, u[j], past[j]));
+#pragma unroll
+    for (int j = 0; j < CPT; ++j) {
+      float acc[4] = {};
+#pragma unroll
+      for (int i = 0; i < DI; ++i) {
+        S[j][i] = fmaf(now.k[i], u[j], S[j][i]);
+        acc[i & 3] = fmaf(S[j][i], now.q[i], acc[i & 3]);
+      }
+      part[j][tb] = (acc[0] + acc[1]) + (acc[2] + acc[3]);
+      past[j] = ahead[j];
+    }
+    mix = ahead_mix;
+  }
+}
+
+template <int DI, bool DELTA, int CPT>
+__global__ void __launch_bounds__(LS_THREADS)
 state_scan_kernel(const float* __restrict__ qf, const float* __restrict__ kf, const float* __restrict__ vf,
                   const float* __restrict__ gf, const float* __restrict__ beta, float* __restrict__ o,
                   float* __restrict__ state, const int* __restrict__ cu_q, const int* __restrict__ prefix_len,
                   const int* __restrict__ state_slots, int heads, int kv_heads, int d, int dv) {
   constexpr int DP = DI * LS_LANES;                                  // d, rounded up to a multiple of 32
-  constexpr int TOK = 3 * DP + LS_COLS + 4;                          // q, k, g, v, beta of one token
-  extern __shared__ __align__(16) float smem[];                      // [2][LS_TOKENS][TOK]
-  const int r = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * LS_COLS;
+  constexpr int THREADS = LS_THREADS, COLS = THREADS / LS_LANES * CPT;
+  constexpr int TOK = 3 * DP + COLS + 4;                             // q, k, g, v, beta of one token
+  extern __shared__ __align__(16) float smem[];                      // [LS_STAGES][LS_TOKENS][TOK]
+  const int r = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * COLS;
   const int hk = h / (heads / kv_heads);
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int l = lane & (LS_LANES - 1);
-  const int cj = warp * 4 + (lane >> 3);                             // column inside the tile
+  const int cj = (warp * 4 + (lane >> 3)) * CPT;                  // the first of this thread's columns inside the tile
   const int col = col0 + cj;
-  const bool col_ok = col < dv;
   const int first = cu_q[r], n = cu_q[r + 1] - first;
   float* st = state + (static_cast<size_t>(state_slots[r]) * heads + h) * d * dv;
   const bool has_past = prefix_len[r] > 0;
 
-  float S[DI];
+  float S[CPT][DI];
 #pragma unroll
   for (int i = 0; i < DI; ++i) {
     const int e = (i >> 2) * 32 + l * 4 + (i & 3);
-    S[i] = (has_past && col_ok && e < d) ? st[static_cast<size_t>(e) * dv + col] : 0.0f;
+#pragma unroll
+    for (int j = 0; j < CPT; ++j)
+      S[j][i] = (has_past && col + j < dv && e < d) ? st[static_cast<size_t>(e) * dv + col + j] : 0.0f;
   }
-  // columns of q, k and g beyond d stay zero in both buffers, and so do columns of v beyond dv
-  for (int i = threadIdx.x; i < 2 * LS_TOKENS * TOK; i += blockDim.x) smem[i] = 0.0f;
-  __syncthreads();
   const bool wide = d % 4 == 0 && dv % 4 == 0;                       // rows of whole 16-byte pieces
-  auto fetch = [&](int base, int buf) {
+  const int vcols = min(COLS, dv - col0);
+  if (d != DP || vcols != COLS) {                                    // columns beyond d and dv stay zero in every buffer
+    for (int i = threadIdx.x; i < LS_STAGES * LS_TOKENS * TOK; i += THREADS) smem[i] = 0.0f;
+    __syncthreads();
+  }
+  // Every thread copies the same pieces of every token: PIECES pairs of an address in the token's inputs (which moves on
+  // by a fixed stride a token) and one in the token's buffer.  16-byte pieces where rows are whole ones, else floats.
+  constexpr int PIECES = (3 * DP / 4 + COLS / 4 + THREADS - 1) / THREADS;
+  const int unit = wide ? 4 : 1;
+  const int dq = d / unit, per = 3 * dq + vcols / unit;
+  auto piece = [&](int p, const float*& src, int& stride, int& to) {
+    const int kind = p < dq ? 0 : p < 2 * dq ? 1 : p < 3 * dq ? 2 : 3;
+    const int at = unit * (p - kind * dq);
+    const int row_heads = kind < 2 ? kv_heads : heads, row_head = kind < 2 ? hk : h, size = kind == 3 ? dv : d;
+    stride = row_heads * size;
+    src = (kind == 0 ? qf : kind == 1 ? kf : kind == 2 ? gf : vf) + static_cast<size_t>(first) * stride + row_head * size +
+          (kind == 3 ? col0 : 0) + at;
+    to = kind * DP + at;
+  };
+  const float* src[PIECES];
+  int stride[PIECES], to[PIECES];
+#pragma unroll
+  for (int i = 0; i < PIECES; ++i) {
+    src[i] = nullptr;
+    stride[i] = to[i] = 0;
+    if (wide && static_cast<int>(threadIdx.x) + i * THREADS < per) piece(threadIdx.x + i * THREADS, src[i], stride[i], to[i]);
+  }
+  auto fetch = [&](int base, int buf) {                              // called for one group after the other
     float* dst = smem + buf * LS_TOKENS * TOK;
     const int nt = min(LS_TOKENS, n - base);
     if (wide) {
-      const int dq = d >> 2, vq = min(LS_COLS, dv - col0) >> 2;
-      const int per = 3 * dq + vq;
-      for (int idx = threadIdx.x; idx < nt * per; idx += blockDim.x) {
-        const int tb = idx / per, p = idx - tb * per;
-        const size_t t = first + base + tb;
-        const float* src;
-        float* to = dst + tb * TOK;
-        if (p < dq) { src = qf + (t * kv_heads + hk) * d + 4 * p; to += 4 * p; }
-        else if (p < 2 * dq) { src = kf + (t * kv_heads + hk) * d + 4 * (p - dq); to += DP + 4 * (p - dq); }
-        else if (p < 3 * dq) { src = gf + (t * heads + h) * d + 4 * (p - 2 * dq); to += 2 * DP + 4 * (p - 2 * dq); }
-        else { src = vf + (t * heads + h) * dv + col0 + 4 * (p - 3 * dq); to += 3 * DP + 4 * (p - 3 * dq); }
-        cp_async16(to, src, true);
+#pragma unroll
+      for (int i = 0; i < PIECES; ++i) {
+        if (src[i] == nullptr) continue;
+        const float* s = src[i] + static_cast<size_t>(base) * stride[i];
+#pragma unroll
+        for (int tb = 0; tb < LS_TOKENS; ++tb) {
+          if (tb < nt) cp_async16(dst + tb * TOK + to[i], s, true);
+          s += stride[i];
+        }
       }
     } else {
-      const int vq = min(LS_COLS, dv - col0), per = 3 * d + vq;
-      for (int idx = threadIdx.x; idx < nt * per; idx += blockDim.x) {
-        const int tb = idx / per, p = idx - tb * per;
-        const size_t t = first + base + tb;
-        float* to = dst + tb * TOK;
-        if (p < d) to[p] = qf[(t * kv_heads + hk) * d + p];
-        else if (p < 2 * d) to[DP + p - d] = kf[(t * kv_heads + hk) * d + p - d];
-        else if (p < 3 * d) to[2 * DP + p - 2 * d] = gf[(t * heads + h) * d + p - 2 * d];
-        else to[3 * DP + p - 3 * d] = vf[(t * heads + h) * dv + col0 + p - 3 * d];
+      for (int p = threadIdx.x; p < per; p += THREADS) {
+        const float* s;
+        int step, at;
+        piece(p, s, step, at);
+        for (int tb = 0; tb < nt; ++tb) dst[tb * TOK + at] = s[static_cast<size_t>(base + tb) * step];
       }
     }
-    if (DELTA && threadIdx.x < nt)
-      dst[threadIdx.x * TOK + 3 * DP + LS_COLS] = beta[static_cast<size_t>(first + base + threadIdx.x) * heads + h];
+    if (DELTA && static_cast<int>(threadIdx.x) < nt)
+      cp_async4(dst + threadIdx.x * TOK + 3 * DP + COLS, beta + static_cast<size_t>(first + base + threadIdx.x) * heads + h);
+  };
+#pragma unroll
+  for (int s = 0; s < LS_STAGES - 1; ++s) {
+    if (s * LS_TOKENS < n) fetch(s * LS_TOKENS, s);
     cp_async_commit();
-  };
-  auto over_lanes = [](float v) {
-    v += __shfl_xor_sync(0xffffffffu, v, 1);
-    v += __shfl_xor_sync(0xffffffffu, v, 2);
-    v += __shfl_xor_sync(0xffffffffu, v, 4);
-    return v;
-  };
-  if (n > 0) fetch(0, 0);
-  for (int base = 0, buf = 0; base < n; base += LS_TOKENS, buf ^= 1) {
-    if (base + LS_TOKENS < n) {
-      fetch(base + LS_TOKENS, buf ^ 1);
-      cp_async_wait<1>();
-    } else {
-      cp_async_wait<0>();
+  }
+  int buf = 0;
+  for (int base = 0; base < n; base += LS_TOKENS) {
+    cp_async_wait<LS_STAGES - 2>();
+    __syncthreads();                                                 // this group is there, the buffer before it is free
+    {
+      const int ahead = base + (LS_STAGES - 1) * LS_TOKENS;
+      if (ahead < n) fetch(ahead, buf == 0 ? LS_STAGES - 1 : buf - 1);
+      cp_async_commit();
     }
-    __syncthreads();
     const int nt = min(LS_TOKENS, n - base);
     const float* cur = smem + buf * LS_TOKENS * TOK;
-    for (int tb = 0; tb < nt; ++tb) {
-      const float* tk = cur + tb * TOK;
-      const float4* q4 = reinterpret_cast<const float4*>(tk) + l;
-      const float4* k4 = reinterpret_cast<const float4*>(tk + DP) + l;
-      const float4* g4 = reinterpret_cast<const float4*>(tk + 2 * DP) + l;
-      const float v = tk[3 * DP + cj];
-      float acc[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-      if constexpr (DELTA) {
-        float kk[DI];
-        float dot[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-#pragma unroll
-        for (int i = 0; i < DI / 4; ++i) {
-          const float4 g = g4[8 * i], k = k4[8 * i];
-          kk[4 * i] = k.x; kk[4 * i + 1] = k.y; kk[4 * i + 2] = k.z; kk[4 * i + 3] = k.w;
-          S[4 * i] *= g.x; S[4 * i + 1] *= g.y; S[4 * i + 2] *= g.z; S[4 * i + 3] *= g.w;
-          dot[0] = fmaf(S[4 * i], k.x, dot[0]); dot[1] = fmaf(S[4 * i + 1], k.y, dot[1]);
-          dot[2] = fmaf(S[4 * i + 2], k.z, dot[2]); dot[3] = fmaf(S[4 * i + 3], k.w, dot[3]);
-        }
-        const float past = over_lanes((dot[0] + dot[1]) + (dot[2] + dot[3]));
-        const float u = tk[3 * DP + LS_COLS] * (v - past);
-#pragma unroll
-        for (int i = 0; i < DI / 4; ++i) {
-          const float4 q = q4[8 * i];
-          S[4 * i] = fmaf(kk[4 * i], u, S[4 * i]); S[4 * i + 1] = fmaf(kk[4 * i + 1], u, S[4 * i + 1]);
-          S[4 * i + 2] = fmaf(kk[4 * i + 2], u, S[4 * i + 2]); S[4 * i + 3] = fmaf(kk[4 * i + 3], u, S[4 * i + 3]);
-          acc[0] = fmaf(S[4 * i], q.x, acc[0]); acc[1] = fmaf(S[4 * i + 1], q.y, acc[1]);
-          acc[2] = fmaf(S[4 * i + 2], q.z, acc[2]); acc[3] = fmaf(S[4 * i + 3], q.w, acc[3]);
-        }
+    float* dst = o + (static_cast<size_t>(first + base) * heads + h) * dv + col;
+    const size_t step = static_cast<size_t>(heads) * dv;
+    if (nt == LS_TOKENS) {
+      // the next token's inputs are on their way to registers while this one's sums go over the lanes (where they fit)
+      constexpr int AHEAD = DI <= 16 ? 2 : 1;
+      float part[CPT][LS_TOKENS];
+      if constexpr (DELTA && AHEAD == 2) {
+        delta_group<DI, CPT>(S, cur, TOK, DP, l, cj, COLS, part);
       } else {
+        LaneInputs<DI, CPT> x[AHEAD];
+        if constexpr (AHEAD == 2) x[0].load(cur, DP, l, cj, COLS, DELTA);
 #pragma unroll
-        for (int i = 0; i < DI / 4; ++i) {
-          const float4 g = g4[8 * i], k = k4[8 * i], q = q4[8 * i];
-          S[4 * i] = fmaf(g.x, S[4 * i], k.x * v); S[4 * i + 1] = fmaf(g.y, S[4 * i + 1], k.y * v);
-          S[4 * i + 2] = fmaf(g.z, S[4 * i + 2], k.z * v); S[4 * i + 3] = fmaf(g.w, S[4 * i + 3], k.w * v);
-          acc[0] = fmaf(S[4 * i], q.x, acc[0]); acc[1] = fmaf(S[4 * i + 1], q.y, acc[1]);
-          acc[2] = fmaf(S[4 * i + 2], q.z, acc[2]); acc[3] = fmaf(S[4 * i + 3], q.w, acc[3]);
+        for (int tb = 0; tb < LS_TOKENS; ++tb) {
+          if constexpr (AHEAD == 2) {
+            if (tb + 1 < LS_TOKENS) x[(tb + 1) & 1].load(cur + (tb + 1) * TOK, DP, l, cj, COLS, DELTA);
+          } else {
+            x[0].load(cur + tb * TOK, DP, l, cj, COLS, DELTA);
+          }
+          float out[CPT];
+          state_token<DI, CPT, DELTA>(S, x[AHEAD == 2 ? tb & 1 : 0], out);
+#pragma unroll
+          for (int j = 0; j < CPT; ++j) part[j][tb] = out[j];
         }
       }
-      const float out = over_lanes((acc[0] + acc[1]) + (acc[2] + acc[3]));
-      if (l == 0 && col_ok) o[(static_cast<size_t>(first + base + tb) * heads + h) * dv + col] = out;
-    }
-    __syncthreads();                                                 // the buffer may be filled again
-  }
-  if (col_ok) {
 #pragma unroll
-    for (int i = 0; i < DI; ++i) {
-      const int e = (i >> 2) * 32 + l * 4 + (i & 3);
-      if (e < d) st[static_cast<size_t>(e) * dv + col] = S[i];
+      for (int j = 0; j < CPT; ++j) {
+        const float mine = eight_over_lanes(part[j], l);             // lane l: token l
+        if (col + j < dv) dst[l * step + j] = mine;
+      }
+    } else {
+      for (int tb = 0; tb < nt; ++tb) {
+        LaneInputs<DI, CPT> x;
+        x.load(cur + tb * TOK, DP, l, cj, COLS, DELTA);
+        float out[CPT];
+        state_token<DI, CPT, DELTA>(S, x, out);
+#pragma unroll
+        for (int j = 0; j < CPT; ++j) {
+          const float mine = over_lanes(out[j]);
+          if (l == 0 && col + j < dv) dst[tb * step + j] = mine;
+        }
+      }
     }
+    buf = buf + 1 == LS_STAGES ? 0 : buf + 1;
+  }
+#pragma unroll
+  for (int i = 0; i < DI; ++i) {
+    const int e = (i >> 2) * 32 + l * 4 + (i & 3);
+#pragma unroll
+    for (int j = 0; j < CPT; ++j)
+      if (col + j < dv && e < d) st[static_cast<size_t>(e) * dv + col + j] = S[j][i];
   }
 }
 
-template <int DI>
+template <int DI, int CPT>
 static int launch_state_scan(const float* qf, const float* kf, const float* vf, const float* gf, const float* beta, float* o,
                              float* state, const int* cu_q, const int* prefix_len, const int* state_slots, int num_rows,
                              int heads, int kv_heads, int d, int dv, cudaStream_t stream) {
-  const size_t smem = 2 * LS_TOKENS * (3 * DI * LS_LANES + LS_COLS + 4) * sizeof(float);
-  const dim3 grid(num_rows, heads, (dv + LS_COLS - 1) / LS_COLS);
-  auto kernel = beta != nullptr ? state_scan_kernel<DI, true> : state_scan_kernel<DI, false>;
+  constexpr int COLS = LS_THREADS / LS_LANES * CPT;
+  const size_t smem = LS_STAGES * LS_TOKENS * (3 * DI * LS_LANES + COLS + 4) * sizeof(float);
+  const dim3 grid(num_rows, heads, (dv + COLS - 1) / COLS);
+  auto kernel = beta != nullptr ? state_scan_kernel<DI, true, CPT> : state_scan_kernel<DI, false, CPT>;
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
     if (e != cudaSuccess) return static_cast<int>(e);
   }
-  kernel<<<grid, 256, smem, stream>>>(qf, kf, vf, gf, beta, o, state, cu_q, prefix_len, state_slots, heads, kv_heads, d, dv);
+  kernel<<<grid, LS_THREADS, smem, stream>>>(qf, kf, vf, gf, beta, o, state, cu_q, prefix_len, state_slots, heads, kv_heads,
+                                                  d, dv);
   return b200_check_launch();
 }
 
@@ -277,6 +528,10 @@ static int launch_state_scan(const float* qf, const float* kf, const float* vf, 
 //   decay pre-activation   z_e = a2[h d + e] . x[a_column ..] (rank a_rank), float sums over the rounded row
 //   gate                   kind 0: sigmoid(g2[h dv + e] . x[g_column ..]) (rank g_rank);  kind 1: silu(x[g_column + h dv + e])
 //   out[t][h dv + e] = o / sqrt(mean(o^2) + eps) * norm_w[e] * gate,   rounded once
+// The launch may overlap the tail of the kernel before it (the packed projection).  What the kernel fetches before it
+// waits for that one is not written by this step's kernels: weights, the step's index arrays, and the states that the
+// step before left, which ended before this step's first kernel began (a step begins with a kernel, the embedding, that
+// does not overlap what is before it).
 struct StateDecodeParams {
   const void *a2, *g2;
   int a_column, a_rank, g_column, g_rank, gate_kind;
@@ -284,8 +539,10 @@ struct StateDecodeParams {
   float eps;
   int own_conv;                // every channel has one reader (as many q/k heads as heads): it brings the row's convolution
                                // state up to date itself
+  int stage;                   // the head's rows of a2 and g2 go through shared memory (ranks of whole 16-byte pieces)
 };
 
+// w . v over `rank` elements, eight at a time where a row is whole 16-byte pieces
 template <typename T>
 __device__ __forceinline__ float low_rank_dot(const T* __restrict__ w, const float* __restrict__ v, int rank) {
   float s = 0.0f;
@@ -302,11 +559,16 @@ __device__ __forceinline__ float low_rank_dot(const T* __restrict__ w, const flo
   return s;
 }
 
+// Bytes of shared memory that a staged row takes: 16 more than its own, so that neighbouring rows begin in other banks.
+template <typename T>
+__host__ __device__ constexpr int staged_row(int rank) { return rank * static_cast<int>(sizeof(T)) + 16; }
+
 template <typename T, int MAXR, bool DELTA, int THREADS>
 __global__ void __launch_bounds__(THREADS, THREADS == 256 ? 2 : 1)
 state_decode_kernel(TapsInput<T> in, LinearStateShape s, StateDecodeParams p, T* __restrict__ out, float* __restrict__ state) {
   pdl_launch_dependents();                          // the kernel after this one may be scheduled; it waits before it reads
   extern __shared__ __align__(16) float smem[];
+  __shared__ float sums[2][THREADS / 32];
   __shared__ float scratch[33];
   const int t = blockIdx.x, h = blockIdx.y;         // a row has one token: row number = token number
   const int d = s.d, dv = s.dv;
@@ -319,12 +581,14 @@ state_decode_kernel(TapsInput<T> in, LinearStateShape s, StateDecodeParams p, T*
   float* low = gate + dv;                           // [a_rank + g_rank]
   const int CG = dv >> 2, RG = THREADS / CG;
   float* part = low + ((p.a_rank + p.g_rank + 3) & ~3);   // [RG][dv] (16-byte aligned: d and dv are multiples of 4)
+  char* rows_a = reinterpret_cast<char*>(part + RG * dv);
+  char* rows_g = rows_a + d * staged_row<T>(p.a_rank);
   const int rg = threadIdx.x / CG, cg = threadIdx.x - rg * CG;
-  pdl_wait();                                        // what this kernel reads belongs to the kernels before it
-  const T* xr = in.x + static_cast<size_t>(t) * in.in_stride;
+  const int slot = in.state_slots[t];
   const bool has_past = in.prefix_len[t] > 0;
-  float* st = state + (static_cast<size_t>(in.state_slots[t]) * s.heads + h) * d * dv;
-  // the state, on its way while the token's inputs are computed
+  const T* a2 = static_cast<const T*>(p.a2) + static_cast<size_t>(h) * d * p.a_rank;
+  const T* g2 = static_cast<const T*>(p.g2) + static_cast<size_t>(h) * dv * p.g_rank;
+  float* st = state + (static_cast<size_t>(slot) * s.heads + h) * d * dv;
   float4 S[MAXR];
 #pragma unroll
   for (int i = 0; i < MAXR; ++i) {
@@ -332,15 +596,31 @@ state_decode_kernel(TapsInput<T> in, LinearStateShape s, StateDecodeParams p, T*
     S[i] = (has_past && rg < RG && e < d) ? *reinterpret_cast<const float4*>(st + static_cast<size_t>(e) * dv + 4 * cg)
                                           : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
   }
-  for (int i = threadIdx.x; i < p.a_rank + (p.gate_kind == 0 ? p.g_rank : 0); i += blockDim.x)
+  if (p.stage) {
+    const int pa = p.a_rank * sizeof(T) / 16, pg = p.gate_kind == 0 ? p.g_rank * static_cast<int>(sizeof(T)) / 16 : 0;
+    for (int i = threadIdx.x; i < d * pa; i += THREADS) {
+      const int e = i / pa, c = i - e * pa;
+      cp_async16(rows_a + e * staged_row<T>(p.a_rank) + 16 * c, reinterpret_cast<const char*>(a2) + 16 * static_cast<size_t>(i), true);
+    }
+    for (int i = threadIdx.x; i < dv * pg; i += THREADS) {
+      const int e = i / pg, c = i - e * pg;
+      cp_async16(rows_g + e * staged_row<T>(p.g_rank) + 16 * c, reinterpret_cast<const char*>(g2) + 16 * static_cast<size_t>(i), true);
+    }
+    cp_async_commit();
+  }
+  pdl_wait();                                        // the packed projection comes from the kernel before
+  const T* xr = in.x + static_cast<size_t>(t) * in.in_stride;
+  for (int i = threadIdx.x; i < p.a_rank + (p.gate_kind == 0 ? p.g_rank : 0); i += THREADS)
     low[i] = to_f32<T>(xr[i < p.a_rank ? p.a_column + i : p.g_column + i - p.a_rank]);
-  TapsRow row = {};
+  TapsRow row;
+  row.local = 0;
+  row.has_past = has_past;
+  row.state = in.w != nullptr ? in.state + static_cast<size_t>(slot) * (in.taps - 1) * in.channels : nullptr;
   const bool conv = in.w != nullptr;
-  if (conv) row = taps_row(in, t);
   auto value = [&](int c) {
     float y = conv ? taps_value(in, row, t, c, false) : to_f32<T>(xr[c]);
     if (p.own_conv && in.taps > 1) {                 // this thread is the channel's only reader and has read it
-      float* past = in.state + static_cast<size_t>(in.state_slots[t]) * (in.taps - 1) * in.channels + c;
+      float* past = in.state + static_cast<size_t>(slot) * (in.taps - 1) * in.channels + c;
       for (int j = 0; j + 2 < in.taps; ++j) past[static_cast<size_t>(j) * in.channels] = has_past ? past[static_cast<size_t>(j + 1) * in.channels] : 0.0f;
       past[static_cast<size_t>(in.taps - 2) * in.channels] = to_f32<T>(xr[c]);
     }
@@ -348,7 +628,8 @@ state_decode_kernel(TapsInput<T> in, LinearStateShape s, StateDecodeParams p, T*
     return y;
   };
   float qq = 0.0f, kk = 0.0f;
-  for (int i = threadIdx.x; i < 2 * d + dv; i += blockDim.x) {
+#pragma unroll 2
+  for (int i = threadIdx.x; i < 2 * d + dv; i += THREADS) {
     if (i < d) {
       const float y = value(hk * d + i);
       q[i] = y;
@@ -361,27 +642,35 @@ state_decode_kernel(TapsInput<T> in, LinearStateShape s, StateDecodeParams p, T*
       v[i - 2 * d] = value(2 * s.kv_heads * d + h * dv + i - 2 * d);
     }
   }
+  qq = warp_sum(qq);
+  kk = warp_sum(kk);
+  if ((threadIdx.x & 31) == 0) { sums[0][threadIdx.x >> 5] = qq; sums[1][threadIdx.x >> 5] = kk; }
+  if (p.stage) cp_async_wait<0>();
+  __syncthreads();
   float qn = s.q_scale, kn = 1.0f;
   if (s.unit_eps > 0.0f) {
-    qn *= 1.0f / sqrtf(block_sum(qq, scratch) + s.unit_eps);
-    kn = 1.0f / sqrtf(block_sum(kk, scratch) + s.unit_eps);
+    qq = kk = 0.0f;
+#pragma unroll
+    for (int w = 0; w < THREADS / 32; ++w) { qq += sums[0][w]; kk += sums[1][w]; }
+    qn *= 1.0f / sqrtf(qq + s.unit_eps);
+    kn = 1.0f / sqrtf(kk + s.unit_eps);
   }
-  __syncthreads();
   const float rate = s.decay_kind == DECAY_SOFTPLUS ? expf(s.a_log[h]) : 0.0f;
-  for (int i = threadIdx.x; i < d + dv; i += blockDim.x) {
+  for (int i = threadIdx.x; i < d + dv; i += THREADS) {
     if (i < d) {
       const float b = s.decay_bias != nullptr ? s.decay_bias[h * d + i] : 0.0f;
-      const float z = low_rank_dot<T>(static_cast<const T*>(p.a2) + static_cast<size_t>(h * d + i) * p.a_rank, low, p.a_rank);
-      g[i] = decay_of(z + b, s, rate);
+      const T* w = p.stage ? reinterpret_cast<const T*>(rows_a + i * staged_row<T>(p.a_rank)) : a2 + static_cast<size_t>(i) * p.a_rank;
+      g[i] = decay_of(low_rank_dot<T>(w, low, p.a_rank) + b, s, rate);
       q[i] *= qn;
       k[i] *= kn;
     } else {
       const int e = i - d;
-      if (p.gate_kind == 0)
-        gate[e] = sigmoid_of(low_rank_dot<T>(static_cast<const T*>(p.g2) + static_cast<size_t>(h * dv + e) * p.g_rank,
-                                             low + p.a_rank, p.g_rank));
-      else
-        gate[e] = silu_of(to_f32<T>(xr[p.g_column + h * dv + e]));
+      if (p.gate_kind == 0) {
+        const T* w = p.stage ? reinterpret_cast<const T*>(rows_g + e * staged_row<T>(p.g_rank)) : g2 + static_cast<size_t>(e) * p.g_rank;
+        gate[e] = sigmoid_of(low_rank_dot<T>(w, low + p.a_rank, p.g_rank)) * p.norm_w[e];
+      } else {
+        gate[e] = silu_of(to_f32<T>(xr[p.g_column + h * dv + e])) * p.norm_w[e];
+      }
     }
   }
   __syncthreads();
@@ -442,7 +731,7 @@ state_decode_kernel(TapsInput<T> in, LinearStateShape s, StateDecodeParams p, T*
   ss = block_sum(ss, scratch);
   const float f = 1.0f / sqrtf(ss / static_cast<float>(dv) + p.eps);
   for (int e = threadIdx.x; e < dv; e += blockDim.x)
-    out[static_cast<size_t>(t) * s.heads * dv + h * dv + e] = from_f32<T>(v[e] * f * p.norm_w[e] * gate[e]);
+    out[static_cast<size_t>(t) * s.heads * dv + h * dv + e] = from_f32<T>(v[e] * f * gate[e]);
 }
 
 // ------------------------------------------------------------------ C interface
@@ -465,7 +754,7 @@ static TapsInput<T> conv_input(const void* x, int in_stride, const float* conv_w
 
 static bool shape_ok(const LinearStateShape& s) {
   return s.heads > 0 && s.heads <= 65535 && s.kv_heads > 0 && s.heads % s.kv_heads == 0 && s.d > 0 && s.d <= 512 && s.dv > 0 &&
-         (s.dv + LS_COLS - 1) / LS_COLS <= 65535 && (s.decay_kind == DECAY_LOGISTIC || (s.decay_kind == DECAY_SOFTPLUS && s.a_log != nullptr));
+         (s.dv + 15) / 16 <= 65535 && (s.decay_kind == DECAY_LOGISTIC || (s.decay_kind == DECAY_SOFTPLUS && s.a_log != nullptr));
 }
 
 B200_EXPORT int b200_linear_state_shape_size() { return static_cast<int>(sizeof(LinearStateShape)); }
@@ -484,6 +773,31 @@ B200_EXPORT int b200_state_prepare(const void* x, int dtype, int in_stride, cons
     return B200_BAD_SIZE;
   const dim3 grid(tokens, (2 * s.kv_heads + 2 * s.heads + LS_PREP_WARPS - 1) / LS_PREP_WARPS);
   if (grid.y > 65535) return B200_BAD_SIZE;
+  const bool vec = s.d % 4 == 0 && s.d <= 128 && s.dv % 4 == 0 && in_stride % 8 == 0 && reinterpret_cast<uintptr_t>(x) % 16 == 0 &&
+                   (conv_w == nullptr || taps <= 4);
+  if (vec) {
+    const dim3 vgrid((tokens + LS_PREP_TOKENS - 1) / LS_PREP_TOKENS, grid.y);
+#define LS_PREP(T, N)                                                                                                    \
+  state_prepare_vec_kernel<T, N><<<vgrid, LS_PREP_WARPS * 32, 0, stream>>>(                                               \
+      conv_input<T>(x, in_stride, conv_w, taps, channels, conv_state, row_of_token, cu_q, prefix_len, state_slots), s, z, \
+      qf, kf, vf, gf, beta, tokens)
+#define LS_PREP_TAPS(T)                          \
+  do {                                           \
+    switch (conv_w == nullptr ? 0 : taps) {      \
+      case 0: LS_PREP(T, 0); break;              \
+      case 1: LS_PREP(T, 1); break;              \
+      case 2: LS_PREP(T, 2); break;              \
+      case 3: LS_PREP(T, 3); break;              \
+      default: LS_PREP(T, 4); break;             \
+    }                                            \
+  } while (0)
+    if (dtype == B200_F32) LS_PREP_TAPS(float);
+    else if (dtype == B200_BF16) LS_PREP_TAPS(__nv_bfloat16);
+    else return B200_BAD_DTYPE;
+#undef LS_PREP_TAPS
+#undef LS_PREP
+    return b200_check_launch();
+  }
   if (dtype == B200_F32)
     state_prepare_kernel<float><<<grid, LS_PREP_WARPS * 32, 0, stream>>>(
         conv_input<float>(x, in_stride, conv_w, taps, channels, conv_state, row_of_token, cu_q, prefix_len, state_slots), s,
@@ -503,13 +817,20 @@ B200_EXPORT int b200_state_scan(const float* qf, const float* kf, const float* v
                                 int heads, int kv_heads, int d, int dv, cudaStream_t stream) {
   if (num_rows <= 0) return 0;
   if (heads <= 0 || heads > 65535 || kv_heads <= 0 || heads % kv_heads || d <= 0 || d > 512 || dv <= 0 ||
-      (dv + LS_COLS - 1) / LS_COLS > 65535)
+      (dv + 15) / 16 > 65535)
     return B200_BAD_SIZE;
   const int blocks = (d + 31) / 32;
+  // The delta rule's longer chain gains from narrow tiles while they leave a scheduler (148 SMs of four) one warp at most;
+  // else wide ones are ahead (measured, one row of 2,048 tokens: 16 heads of 128 x 128 with the delta rule 466 us narrow;
+  // 32 heads 740 us narrow, 646 us wide; without it 16 heads of 64 x 128 218 against 191 us, 32 heads 355 against 239 us).
+  const bool narrow = beta != nullptr && static_cast<long long>(num_rows) * heads * ((dv + 3) / 4) <= 4 * 148;
 #define LS_CASE(N)                                                                                                    \
+  if (blocks <= N && narrow)                                                                                          \
+    return launch_state_scan<4 * N, 1>(qf, kf, vf, gf, beta, o, state, cu_q, prefix_len, state_slots, num_rows,        \
+                                       heads, kv_heads, d, dv, stream);                                               \
   if (blocks <= N)                                                                                                    \
-    return launch_state_scan<4 * N>(qf, kf, vf, gf, beta, o, state, cu_q, prefix_len, state_slots, num_rows, heads,   \
-                                    kv_heads, d, dv, stream)
+    return launch_state_scan<4 * N, 2>(qf, kf, vf, gf, beta, o, state, cu_q, prefix_len, state_slots, num_rows,        \
+                                       heads, kv_heads, d, dv, stream)
   LS_CASE(1);
   LS_CASE(2);
   LS_CASE(3);
@@ -525,6 +846,10 @@ template <typename T, int MAXR, int THREADS>
 static int launch_state_decode(const TapsInput<T>& in, const LinearStateShape& s, const StateDecodeParams& p, void* out,
                                float* state, int rows, size_t smem, cudaStream_t stream) {
   auto kernel = s.beta_column >= 0 ? state_decode_kernel<T, MAXR, true, THREADS> : state_decode_kernel<T, MAXR, false, THREADS>;
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    if (e != cudaSuccess) return static_cast<int>(e);
+  }
   return b200_launch(kernel, dim3(rows, s.heads), dim3(THREADS), smem, stream, 0, in, s, p, static_cast<T*>(out), state);
 }
 
@@ -537,7 +862,7 @@ B200_EXPORT int b200_state_decode(const void* x, int dtype, int in_stride, const
                                   int rows, cudaStream_t stream) {
   if (rows <= 0) return 0;
   const LinearStateShape s = *shape;
-  const StateDecodeParams p = *params;
+  StateDecodeParams p = *params;
   const int channels = 2 * s.kv_heads * s.d + s.heads * s.dv;
   if (!shape_ok(s) || in_stride < channels || taps > TAPS_MAX || (conv_w != nullptr && taps > 1 && conv_state == nullptr) ||
       s.dv % 4 != 0 || s.d % 4 != 0 || s.dv > 1024 || (p.own_conv && s.heads != s.kv_heads) || p.a_rank < 0 || p.g_rank < 0 || reinterpret_cast<uintptr_t>(state) % 16 != 0)
@@ -547,8 +872,14 @@ B200_EXPORT int b200_state_decode(const void* x, int dtype, int in_stride, const
   if (cg > threads || (s.d + threads / cg - 1) / (threads / cg) > 16) threads = 512;
   if (cg > threads) return B200_BAD_SIZE;
   const int rg = threads / cg, per = (s.d + rg - 1) / rg;
-  const size_t smem = (3 * static_cast<size_t>(s.d) + 2 * s.dv + ((p.a_rank + p.g_rank + 3) & ~3) + static_cast<size_t>(rg) * s.dv) * sizeof(float);
-  if (per > 20 || smem > 48 * 1024) return B200_BAD_SIZE;
+  const size_t plain = (3 * static_cast<size_t>(s.d) + 2 * s.dv + ((p.a_rank + p.g_rank + 3) & ~3) + static_cast<size_t>(rg) * s.dv) * sizeof(float);
+  if (per > 20 || plain > 48 * 1024) return B200_BAD_SIZE;
+  // the low-rank factors' rows of a head through shared memory, if they are whole pieces and two blocks still fit an SM
+  const size_t item = dtype == B200_F32 ? 4 : 2;
+  const size_t staged = s.d * (p.a_rank * item + 16) + (p.gate_kind == 0 ? s.dv * (p.g_rank * item + 16) : 0);
+  p.stage = p.a_rank % 8 == 0 && (p.gate_kind != 0 || p.g_rank % 8 == 0) && plain + staged <= 100 * 1024 &&
+            (reinterpret_cast<uintptr_t>(p.a2) | reinterpret_cast<uintptr_t>(p.g2)) % 16 == 0;
+  const size_t smem = plain + (p.stage ? staged : 0);
 #define LS_DECODE(T)                                                                                                    \
   do {                                                                                                                  \
     const TapsInput<T> in = conv_input<T>(x, in_stride, conv_w, taps, channels, conv_state, row_of_token, cu_q, prefix_len, \

@@ -714,7 +714,7 @@ skinny_linear_kernel(const __grid_constant__ CUtensorMap wmap, const SkinnyParam
       const float gf[4] = {gate4.x, gate4.y, gate4.z, gate4.w}, uf[4] = {up4.x, up4.y, up4.z, up4.w};
       __align__(8) bf16 h[4];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) h[e] = __float2bfloat16_rn(gf[e] / (1.0f + expf(-gf[e])) * uf[e]);
+      for (int e = 0; e < 4; ++e) h[e] = __float2bfloat16_rn(glu_gate(gf[e]) * uf[e]);
       const size_t at = static_cast<size_t>(m) * inter + col;
       if (whole) *reinterpret_cast<uint2*>(static_cast<bf16*>(p.out) + at) = *reinterpret_cast<uint2*>(h);
       else

@@ -448,7 +448,7 @@ __global__ void __launch_bounds__(MAX_THREADS, 1) stream_linear_kernel(const Str
         const int m = i / COLS, rr = i - m * COLS, col = tile * COLS + rr;
         if (col >= inter) continue;
         const float gate = total_of(rr, m), up = total_of(COLS + rr, m);
-        static_cast<bf16*>(p.out)[static_cast<size_t>(m) * inter + col] = __float2bfloat16_rn(gate / (1.0f + expf(-gate)) * up);
+        static_cast<bf16*>(p.out)[static_cast<size_t>(m) * inter + col] = __float2bfloat16_rn(glu_gate(gate) * up);
       }
     }
     group_barrier(grp, gthreads);       // the sums are read: the next tile may overwrite them

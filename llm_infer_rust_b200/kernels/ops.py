@@ -597,7 +597,11 @@ def _sm_count(device) -> int:
     return _sm_counts[key]
 
 
-def _skinny(qkv_forms: bool = False):
+# The gate's activation in a fused product: builds of their own, so that the dense models' stay as they are.
+_GLU_DEFINES = {"silu": {}, "gelu_tanh": {"GLU_GELU_TANH": 1}}
+
+
+def _skinny(qkv_forms: bool = False, glu: str = "silu"):
     # (with a trace buffer set, the build that stamps its clocks: a tuning aid, compiled when first asked for;
     # ``qkv_forms``: the build whose QKV epilogue knows the further forms, which the dense models' build leaves out)
     defines = {}
@@ -605,6 +609,7 @@ def _skinny(qkv_forms: bool = False):
         defines["SKINNY_TRACE"] = 1
     if qkv_forms:
         defines["SKINNY_QKV_FORMS"] = 1
+    defines.update(_GLU_DEFINES[glu])
     lib = load_cuda_library("skinny_linear.cu", defines or None)
     if not getattr(lib, "_checked", False):
         if lib.b200_skinny_params_size() != ctypes.sizeof(_SkinnyParams):
@@ -669,7 +674,7 @@ def graph_capture(graph: "torch.cuda.CUDAGraph"):
 
 def skinny_linear(x, weight: torch.Tensor, mode: int = EPI_PLAIN_BF16, x_rows: Optional[torch.Tensor] = None,
                   qkv: Optional[dict] = None, out: Optional[torch.Tensor] = None, norm_after=None,
-                  stats=None) -> torch.Tensor:
+                  stats=None, glu: str = "silu") -> torch.Tensor:
     """epilogue(prologue(x) . weight^T) for at most 16 rows, in one kernel.
 
     ``out``: the tensor to fill (PLAIN and SWIGLU; made here when None).  ``norm_after`` = (residual, sum_out,
@@ -703,7 +708,7 @@ def skinny_linear(x, weight: torch.Tensor, mode: int = EPI_PLAIN_BF16, x_rows: O
     if not skinny_ok(m, weight, src.dtype, mode, head_dim):
         raise KernelError("the few-row product refuses this size or dtype")
     lib = _skinny(qkv_forms=bool(qkv) and (qkv.get("inv_freq") is not None or bool(qkv.get("plain_norm"))
-                                           or bool(qkv.get("norm_after_rotation")) or bool(qkv.get("values_are_keys"))))
+                                           or bool(qkv.get("norm_after_rotation")) or bool(qkv.get("values_are_keys"))), glu=glu)
     P = _SkinnyParams()
     P.x, P.x_rows = src.data_ptr(), (0 if rows_t is None else rows_t.data_ptr())
     if pending is not None:
@@ -785,8 +790,8 @@ class _StreamParams(ctypes.Structure):
                 ("xd", ctypes.c_int), ("pair", ctypes.c_int)]
 
 
-def _stream_lib():
-    lib = load_cuda_library("stream_linear.cu")
+def _stream_lib(glu: str = "silu"):
+    lib = load_cuda_library("stream_linear.cu", _GLU_DEFINES[glu] or None)
     if not getattr(lib, "_checked", False):
         if lib.b200_stream_params_size() != ctypes.sizeof(_StreamParams):
             raise KernelError("the parameter block of stream_linear.cu and its Python mirror differ")
@@ -843,7 +848,7 @@ def stream_tile_cols(mode: int, m: int, n: int, k: int, norm: bool) -> int:
 
 def stream_linear(x, weight: torch.Tensor, mode: int = EPI_PLAIN_BF16, x_rows: Optional[torch.Tensor] = None,
                   out: Optional[torch.Tensor] = None, norm_after=None, rw: int = 0, ks: int = 0,
-                  xd: int = -1, pair: Optional[int] = None) -> torch.Tensor:
+                  xd: int = -1, pair: Optional[int] = None, glu: str = "silu") -> torch.Tensor:
     """epilogue(prologue(x) . weight^T) for at most 16 rows and a large weight (csrc/stream_linear.cu).
 
     ``x``: a bfloat16 tensor [rows, K] or a ``PendingNorm`` (with or without a residual); ``mode``: EPI_PLAIN_BF16,
@@ -885,7 +890,7 @@ def stream_linear(x, weight: torch.Tensor, mode: int = EPI_PLAIN_BF16, x_rows: O
         P.post_residual, P.post_sum_out, P.post_stats = (t.data_ptr() for t in norm_after)
     P.out, P.rw, P.ks, P.xd = out.data_ptr(), rw, ks, xd
     P.pair = stream_pair if pair is None else pair
-    rc = _stream_lib().b200_stream_linear(ctypes.byref(P), _sm_count(src.device), _stream())
+    rc = _stream_lib(glu).b200_stream_linear(ctypes.byref(P), _sm_count(src.device), _stream())
     _ok(rc, "stream_linear")
     return out
 
@@ -1110,6 +1115,15 @@ def few_row_linear(x, weight: torch.Tensor, mode: int = EPI_PLAIN_BF16, x_rows: 
     return _single_lazy(x, weight, mode, x_rows, qkv, lazy)
 
 
+def few_row_glu(x: torch.Tensor, weight: torch.Tensor, activation: str = "silu") -> torch.Tensor:
+    """act(gate x) * (up x) for few rows of a plain tensor, weight = [gate rows; up rows], in one kernel (where
+    ``few_row_takes`` an EPI_SWIGLU product on the single route): ``activation`` silu or gelu_tanh."""
+    flush_chain()
+    if stream_takes(x.shape[0], weight, x.dtype, EPI_SWIGLU, False):
+        return stream_linear(x, weight, EPI_SWIGLU, glu=activation)
+    return skinny_linear(x, weight, EPI_SWIGLU, glu=activation)
+
+
 def _chain_append(pending, src, rows_t, m, weight, mode, qkv) -> torch.Tensor:
     global _chain
     _cuda_only(src, weight, rows_t)
@@ -1273,9 +1287,10 @@ def gemm_tc_pays(x: torch.Tensor, weight: torch.Tensor, mode: int = GEMM_PLAIN) 
     return x.shape[1] >= 2048 and tiles >= 4 * _sm_count(x.device)
 
 
-def gemm_tc(x: torch.Tensor, weight: torch.Tensor, mode: int = GEMM_PLAIN) -> torch.Tensor:
+def gemm_tc(x: torch.Tensor, weight: torch.Tensor, mode: int = GEMM_PLAIN, glu: str = "silu") -> torch.Tensor:
     """x . weight^T on the tcgen05 tensor cores (TMA-fed, float sums in tensor memory), bfloat16 out.
-    ``GEMM_SWIGLU``: weight = [gate rows; up rows]; the result is silu(x . gate^T) * (x . up^T)."""
+    ``GEMM_SWIGLU``: weight = [gate rows; up rows]; the result is silu(x . gate^T) * (x . up^T) (``glu`` "gelu_tanh":
+    that activation)."""
     flush_chain()
     if not gemm_tc_ok(x, weight, mode):
         raise KernelError("the tcgen05 product takes contiguous bfloat16 [M, K] and [N, K] with K a multiple of 8")
@@ -1283,7 +1298,7 @@ def gemm_tc(x: torch.Tensor, weight: torch.Tensor, mode: int = GEMM_PLAIN) -> to
     n = weight.shape[0]
     out = torch.empty((m, n // 2 if mode == GEMM_SWIGLU else n), dtype=torch.bfloat16, device=x.device)
     a_map = ctypes.create_string_buffer(128)          # activations move: their descriptor is made per call
-    lib = load_cuda_library("gemm_tcgen05.cu")
+    lib = load_cuda_library("gemm_tcgen05.cu", _GLU_DEFINES[glu] or None)
     rc = lib.b200_gemm_tensor_map(a_map, _p(x), ctypes.c_longlong(m), ctypes.c_longlong(k))
     if rc != 0:
         raise KernelError(f"the TMA descriptor of the activations could not be made (code {rc})")
@@ -1635,7 +1650,8 @@ class _StateDecodeParams(ctypes.Structure):
     """Mirror of ``StateDecodeParams`` in csrc/linear_state.cu."""
     _fields_ = [("a2", ctypes.c_void_p), ("g2", ctypes.c_void_p), ("a_column", ctypes.c_int), ("a_rank", ctypes.c_int),
                 ("g_column", ctypes.c_int), ("g_rank", ctypes.c_int), ("gate_kind", ctypes.c_int),
-                ("norm_w", ctypes.c_void_p), ("eps", ctypes.c_float), ("own_conv", ctypes.c_int)]
+                ("norm_w", ctypes.c_void_p), ("eps", ctypes.c_float), ("own_conv", ctypes.c_int),
+                ("stage", ctypes.c_int)]
 
 
 def _linear_state():
@@ -1714,7 +1730,7 @@ def state_decode(form: LinearStateForm, x: torch.Tensor, conv: Optional[torch.Te
     own = form.heads == form.kv_heads
     params = _StateDecodeParams(a2.data_ptr(), g2.data_ptr() if g2 is not None else None, int(a_column), a2.shape[1],
                                 int(gate_column), g2.shape[1] if g2 is not None else 0, int(g2 is None), norm.data_ptr(),
-                                float(eps), int(own))
+                                float(eps), int(own), 0)
     rc = _linear_state().b200_state_decode(
         _p(x), _code(x), x.shape[1], _p(conv), taps, _p(conv_state), _p(ctx.row_of_token), _p(ctx.cu_q), _p(ctx.prefix_len),
         _p(ctx.state_slots), ctypes.byref(form.shape), ctypes.byref(params), _p(out), _p(state), x.shape[0], _stream())

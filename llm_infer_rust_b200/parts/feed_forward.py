@@ -92,7 +92,7 @@ class DenseActFF(Part):
 
 class GatedActFF(Part):
     """down(act(gate(x)) * up(x)), no bias, gate and up packed into one matrix (gate rows first); ``activation``:
-    gelu_tanh or silu, computed in float on the rounded projections and rounded once."""
+    gelu_tanh or silu, computed in float.  The dense models' fused products (few tokens; large portions) serve it too."""
     category = "feed_forward"
     _GLU = {"gelu_tanh": "gelu_tanh", "silu": "silu"}
 
@@ -109,8 +109,15 @@ class GatedActFF(Part):
                 "down_proj": ParamDecl((self.hidden, self.inter))}
 
     def forward(self, x):
-        gate_up = ops.linear(x, self.params["gate_up_proj"])
-        return ops.linear(ops.glu_columns(gate_up, self._GLU[self.activation]), self.params["down_proj"])
+        w, act = self.params["gate_up_proj"], self._GLU[self.activation]
+        if x.dtype == torch.bfloat16 and ops.few_row_route == "single" and \
+                ops.few_row_takes(x.shape[0], w, self.env.dtype, ops.EPI_SWIGLU, norm=False):
+            a = ops.few_row_glu(x, w, act)                       # few tokens: both projections and the activation in one kernel
+        elif x.dtype == torch.bfloat16 and ops.gemm_tc_pays(x, w, ops.GEMM_SWIGLU):
+            a = ops.gemm_tc(x, w, ops.GEMM_SWIGLU, glu=act)      # many tokens, large matrices: as the tcgen05 product's epilogue
+        else:
+            a = ops.glu_columns(ops.linear(x, w), act)
+        return ops.linear(a, self.params["down_proj"])
 
 
 class TableExperts(Part):
