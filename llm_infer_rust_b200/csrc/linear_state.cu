@@ -216,11 +216,12 @@ state_prepare_vec_kernel(TapsInput<T> in, LinearStateShape s, const float* __res
 // columns belong to eight neighbouring lanes, lane l of them holding the rows 32 n + 4 l .. + 3 in registers (DI =
 // 4 ceil(d / 32) a column).  Two columns a thread fetch a token's q, k and decays from shared memory, whose bandwidth a
 // scan runs into, half as often; one a thread spreads a small grid over more warps.
-// A column's products with k and q are sums over its eight lanes (three shuffles), so a token needs no barrier.  Eight
-// tokens at a time come through a ring of LS_STAGES buffers in shared memory (the copies of three more groups are in
-// flight beside the recurrence); a whole group is unrolled, so that a token's read-out overlaps the next token's update.
-constexpr int LS_TOKENS = 8;
-constexpr int LS_STAGES = 4;
+// A column's products with k and q are sums over its eight lanes (three shuffles), so a token needs no barrier.  Groups of
+// tokens come through a ring of buffers in shared memory (the copies of the next groups are in flight beside the
+// recurrence); eight tokens are unrolled, so that a token's read-out overlaps the next token's update.
+constexpr int LS_TOKENS = 8;                               // tokens that are unrolled
+constexpr int ls_group(int di) { return di <= 16 ? 16 : 8; }      // tokens of a buffer
+constexpr int ls_stages(int di) { return di <= 16 ? 3 : 4; }
 constexpr int LS_LANES = 8;
 constexpr int LS_THREADS = 128;
 
@@ -363,7 +364,8 @@ state_scan_kernel(const float* __restrict__ qf, const float* __restrict__ kf, co
   constexpr int DP = DI * LS_LANES;                                  // d, rounded up to a multiple of 32
   constexpr int THREADS = LS_THREADS, COLS = THREADS / LS_LANES * CPT;
   constexpr int TOK = 3 * DP + COLS + 4;                             // q, k, g, v, beta of one token
-  extern __shared__ __align__(16) float smem[];                      // [LS_STAGES][LS_TOKENS][TOK]
+  constexpr int GROUP = ls_group(DI), STAGES = ls_stages(DI);
+  extern __shared__ __align__(16) float smem[];                      // [STAGES][GROUP][TOK]
   const int r = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * COLS;
   const int hk = h / (heads / kv_heads);
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -385,12 +387,15 @@ state_scan_kernel(const float* __restrict__ qf, const float* __restrict__ kf, co
   const bool wide = d % 4 == 0 && dv % 4 == 0;                       // rows of whole 16-byte pieces
   const int vcols = min(COLS, dv - col0);
   if (d != DP || vcols != COLS) {                                    // columns beyond d and dv stay zero in every buffer
-    for (int i = threadIdx.x; i < LS_STAGES * LS_TOKENS * TOK; i += THREADS) smem[i] = 0.0f;
+    for (int i = threadIdx.x; i < STAGES * GROUP * TOK; i += THREADS) smem[i] = 0.0f;
     __syncthreads();
   }
-  // Every thread copies the same pieces of every token: PIECES pairs of an address in the token's inputs (which moves on
-  // by a fixed stride a token) and one in the token's buffer.  16-byte pieces where rows are whole ones, else floats.
-  constexpr int PIECES = (3 * DP / 4 + COLS / 4 + THREADS - 1) / THREADS;
+  // Every thread copies the same pieces of every SLOTS-th token: PIECES pairs of an address in the token's inputs (which
+  // moves on by a fixed stride a token) and one in the token's buffer.  16-byte pieces where rows are whole ones, else floats.
+  constexpr int MOST = 3 * DP / 4 + COLS / 4;                        // pieces of a token
+  constexpr int SLOTS = MOST <= THREADS / 4 ? 4 : MOST <= THREADS / 2 ? 2 : 1;
+  constexpr int LINE = THREADS / SLOTS, PIECES = (MOST + LINE - 1) / LINE;
+  const int line = threadIdx.x % LINE, slot = threadIdx.x / LINE;
   const int unit = wide ? 4 : 1;
   const int dq = d / unit, per = 3 * dq + vcols / unit;
   auto piece = [&](int p, const float*& src, int& stride, int& to) {
@@ -408,20 +413,21 @@ state_scan_kernel(const float* __restrict__ qf, const float* __restrict__ kf, co
   for (int i = 0; i < PIECES; ++i) {
     src[i] = nullptr;
     stride[i] = to[i] = 0;
-    if (wide && static_cast<int>(threadIdx.x) + i * THREADS < per) piece(threadIdx.x + i * THREADS, src[i], stride[i], to[i]);
+    if (wide && line + i * LINE < per) piece(line + i * LINE, src[i], stride[i], to[i]);
   }
   auto fetch = [&](int base, int buf) {                              // called for one group after the other
-    float* dst = smem + buf * LS_TOKENS * TOK;
-    const int nt = min(LS_TOKENS, n - base);
+    float* dst = smem + buf * GROUP * TOK;
+    const int nt = min(GROUP, n - base);
     if (wide) {
 #pragma unroll
       for (int i = 0; i < PIECES; ++i) {
         if (src[i] == nullptr) continue;
-        const float* s = src[i] + static_cast<size_t>(base) * stride[i];
+        const float* s = src[i] + static_cast<size_t>(base + slot) * stride[i];
+        float* d = dst + slot * TOK + to[i];
 #pragma unroll
-        for (int tb = 0; tb < LS_TOKENS; ++tb) {
-          if (tb < nt) cp_async16(dst + tb * TOK + to[i], s, true);
-          s += stride[i];
+        for (int tb = 0; tb < GROUP; tb += SLOTS) {
+          if (tb + slot < nt) cp_async16(d + tb * TOK, s, true);
+          s += SLOTS * stride[i];
         }
       }
     } else {
@@ -436,64 +442,67 @@ state_scan_kernel(const float* __restrict__ qf, const float* __restrict__ kf, co
       cp_async4(dst + threadIdx.x * TOK + 3 * DP + COLS, beta + static_cast<size_t>(first + base + threadIdx.x) * heads + h);
   };
 #pragma unroll
-  for (int s = 0; s < LS_STAGES - 1; ++s) {
-    if (s * LS_TOKENS < n) fetch(s * LS_TOKENS, s);
+  for (int s = 0; s < STAGES - 1; ++s) {
+    if (s * GROUP < n) fetch(s * GROUP, s);
     cp_async_commit();
   }
   int buf = 0;
-  for (int base = 0; base < n; base += LS_TOKENS) {
-    cp_async_wait<LS_STAGES - 2>();
+  for (int base = 0; base < n; base += GROUP) {
+    cp_async_wait<STAGES - 2>();
     __syncthreads();                                                 // this group is there, the buffer before it is free
     {
-      const int ahead = base + (LS_STAGES - 1) * LS_TOKENS;
-      if (ahead < n) fetch(ahead, buf == 0 ? LS_STAGES - 1 : buf - 1);
+      const int ahead = base + (STAGES - 1) * GROUP;
+      if (ahead < n) fetch(ahead, buf == 0 ? STAGES - 1 : buf - 1);
       cp_async_commit();
     }
-    const int nt = min(LS_TOKENS, n - base);
-    const float* cur = smem + buf * LS_TOKENS * TOK;
-    float* dst = o + (static_cast<size_t>(first + base) * heads + h) * dv + col;
-    const size_t step = static_cast<size_t>(heads) * dv;
-    if (nt == LS_TOKENS) {
-      // the next token's inputs are on their way to registers while this one's sums go over the lanes (where they fit)
-      constexpr int AHEAD = DI <= 16 ? 2 : 1;
-      float part[CPT][LS_TOKENS];
-      if constexpr (DELTA && AHEAD == 2) {
-        delta_group<DI, CPT>(S, cur, TOK, DP, l, cj, COLS, part);
-      } else {
-        LaneInputs<DI, CPT> x[AHEAD];
-        if constexpr (AHEAD == 2) x[0].load(cur, DP, l, cj, COLS, DELTA);
+#pragma unroll 1
+    for (int half = 0; half < GROUP && base + half < n; half += LS_TOKENS) {
+      const int nt = min(LS_TOKENS, n - base - half);
+      const float* cur = smem + (buf * GROUP + half) * TOK;
+      float* dst = o + (static_cast<size_t>(first + base + half) * heads + h) * dv + col;
+      const size_t step = static_cast<size_t>(heads) * dv;
+      if (nt == LS_TOKENS) {
+        // the next token's inputs are on their way to registers while this one's sums go over the lanes (where they fit)
+        constexpr int AHEAD = DI <= 16 ? 2 : 1;
+        float part[CPT][LS_TOKENS];
+        if constexpr (DELTA && AHEAD == 2) {
+          delta_group<DI, CPT>(S, cur, TOK, DP, l, cj, COLS, part);
+        } else {
+          LaneInputs<DI, CPT> x[AHEAD];
+          if constexpr (AHEAD == 2) x[0].load(cur, DP, l, cj, COLS, DELTA);
 #pragma unroll
-        for (int tb = 0; tb < LS_TOKENS; ++tb) {
-          if constexpr (AHEAD == 2) {
-            if (tb + 1 < LS_TOKENS) x[(tb + 1) & 1].load(cur + (tb + 1) * TOK, DP, l, cj, COLS, DELTA);
-          } else {
-            x[0].load(cur + tb * TOK, DP, l, cj, COLS, DELTA);
+          for (int tb = 0; tb < LS_TOKENS; ++tb) {
+            if constexpr (AHEAD == 2) {
+              if (tb + 1 < LS_TOKENS) x[(tb + 1) & 1].load(cur + (tb + 1) * TOK, DP, l, cj, COLS, DELTA);
+            } else {
+              x[0].load(cur + tb * TOK, DP, l, cj, COLS, DELTA);
+            }
+            float out[CPT];
+            state_token<DI, CPT, DELTA>(S, x[AHEAD == 2 ? tb & 1 : 0], out);
+#pragma unroll
+            for (int j = 0; j < CPT; ++j) part[j][tb] = out[j];
           }
-          float out[CPT];
-          state_token<DI, CPT, DELTA>(S, x[AHEAD == 2 ? tb & 1 : 0], out);
-#pragma unroll
-          for (int j = 0; j < CPT; ++j) part[j][tb] = out[j];
         }
-      }
-#pragma unroll
-      for (int j = 0; j < CPT; ++j) {
-        const float mine = eight_over_lanes(part[j], l);             // lane l: token l
-        if (col + j < dv) dst[l * step + j] = mine;
-      }
-    } else {
-      for (int tb = 0; tb < nt; ++tb) {
-        LaneInputs<DI, CPT> x;
-        x.load(cur + tb * TOK, DP, l, cj, COLS, DELTA);
-        float out[CPT];
-        state_token<DI, CPT, DELTA>(S, x, out);
 #pragma unroll
         for (int j = 0; j < CPT; ++j) {
-          const float mine = over_lanes(out[j]);
-          if (l == 0 && col + j < dv) dst[tb * step + j] = mine;
+          const float mine = eight_over_lanes(part[j], l);             // lane l: token l
+          if (col + j < dv) dst[l * step + j] = mine;
+        }
+      } else {
+        for (int tb = 0; tb < nt; ++tb) {
+          LaneInputs<DI, CPT> x;
+          x.load(cur + tb * TOK, DP, l, cj, COLS, DELTA);
+          float out[CPT];
+          state_token<DI, CPT, DELTA>(S, x, out);
+#pragma unroll
+          for (int j = 0; j < CPT; ++j) {
+            const float mine = over_lanes(out[j]);
+            if (l == 0 && col + j < dv) dst[tb * step + j] = mine;
+          }
         }
       }
     }
-    buf = buf + 1 == LS_STAGES ? 0 : buf + 1;
+    buf = buf + 1 == STAGES ? 0 : buf + 1;
   }
 #pragma unroll
   for (int i = 0; i < DI; ++i) {
@@ -509,7 +518,7 @@ static int launch_state_scan(const float* qf, const float* kf, const float* vf, 
                              float* state, const int* cu_q, const int* prefix_len, const int* state_slots, int num_rows,
                              int heads, int kv_heads, int d, int dv, cudaStream_t stream) {
   constexpr int COLS = LS_THREADS / LS_LANES * CPT;
-  const size_t smem = LS_STAGES * LS_TOKENS * (3 * DI * LS_LANES + COLS + 4) * sizeof(float);
+  const size_t smem = ls_stages(DI) * ls_group(DI) * (3 * DI * LS_LANES + COLS + 4) * sizeof(float);
   const dim3 grid(num_rows, heads, (dv + COLS - 1) / COLS);
   auto kernel = beta != nullptr ? state_scan_kernel<DI, true, CPT> : state_scan_kernel<DI, false, CPT>;
   if (smem > 48 * 1024) {
