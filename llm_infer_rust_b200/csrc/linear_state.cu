@@ -356,7 +356,7 @@ __device__ __forceinline__ void delta_group(float (&S)[CPT][DI], const float* cu
 }
 
 template <int DI, bool DELTA, int CPT>
-__global__ void __launch_bounds__(LS_THREADS)
+__global__ void __launch_bounds__(LS_THREADS, DI <= 16 ? 3 : 1)
 state_scan_kernel(const float* __restrict__ qf, const float* __restrict__ kf, const float* __restrict__ vf,
                   const float* __restrict__ gf, const float* __restrict__ beta, float* __restrict__ o,
                   float* __restrict__ state, const int* __restrict__ cu_q, const int* __restrict__ prefix_len,
@@ -829,10 +829,8 @@ B200_EXPORT int b200_state_scan(const float* qf, const float* kf, const float* v
       (dv + 15) / 16 > 65535)
     return B200_BAD_SIZE;
   const int blocks = (d + 31) / 32;
-  // The delta rule's longer chain gains from narrow tiles while they leave a scheduler (148 SMs of four) one warp at most;
-  // else wide ones are ahead (measured, one row of 2,048 tokens: 16 heads of 128 x 128 with the delta rule 466 us narrow;
-  // 32 heads 740 us narrow, 646 us wide; without it 16 heads of 64 x 128 218 against 191 us, 32 heads 355 against 239 us).
-  const bool narrow = beta != nullptr && static_cast<long long>(num_rows) * heads * ((dv + 3) / 4) <= 4 * 148;
+  // One column a thread while that leaves a scheduler (148 SMs of four) one warp at most, else two.
+  const bool narrow = static_cast<long long>(num_rows) * heads * ((dv + 3) / 4) <= 4 * 148;
 #define LS_CASE(N)                                                                                                    \
   if (blocks <= N && narrow)                                                                                          \
     return launch_state_scan<4 * N, 1>(qf, kf, vf, gf, beta, o, state, cu_q, prefix_len, state_slots, num_rows,        \
