@@ -58,10 +58,13 @@ class RunEntry:
     ``layer`` indexes ``ModelSpec.layers`` (the weights); the same layer may be
     named by several entries.  Every entry owns a cache of its own unless
     ``reads`` names an EARLIER entry of the run list: then this execution writes
-    no keys and values and its mixer reads the cache of that entry.
+    no keys and values and its mixer reads the cache of that entry.  ``input``
+    names one of ``ModelSpec.stream_inputs``: the stream goes through that part
+    before the layer runs (the first layer of a pass through repeated layers).
     """
     layer: int
     reads: Optional[int] = None
+    input: Optional[str] = None
 
 
 @dataclass(frozen=True)
@@ -76,12 +79,15 @@ class ModelSpec:
     final_norm: PartSpec
     lm_head: PartSpec
     position_encodings: Mapping[str, PartSpec] = field(default_factory=dict)
+    stream_inputs: Mapping[str, PartSpec] = field(default_factory=dict)
 
     def validate(self) -> None:
         for e, entry in enumerate(self.run_list):
             if not 0 <= entry.layer < len(self.layers):
                 raise ConfigError(f"run list entry {e} names layer {entry.layer}, "
                                   f"the model has {len(self.layers)}")
+            if entry.input is not None and entry.input not in self.stream_inputs:
+                raise ConfigError(f"run list entry {e} names the stream input {entry.input!r}, which the model lacks")
             if entry.reads is not None:
                 if not 0 <= entry.reads < e:
                     raise ConfigError(f"run list entry {e} reads the cache of entry {entry.reads}, "

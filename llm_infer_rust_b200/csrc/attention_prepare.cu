@@ -9,6 +9,12 @@
 //     (x / sqrt(mean(x^2) + eps)); PREP_NORM_AFTER_ROTATION: the norm follows the rotation instead of preceding it;
 //     PREP_VALUES_ARE_KEYS: the row holds no v columns and a token's value is its key as projected (with its bias,
 //     before norm and rotation; dv = d).
+//     `maps` M > 1: a query head holds M query vectors and a key head M key vectors of width d, side by side in the
+//     packed row (nh counts query vectors, nkv key/value heads); every vector is normed and rotated by itself.  A key
+//     head's vectors are ONE cache row M d wide, and query vector h goes to a row of that width of its own, zero outside
+//     the columns of its map h % M: its product with the key row is its product with its own map's key, so attention
+//     over keys M d wide serves every map with one fetch of keys and values.
+//     `rot_gain` multiplies cosines and sines (a frequency scaling that also scales the rotated coordinates).
 //
 // (2) latent_prepare: attention over a narrow latent.  The packed row holds per head [d plain | r rotated] query
 //     coordinates (nh * (d + r)), and a second row (`down`, which may be a column range of the same matrix or of
@@ -33,12 +39,14 @@ constexpr int WARPS = 4;
 enum : int { PREP_NORM_PLAIN = 1, PREP_NORM_AFTER_ROTATION = 2, PREP_VALUES_ARE_KEYS = 4 };
 
 __device__ __forceinline__ void rotate_row(float* row, int rot_dims, float pos, const float* __restrict__ inv_freq,
-                                           bool interleaved, int lane) {
+                                           bool interleaved, int lane, float gain = 1.0f) {
   const int half = rot_dims >> 1;
   for (int i = lane; i < half; i += 32) {
     const int a = interleaved ? 2 * i : i, b = interleaved ? 2 * i + 1 : i + half;
     float sn, cs;
     sincosf(pos * inv_freq[i], &sn, &cs);
+    sn *= gain;
+    cs *= gain;
     const float u = row[a], v = row[b];
     row[a] = u * cs - v * sn;
     row[b] = v * cs + u * sn;
@@ -65,29 +73,36 @@ heads_prepare_kernel(const T* __restrict__ x, int in_stride, const float* __rest
                      const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
                      const float* __restrict__ inv_freq, int rot_dims, int interleaved,
                      const int* __restrict__ positions, const int* __restrict__ slots, int tokens, int nh, int nkv,
-                     int d, int dv, int flags, int page_size, long long cache_slots, T* __restrict__ q_out,
-                     T* __restrict__ k_cache, T* __restrict__ v_cache, int* err) {
+                     int d, int dv, int flags, int maps, float rot_gain, int page_size, long long cache_slots,
+                     T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache, int* err) {
   pdl_launch_dependents();                          // the kernel after this one may be scheduled; it waits before it reads
   pdl_wait();                                        // what this kernel reads belongs to the kernels before it
   __shared__ float buf[WARPS][MAX_VEC];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int vectors = nh + 2 * nkv;
+  const int nk = nkv * maps;                         // key vectors
+  const int vectors = nh + nk + nkv;
   const bool v_is_k = (flags & PREP_VALUES_ARE_KEYS) != 0;
   const long long work = static_cast<long long>(blockIdx.x) * WARPS + warp;
   if (work >= static_cast<long long>(tokens) * vectors) return;
   const int t = static_cast<int>(work / vectors);
   const int h = static_cast<int>(work - static_cast<long long>(t) * vectors);
-  const bool is_q = h < nh, is_k = !is_q && h < nh + nkv;
-  const int kvh = is_q ? 0 : (is_k ? h - nh : h - nh - nkv);
+  const bool is_q = h < nh, is_k = !is_q && h < nh + nk;
+  const int vec = is_q ? h : (is_k ? h - nh : h - nh - nk);          // which query vector, key vector or value head
+  const int map = (is_q || is_k) ? vec % maps : 0;
   const int width = (is_q || is_k) ? d : dv;
-  const int col = is_q ? h * d : ((is_k || v_is_k) ? nh * d + kvh * d : (nh + nkv) * d + kvh * dv);
+  const int col = is_q ? vec * d : ((is_k || v_is_k) ? (nh + vec) * d : (nh + nk) * d + vec * dv);
   T* dst;
   if (is_q) {
-    dst = q_out + (static_cast<size_t>(t) * nh + h) * d;
+    dst = q_out + (static_cast<size_t>(t) * nh + vec) * maps * d;
+    for (int i = lane; i < maps * d; i += 32)
+      if (i / d != map) dst[i] = from_f32<T>(0.0f);
+    dst += map * d;
   } else {
     if (slots == nullptr) return;
-    dst = cache_row(is_k ? k_cache : v_cache, slots[t], kvh, nkv, page_size, cache_slots, width, lane, err);
+    dst = cache_row(is_k ? k_cache : v_cache, slots[t], is_k ? vec / maps : vec, nkv, page_size, cache_slots,
+                    is_k ? maps * d : dv, lane, err);
     if (dst == nullptr) return;
+    dst += map * d;
   }
   const T* src = x + static_cast<size_t>(t) * in_stride + col;
   float* row = buf[warp];
@@ -109,7 +124,7 @@ heads_prepare_kernel(const T* __restrict__ x, int in_stride, const float* __rest
   }
   __syncwarp();
   if (rotated) {
-    rotate_row(row, rot_dims, static_cast<float>(positions[t]), inv_freq, interleaved != 0, lane);
+    rotate_row(row, rot_dims, static_cast<float>(positions[t]), inv_freq, interleaved != 0, lane, rot_gain);
     __syncwarp();
   }
   if (normed && norm_last) {
@@ -316,23 +331,24 @@ joint_heads_prepare_kernel(const T* __restrict__ x, int in_stride, const float* 
 B200_EXPORT int b200_heads_prepare(const void* x, int dtype, int in_stride, const float* bias, const float* q_w,
                                    const float* k_w, float eps, const float* inv_freq, int rot_dims, int interleaved,
                                    const int* positions, const int* slots, int tokens, int nh, int nkv, int d, int dv,
-                                   int flags, int page_size, long long cache_slots, void* q_out, void* k_cache,
-                                   void* v_cache, int* err, cudaStream_t stream) {
+                                   int flags, int maps, float rot_gain, int page_size, long long cache_slots,
+                                   void* q_out, void* k_cache, void* v_cache, int* err, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (nh <= 0 || nkv <= 0 || d <= 0 || dv <= 0 || d > MAX_VEC || dv > MAX_VEC || rot_dims < 0 || rot_dims > d ||
-      (rot_dims & 1) || page_size <= 0 || ((flags & PREP_VALUES_ARE_KEYS) && dv != d))
+      (rot_dims & 1) || page_size <= 0 || ((flags & PREP_VALUES_ARE_KEYS) && (dv != d || maps != 1)) || maps < 1 ||
+      nh % maps != 0)
     return B200_BAD_SIZE;
-  const long long work = static_cast<long long>(tokens) * (nh + 2 * nkv);
+  const long long work = static_cast<long long>(tokens) * (nh + nkv * maps + nkv);
   const unsigned blocks = static_cast<unsigned>((work + WARPS - 1) / WARPS);
   if (dtype == B200_F32)
     return b200_launch(heads_prepare_kernel<float>, dim3(blocks), dim3(WARPS * 32), 0, stream, 0,
         static_cast<const float*>(x), in_stride, bias, q_w, k_w, eps, inv_freq, rot_dims, interleaved, positions, slots,
-        tokens, nh, nkv, d, dv, flags, page_size, cache_slots, static_cast<float*>(q_out), static_cast<float*>(k_cache),
+        tokens, nh, nkv, d, dv, flags, maps, rot_gain, page_size, cache_slots, static_cast<float*>(q_out), static_cast<float*>(k_cache),
         static_cast<float*>(v_cache), err);
   else if (dtype == B200_BF16)
     return b200_launch(heads_prepare_kernel<__nv_bfloat16>, dim3(blocks), dim3(WARPS * 32), 0, stream, 0,
         static_cast<const __nv_bfloat16*>(x), in_stride, bias, q_w, k_w, eps, inv_freq, rot_dims, interleaved,
-        positions, slots, tokens, nh, nkv, d, dv, flags, page_size, cache_slots, static_cast<__nv_bfloat16*>(q_out),
+        positions, slots, tokens, nh, nkv, d, dv, flags, maps, rot_gain, page_size, cache_slots, static_cast<__nv_bfloat16*>(q_out),
         static_cast<__nv_bfloat16*>(k_cache), static_cast<__nv_bfloat16*>(v_cache), err);
   else
     return B200_BAD_DTYPE;

@@ -41,13 +41,22 @@ __device__ __forceinline__ float warp_max(float v) {
   return v;
 }
 
-// What joins a gate projection to its up projection in the products that do it as their epilogue: silu(g), or
-// gelu_tanh(g) in a build with GLU_GELU_TANH.
+// What joins a gate projection to its up projection in the products that do it as their epilogue: silu(g) u, gelu_tanh(g) u
+// in a build with GLU_GELU_TANH, g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit) and u' = clamp(u, -limit, limit) in
+// a build with GLU_CLAMPED_SWISH (the other builds do not read limit and alpha).
 __device__ __forceinline__ float glu_gate(float g) {
 #ifdef GLU_GELU_TANH
   return 0.5f * g * (1.0f + tanhf(0.79788456080286535588f * (g + 0.044715f * g * g * g)));
 #else
   return g / (1.0f + expf(-g));
+#endif
+}
+__device__ __forceinline__ float glu_product(float g, float u, float limit, float alpha) {
+#ifdef GLU_CLAMPED_SWISH
+  g = fminf(g, limit);
+  return g / (1.0f + expf(-alpha * g)) * (fminf(fmaxf(u, -limit), limit) + 1.0f);
+#else
+  return glu_gate(g) * u;
 #endif
 }
 

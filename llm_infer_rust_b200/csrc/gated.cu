@@ -324,6 +324,45 @@ B200_EXPORT int b200_tanh_cap(float* z, long long n, float cap, cudaStream_t str
   return b200_check_launch();
 }
 
+// ------------------------------------------------------------------ the difference of two attention maps
+// a [tokens, 2 heads, dv]: a head's two outputs over the same values.  out[t][h] = o / sqrt(mean(o^2) + eps) * gain with
+// o = a[t][2h] - lambda a[t][2h + 1]; a warp a head, in float, rounded once.
+template <typename T>
+__global__ void __launch_bounds__(128)
+head_difference_kernel(T* __restrict__ out, const T* __restrict__ a, float lambda, float gain, float eps, long long heads,
+                       int dv) {
+  pdl_launch_dependents();                          // the kernel after this one may be scheduled; it waits before it reads
+  pdl_wait();                                        // what this kernel reads belongs to the kernels before it
+  const long long h = static_cast<long long>(blockIdx.x) * 4 + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (h >= heads) return;
+  const T* first = a + 2 * h * dv;
+  const T* second = first + dv;
+  T* dst = out + h * dv;
+  float ss = 0.0f;
+  for (int c = lane; c < dv; c += 32) {
+    const float o = fmaf(-lambda, to_f32<T>(second[c]), to_f32<T>(first[c]));
+    ss = fmaf(o, o, ss);
+  }
+  const float r = gain / sqrtf(warp_sum(ss) / static_cast<float>(dv) + eps);
+  for (int c = lane; c < dv; c += 32) dst[c] = from_f32<T>(fmaf(-lambda, to_f32<T>(second[c]), to_f32<T>(first[c])) * r);
+}
+
+// heads: of all tokens together.
+B200_EXPORT int b200_head_difference(void* out, const void* a, float lambda, float gain, float eps, long long heads, int dv,
+                                     int dtype, cudaStream_t stream) {
+  if (heads <= 0) return 0;
+  if (dv <= 0) return B200_BAD_SIZE;
+  const dim3 grid(static_cast<unsigned>((heads + 3) / 4));
+  if (dtype == B200_F32)
+    return b200_launch(head_difference_kernel<float>, grid, dim3(128), 0, stream, 0, static_cast<float*>(out),
+                       static_cast<const float*>(a), lambda, gain, eps, heads, dv);
+  if (dtype == B200_BF16)
+    return b200_launch(head_difference_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, 0,
+                       static_cast<__nv_bfloat16*>(out), static_cast<const __nv_bfloat16*>(a), lambda, gain, eps, heads, dv);
+  return B200_BAD_DTYPE;
+}
+
 // ------------------------------------------------------------------ gate and up joined; an activation times a table row
 // out[t][c] = glu(gate_up[t][c], gate_up[t][ff + c]).  kind 0: silu(g) u.  kind 1: g' sigmoid(alpha g') (u' + 1) with
 // g' = min(g, limit), u' = clamp(u, -limit, limit).  kind 2: gelu_tanh(g) u.  Computed in float, rounded once.

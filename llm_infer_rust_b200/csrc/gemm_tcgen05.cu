@@ -92,7 +92,7 @@ __device__ __forceinline__ void mbar_arrive(uint64_t* bar) {
 // so the epilogue of one tile runs under the MMAs of the next (acc_full / acc_empty hand them over).
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap amap, const __grid_constant__ CUtensorMap wmap,
-                    bf16* __restrict__ out, int M, int N, int K, int mode, int* err) {
+                    bf16* __restrict__ out, int M, int N, int K, int mode, float glu_limit, float glu_alpha, int* err) {
   extern __shared__ unsigned char smem_raw[];
   unsigned char* ring = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint64_t* full = reinterpret_cast<uint64_t*>(ring + STAGES * STAGE_BYTES);
@@ -214,7 +214,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap amap, const __grid_const
             for (int e = 0; e < 32; ++e) {
               const float gate = __bfloat162float(__float2bfloat16_rn(g[e]));
               const float up = __bfloat162float(__float2bfloat16_rn(u[e]));
-              r[e] = __float2bfloat16_rn(glu_gate(gate) * up);
+              r[e] = __float2bfloat16_rn(glu_product(gate, up, glu_limit, glu_alpha));
             }
             if (col0 + 32 <= half && (half % 8) == 0) {
 #pragma unroll
@@ -271,10 +271,11 @@ B200_EXPORT int b200_gemm_tensor_map(void* out_map, const void* matrix, long lon
   return 0;
 }
 
-// out = a . w^T (mode 0: [m, n]) or silu(a . gate^T) * (a . up^T) (mode 1: w = [gate; up], out [m, n / 2]).
+// out = a . w^T (mode 0: [m, n]) or silu(a . gate^T) * (a . up^T) (mode 1: w = [gate; up], out [m, n / 2]; in a build with
+// another gate, see glu_product, that one).
 // `a_map`, `w_map`: descriptors of b200_gemm_tensor_map for a [m, k] and w [n, k].
-B200_EXPORT int b200_gemm_tcgen05(const void* a_map, const void* w_map, void* out, int m, int n, int k, int mode, int* err,
-                                  cudaStream_t stream) {
+B200_EXPORT int b200_gemm_tcgen05(const void* a_map, const void* w_map, void* out, int m, int n, int k, int mode,
+                                  float glu_limit, float glu_alpha, int* err, cudaStream_t stream) {
   if (m <= 0 || n <= 0) return 0;
   if (k <= 0 || k % 8 != 0 || (mode != GEMM_PLAIN && mode != GEMM_SWIGLU)) return B200_BAD_SIZE;
   if (mode == GEMM_SWIGLU && n % 2 != 0) return B200_BAD_SIZE;
@@ -296,5 +297,5 @@ B200_EXPORT int b200_gemm_tcgen05(const void* a_map, const void* w_map, void* ou
   if (cudaGetDevice(&device) == cudaSuccess) cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device);
   const int grid = m_tiles * n_tiles < sms ? m_tiles * n_tiles : sms;       // persistent: at most one CTA per SM
   return b200_launch(gemm_tcgen05_kernel, dim3(grid), dim3(THREADS), smem, stream, 0, amap, wmap,
-                     static_cast<bf16*>(out), m, n, k, mode, err);
+                     static_cast<bf16*>(out), m, n, k, mode, glu_limit, glu_alpha, err);
 }

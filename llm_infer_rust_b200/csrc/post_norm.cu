@@ -9,6 +9,10 @@
 //                 column, or none (an output projection's bias, added here in float instead of in a kernel of its own).
 //   norm_add_pair the same update with the mean of two normed branches in place of y: y = (R(a; wa) + R(b; wb)) / 2, R the
 //                 RMS norm of a branch with its own weights (a layer of two mixers side by side)
+//   residual_sum  the other arrangement, whose norm sits on a sublayer's INPUT and is handed the sum of the layer before:
+//                 x <- x + m (y + bias + f), y the mixer's output (or the mean of two normed branches, as above) and f the
+//                 feed-forward's, both of the same input; then out = R(x) w or, without a weight, x itself, rounded once
+//                 (rows of `out` may lie further apart than they are wide).
 //   norm_rows     out[r] = N(x[rows[r]]) without the add (the model's last norm, at the rows whose logits are wanted).
 //
 // One block a token; a row's sum of squares is added in an order fixed by the thread layout, so a token's result does
@@ -171,6 +175,100 @@ norm_add_pair_kernel(float* __restrict__ x, const TY* __restrict__ a, const TY* 
   }
 }
 
+// Shared memory: width floats.  rows (null: every token): out[r] is made of token rows[r].
+template <typename TY>
+struct ResidualTerms {
+  const TY* y;               // the mixer's output, or null
+  const TY* b;               // the second branch: y and b are then normed with wa and wb and their mean taken
+  const TY* f;               // the feed-forward's output, or null
+  const float* bias;         // per column, on y (without a second branch), or null
+  const float* wa;
+  const float* wb;
+};
+
+template <typename TY, typename TO, int VEC>
+__global__ void __launch_bounds__(PN_MAX_THREADS)
+residual_sum_kernel(float* __restrict__ x, ResidualTerms<TY> in, float mult, const float* __restrict__ w, float eps,
+                    const int* __restrict__ rows, TO* __restrict__ out, size_t out_stride, int store, int width) {
+  pdl_launch_dependents();                          // the kernel after this one may be scheduled; it waits before it reads
+  pdl_wait();                                        // what this kernel reads belongs to the kernels before it
+  __shared__ float scratch[33];
+  extern __shared__ float row[];                     // x after the sum
+  const size_t t = rows != nullptr ? static_cast<size_t>(rows[blockIdx.x]) : blockIdx.x;
+  float* xr = x + t * width;
+  auto load = [](const TY* p, float (&v)[VEC]) {
+    if constexpr (VEC == 4) load_floats<TY, 4>(p, v);
+    else v[0] = to_f32<TY>(*p);
+  };
+  auto load_f = [](const float* p, float (&v)[VEC]) {
+    if constexpr (VEC == 4) load_floats<float, 4>(p, v);
+    else v[0] = *p;
+  };
+  float fa = 0.0f, fb = 0.0f;
+  if (in.b != nullptr) {
+    float sa = 0.0f, sb = 0.0f;
+    for (int c = VEC * threadIdx.x; c < width; c += VEC * blockDim.x) {
+      float u[VEC], v[VEC];
+      load(in.y + t * width + c, u);
+      load(in.b + t * width + c, v);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) { sa = fmaf(u[i], u[i], sa); sb = fmaf(v[i], v[i], sb); }
+    }
+    fa = 0.5f / sqrtf(block_sum(sa, scratch) / static_cast<float>(width) + eps);
+    fb = 0.5f / sqrtf(block_sum(sb, scratch) / static_cast<float>(width) + eps);
+  }
+  float ss = 0.0f;
+#pragma unroll 2
+  for (int c = VEC * threadIdx.x; c < width; c += VEC * blockDim.x) {
+    float s[VEC] = {}, v[VEC], g[VEC];
+    if (in.y != nullptr) {
+      load(in.y + t * width + c, s);
+      if (in.b != nullptr) {
+        float h[VEC];
+        load(in.b + t * width + c, v);
+        load_f(in.wa + c, g);
+        load_f(in.wb + c, h);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) s[i] = s[i] * fa * g[i] + v[i] * fb * h[i];
+      } else if (in.bias != nullptr) {
+        load_f(in.bias + c, g);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) s[i] += g[i];
+      }
+    }
+    if (in.f != nullptr) {
+      load(in.f + t * width + c, v);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) s[i] += v[i];
+    }
+    load_f(xr + c, v);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) {
+      v[i] = fmaf(mult, s[i], v[i]);
+      ss = fmaf(v[i], v[i], ss);
+    }
+    if constexpr (VEC == 4) {
+      const float4 sum = make_float4(v[0], v[1], v[2], v[3]);
+      *reinterpret_cast<float4*>(row + c) = sum;
+      if (store) *reinterpret_cast<float4*>(xr + c) = sum;
+    } else {
+      row[c] = v[0];
+      if (store) xr[c] = v[0];
+    }
+  }
+  if (out == nullptr) return;
+  float r = 1.0f;
+  if (w != nullptr) r = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(width) + eps);
+  for (int c = VEC * threadIdx.x; c < width; c += VEC * blockDim.x) {     // (a thread reads what it wrote itself)
+    float v[VEC];
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = w != nullptr ? row[c + i] * r * w[c + i] : row[c + i];
+    TO* dst = out + blockIdx.x * out_stride + c;
+    if constexpr (VEC == 4) store4<TO>(dst, v[0], v[1], v[2], v[3]);
+    else *dst = from_f32<TO>(v[0]);
+  }
+}
+
 template <typename TO, bool CENTER>
 __global__ void __launch_bounds__(PN_THREADS)
 norm_rows_kernel(TO* __restrict__ out, const float* __restrict__ x, const int* __restrict__ rows,
@@ -252,6 +350,45 @@ B200_EXPORT int b200_norm_add_pair(float* x, const void* a, const void* b, int y
                                    cudaStream_t stream) {
   if (a == nullptr || b == nullptr) return B200_BAD_SIZE;
   return run_norm_add(x, a, b, y_dtype, nullptr, wa, wb, w, eps, center, cast_out, out_dtype, tokens, width, stream);
+}
+
+// x [.., width] float.  y, b, f: dtype y_dtype, any of them null (b only with y, wa and wb); w null: no norm.  n: rows of
+// out (and of `rows`); store 0: x stays as it is.
+B200_EXPORT int b200_residual_sum(float* x, const void* y, const void* b, const void* f, int y_dtype, const float* bias,
+                                  const float* wa, const float* wb, float mult, const float* w, float eps, const int* rows,
+                                  void* out, int out_dtype, int out_stride, int store, int n, int width,
+                                  cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (width <= 0 || width * sizeof(float) > 200 * 1024 || (b != nullptr && (y == nullptr || wa == nullptr || wb == nullptr)))
+    return B200_BAD_SIZE;
+  if (out != nullptr && out_stride < width) return B200_BAD_SIZE;
+  const size_t smem = static_cast<size_t>(width) * sizeof(float);
+  const int threads = n <= 64 ? min(PN_MAX_THREADS, max(PN_THREADS, (width / 4 + 31) / 32 * 32)) : PN_THREADS;
+  const bool vec = width % 4 == 0 && out_stride % 4 == 0 && reinterpret_cast<uintptr_t>(out) % 16 == 0;
+#define B200_RESIDUAL(TY, TO, V)                                                                                     \
+  do {                                                                                                               \
+    const ResidualTerms<TY> in = {static_cast<const TY*>(y), static_cast<const TY*>(b), static_cast<const TY*>(f),   \
+                                  bias, wa, wb};                                                                     \
+    if (smem > 48 * 1024) {                                                                                          \
+      cudaError_t e = cudaFuncSetAttribute(residual_sum_kernel<TY, TO, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+                                           static_cast<int>(smem));                                                  \
+      if (e != cudaSuccess) return static_cast<int>(e);                                                              \
+    }                                                                                                                \
+    return b200_launch(residual_sum_kernel<TY, TO, V>, dim3(n), dim3(threads), smem, stream, 0, x, in, mult, w, eps,  \
+                       rows, static_cast<TO*>(out), static_cast<size_t>(out_stride), store, width);                  \
+  } while (0)
+#define B200_RESIDUAL_V(TY, TO)        \
+  do {                                 \
+    if (vec) B200_RESIDUAL(TY, TO, 4); \
+    B200_RESIDUAL(TY, TO, 1);          \
+  } while (0)
+  if (y_dtype == B200_F32 && out_dtype == B200_F32) B200_RESIDUAL_V(float, float);
+  if (y_dtype == B200_F32 && out_dtype == B200_BF16) B200_RESIDUAL_V(float, __nv_bfloat16);
+  if (y_dtype == B200_BF16 && out_dtype == B200_F32) B200_RESIDUAL_V(__nv_bfloat16, float);
+  if (y_dtype == B200_BF16 && out_dtype == B200_BF16) B200_RESIDUAL_V(__nv_bfloat16, __nv_bfloat16);
+#undef B200_RESIDUAL_V
+#undef B200_RESIDUAL
+  return B200_BAD_DTYPE;
 }
 
 B200_EXPORT int b200_norm_rows(void* out, int out_dtype, const float* x, const int* rows, const float* w, float eps, int center,

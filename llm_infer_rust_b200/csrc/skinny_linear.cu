@@ -98,6 +98,7 @@ struct SkinnyParams {
   const float* inv_freq;    // [rot_dim / 2]: the angle of pair i is position * inv_freq[i], its cosine and sine taken here
                             // (instead of cos_table / sin_table; any position)
   int qkv_flags;            // QKV_PLAIN_NORM | QKV_NORM_AFTER_ROTATION | QKV_VALUES_ARE_KEYS
+  float glu_limit, glu_alpha;   // SWIGLU in the build with GLU_CLAMPED_SWISH
 };
 // QKV_PLAIN_NORM: q and k heads are normed without weights (x / sqrt(mean(x^2) + qk_eps)); QKV_NORM_AFTER_ROTATION: the
 // norm follows the rotation; QKV_VALUES_ARE_KEYS: the weight holds q and k heads only (N = (nh + nkv) * d) and a key
@@ -714,7 +715,7 @@ skinny_linear_kernel(const __grid_constant__ CUtensorMap wmap, const SkinnyParam
       const float gf[4] = {gate4.x, gate4.y, gate4.z, gate4.w}, uf[4] = {up4.x, up4.y, up4.z, up4.w};
       __align__(8) bf16 h[4];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) h[e] = __float2bfloat16_rn(glu_gate(gf[e]) * uf[e]);
+      for (int e = 0; e < 4; ++e) h[e] = __float2bfloat16_rn(glu_product(gf[e], uf[e], p.glu_limit, p.glu_alpha));
       const size_t at = static_cast<size_t>(m) * inter + col;
       if (whole) *reinterpret_cast<uint2*>(static_cast<bf16*>(p.out) + at) = *reinterpret_cast<uint2*>(h);
       else

@@ -77,6 +77,7 @@ struct StreamParams {
   int groups, tiles;        // (filled by the launcher: groups of KS warps a CTA, tiles of the product)
   int xd;                   // the rows of x come with the weights' copies instead of waiting in shared memory: 1 yes, 0 no, -1 where they do not fit
   int pair;                 // CTAs are launched as clusters of two that stage half of the rows of x each (1 yes, 0 no, -1 the launcher's choice)
+  float glu_limit, glu_alpha;   // SWIGLU in the build with GLU_CLAMPED_SWISH
 };
 
 __device__ __forceinline__ void mma_16816(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0,
@@ -448,7 +449,7 @@ __global__ void __launch_bounds__(MAX_THREADS, 1) stream_linear_kernel(const Str
         const int m = i / COLS, rr = i - m * COLS, col = tile * COLS + rr;
         if (col >= inter) continue;
         const float gate = total_of(rr, m), up = total_of(COLS + rr, m);
-        static_cast<bf16*>(p.out)[static_cast<size_t>(m) * inter + col] = __float2bfloat16_rn(glu_gate(gate) * up);
+        static_cast<bf16*>(p.out)[static_cast<size_t>(m) * inter + col] = __float2bfloat16_rn(glu_product(gate, up, p.glu_limit, p.glu_alpha));
       }
     }
     group_barrier(grp, gthreads);       // the sums are read: the next tile may overwrite them

@@ -550,7 +550,8 @@ class _SkinnyParams(ctypes.Structure):
                 ("slots", ctypes.c_void_p), ("k_cache", ctypes.c_void_p), ("v_cache", ctypes.c_void_p),
                 ("err", ctypes.c_void_p), ("post_residual", ctypes.c_void_p), ("post_sum_out", ctypes.c_void_p),
                 ("post_stats", ctypes.c_void_p), ("stats_in", ctypes.c_void_p), ("stats_tiles", ctypes.c_int),
-                ("trace", ctypes.c_void_p), ("inv_freq", ctypes.c_void_p), ("qkv_flags", ctypes.c_int)]
+                ("trace", ctypes.c_void_p), ("inv_freq", ctypes.c_void_p), ("qkv_flags", ctypes.c_int),
+                ("glu_limit", ctypes.c_float), ("glu_alpha", ctypes.c_float)]
 
 
 # For tuning: an int64 tensor [4096, 32] on the device; the first thread of every CTA of the next single-product
@@ -598,7 +599,7 @@ def _sm_count(device) -> int:
 
 
 # The gate's activation in a fused product: builds of their own, so that the dense models' stay as they are.
-_GLU_DEFINES = {"silu": {}, "gelu_tanh": {"GLU_GELU_TANH": 1}}
+_GLU_DEFINES = {"silu": {}, "gelu_tanh": {"GLU_GELU_TANH": 1}, "clamped_swish": {"GLU_CLAMPED_SWISH": 1}}
 
 
 def _skinny(qkv_forms: bool = False, glu: str = "silu"):
@@ -674,7 +675,7 @@ def graph_capture(graph: "torch.cuda.CUDAGraph"):
 
 def skinny_linear(x, weight: torch.Tensor, mode: int = EPI_PLAIN_BF16, x_rows: Optional[torch.Tensor] = None,
                   qkv: Optional[dict] = None, out: Optional[torch.Tensor] = None, norm_after=None,
-                  stats=None, glu: str = "silu") -> torch.Tensor:
+                  stats=None, glu: str = "silu", limit: float = 0.0, alpha: float = 1.0) -> torch.Tensor:
     """epilogue(prologue(x) . weight^T) for at most 16 rows, in one kernel.
 
     ``out``: the tensor to fill (PLAIN and SWIGLU; made here when None).  ``norm_after`` = (residual, sum_out,
@@ -722,6 +723,7 @@ def skinny_linear(x, weight: torch.Tensor, mode: int = EPI_PLAIN_BF16, x_rows: O
         if pending.weight.numel() != k or pending.weight.dtype not in (torch.float32, torch.bfloat16):
             raise KernelError("the norm weight must have K elements, bfloat16 or float32")
     P.M, P.N, P.K, P.mode = m, n, k, mode
+    P.glu_limit, P.glu_alpha = float(limit), float(alpha)
     dev = src.device
     P.err = error_word(dev).data_ptr()
     P.trace = 0 if skinny_trace is None else skinny_trace.data_ptr()
@@ -787,7 +789,7 @@ class _StreamParams(ctypes.Structure):
                 ("K", ctypes.c_int), ("mode", ctypes.c_int), ("out", ctypes.c_void_p),
                 ("post_residual", ctypes.c_void_p), ("post_sum_out", ctypes.c_void_p), ("post_stats", ctypes.c_void_p),
                 ("rw", ctypes.c_int), ("ks", ctypes.c_int), ("groups", ctypes.c_int), ("tiles", ctypes.c_int),
-                ("xd", ctypes.c_int), ("pair", ctypes.c_int)]
+                ("xd", ctypes.c_int), ("pair", ctypes.c_int), ("glu_limit", ctypes.c_float), ("glu_alpha", ctypes.c_float)]
 
 
 def _stream_lib(glu: str = "silu"):
@@ -848,7 +850,8 @@ def stream_tile_cols(mode: int, m: int, n: int, k: int, norm: bool) -> int:
 
 def stream_linear(x, weight: torch.Tensor, mode: int = EPI_PLAIN_BF16, x_rows: Optional[torch.Tensor] = None,
                   out: Optional[torch.Tensor] = None, norm_after=None, rw: int = 0, ks: int = 0,
-                  xd: int = -1, pair: Optional[int] = None, glu: str = "silu") -> torch.Tensor:
+                  xd: int = -1, pair: Optional[int] = None, glu: str = "silu", limit: float = 0.0,
+                  alpha: float = 1.0) -> torch.Tensor:
     """epilogue(prologue(x) . weight^T) for at most 16 rows and a large weight (csrc/stream_linear.cu).
 
     ``x``: a bfloat16 tensor [rows, K] or a ``PendingNorm`` (with or without a residual); ``mode``: EPI_PLAIN_BF16,
@@ -884,6 +887,7 @@ def stream_linear(x, weight: torch.Tensor, mode: int = EPI_PLAIN_BF16, x_rows: O
             P.residual = res.data_ptr()
             P.residual_out = 0 if pending.residual_out is None else pending.residual_out.data_ptr()
     P.w, P.M, P.N, P.K, P.mode = weight.data_ptr(), m, n, k, mode
+    P.glu_limit, P.glu_alpha = float(limit), float(alpha)
     if out is None:
         out = _few_row_out(m, n, mode, src.device)
     if norm_after is not None:
@@ -1115,13 +1119,14 @@ def few_row_linear(x, weight: torch.Tensor, mode: int = EPI_PLAIN_BF16, x_rows: 
     return _single_lazy(x, weight, mode, x_rows, qkv, lazy)
 
 
-def few_row_glu(x: torch.Tensor, weight: torch.Tensor, activation: str = "silu") -> torch.Tensor:
-    """act(gate x) * (up x) for few rows of a plain tensor, weight = [gate rows; up rows], in one kernel (where
-    ``few_row_takes`` an EPI_SWIGLU product on the single route): ``activation`` silu or gelu_tanh."""
+def few_row_glu(x: torch.Tensor, weight: torch.Tensor, activation: str = "silu", limit: float = 0.0,
+                alpha: float = 1.0) -> torch.Tensor:
+    """glu(gate x, up x) for few rows of a plain tensor, weight = [gate rows; up rows], in one kernel (where
+    ``few_row_takes`` an EPI_SWIGLU product on the single route), with the forms of ``glu_columns``."""
     flush_chain()
     if stream_takes(x.shape[0], weight, x.dtype, EPI_SWIGLU, False):
-        return stream_linear(x, weight, EPI_SWIGLU, glu=activation)
-    return skinny_linear(x, weight, EPI_SWIGLU, glu=activation)
+        return stream_linear(x, weight, EPI_SWIGLU, glu=activation, limit=limit, alpha=alpha)
+    return skinny_linear(x, weight, EPI_SWIGLU, glu=activation, limit=limit, alpha=alpha)
 
 
 def _chain_append(pending, src, rows_t, m, weight, mode, qkv) -> torch.Tensor:
@@ -1287,10 +1292,11 @@ def gemm_tc_pays(x: torch.Tensor, weight: torch.Tensor, mode: int = GEMM_PLAIN) 
     return x.shape[1] >= 2048 and tiles >= 4 * _sm_count(x.device)
 
 
-def gemm_tc(x: torch.Tensor, weight: torch.Tensor, mode: int = GEMM_PLAIN, glu: str = "silu") -> torch.Tensor:
+def gemm_tc(x: torch.Tensor, weight: torch.Tensor, mode: int = GEMM_PLAIN, glu: str = "silu", limit: float = 0.0,
+            alpha: float = 1.0) -> torch.Tensor:
     """x . weight^T on the tcgen05 tensor cores (TMA-fed, float sums in tensor memory), bfloat16 out.
-    ``GEMM_SWIGLU``: weight = [gate rows; up rows]; the result is silu(x . gate^T) * (x . up^T) (``glu`` "gelu_tanh":
-    that activation)."""
+    ``GEMM_SWIGLU``: weight = [gate rows; up rows]; the result is silu(x . gate^T) * (x . up^T) (``glu``: another of
+    the forms of ``glu_columns``)."""
     flush_chain()
     if not gemm_tc_ok(x, weight, mode):
         raise KernelError("the tcgen05 product takes contiguous bfloat16 [M, K] and [N, K] with K a multiple of 8")
@@ -1302,7 +1308,8 @@ def gemm_tc(x: torch.Tensor, weight: torch.Tensor, mode: int = GEMM_PLAIN, glu: 
     rc = lib.b200_gemm_tensor_map(a_map, _p(x), ctypes.c_longlong(m), ctypes.c_longlong(k))
     if rc != 0:
         raise KernelError(f"the TMA descriptor of the activations could not be made (code {rc})")
-    rc = lib.b200_gemm_tcgen05(a_map, _gemm_map(weight), _p(out), m, n, k, mode, _p(error_word(x.device)), _stream())
+    rc = lib.b200_gemm_tcgen05(a_map, _gemm_map(weight), _p(out), m, n, k, mode, ctypes.c_float(limit), ctypes.c_float(alpha),
+                               _p(error_word(x.device)), _stream())
     _ok(rc, "gemm_tcgen05")
     return out
 
@@ -1545,14 +1552,15 @@ def add_norm_taps_single(x: torch.Tensor, y: Optional[torch.Tensor], gain: torch
     return out
 
 
-def taps_state_update(x: torch.Tensor, taps: int, channels: int, state: torch.Tensor, ctx) -> None:
-    """The last ``taps - 1`` rows of x (first ``channels`` columns) of every row of the step become its state."""
+def taps_state_update(x: torch.Tensor, taps: int, channels: int, state: torch.Tensor, ctx, column: int = 0) -> None:
+    """The last ``taps - 1`` rows of x (``channels`` columns from ``column`` on) of every row of the step become its state."""
     if taps <= 1:
         return
     _cuda(x, state)
     _contig(x, state)
     _f32(state)
-    rc = _token_conv().b200_taps_state_update(_p(x), _code(x), x.shape[1], None, taps, channels, _p(state),
+    at = ctypes.c_void_p(x.data_ptr() + column * x.element_size())
+    rc = _token_conv().b200_taps_state_update(at, _code(x), x.shape[1], None, taps, channels, _p(state),
                                               _p(ctx.cu_q), _p(ctx.prefix_len), _p(ctx.state_slots), ctx.num_rows,
                                               0, _stream())
     _ok(rc, "taps_state_update")
@@ -1642,7 +1650,8 @@ class _LinearStateShape(ctypes.Structure):
     """Mirror of ``LinearStateShape`` in csrc/linear_state.cu (same order, native alignment)."""
     _fields_ = [("heads", ctypes.c_int), ("kv_heads", ctypes.c_int), ("d", ctypes.c_int), ("dv", ctypes.c_int),
                 ("beta_column", ctypes.c_int), ("silu", ctypes.c_int), ("unit_eps", ctypes.c_float),
-                ("q_scale", ctypes.c_float), ("decay_kind", ctypes.c_int), ("inv_tau", ctypes.c_float),
+                ("q_scale", ctypes.c_float), ("decay_kind", ctypes.c_int), ("decay_column", ctypes.c_int),
+                ("inv_tau", ctypes.c_float),
                 ("decay_bias", ctypes.c_void_p), ("a_log", ctypes.c_void_p)]
 
 
@@ -1652,6 +1661,16 @@ class _StateDecodeParams(ctypes.Structure):
                 ("g_column", ctypes.c_int), ("g_rank", ctypes.c_int), ("gate_kind", ctypes.c_int),
                 ("norm_w", ctypes.c_void_p), ("eps", ctypes.c_float), ("own_conv", ctypes.c_int),
                 ("stage", ctypes.c_int)]
+
+
+def state_head_blocks(head_dim: int) -> int:
+    """Blocks of 32 rows of a state for which the scan with one decay a head is compiled."""
+    return next(n for n in (1, 2, 3, 4, 6, 8, 16) if 32 * n >= head_dim)
+
+
+def _state_scan(form: "LinearStateForm"):
+    """The scan of a form: the build for decays per key channel, or one per range of head sizes for one decay a head."""
+    return load_cuda_library("state_scan.cu", {"STATE_HEAD_BLOCKS": state_head_blocks(form.d)} if form.head_decay else None)
 
 
 def _linear_state():
@@ -1665,42 +1684,48 @@ def _linear_state():
 
 
 class LinearStateForm:
-    """What a linear-attention layer with per-channel decays does between its projections (csrc/linear_state.cu):
+    """What a linear-attention layer with decays per key channel or per head does between its projections
+    (csrc/linear_state.cu, csrc/state_scan.cu):
 
     ``decay`` "logistic": sigmoid(z + bias)^(1 / tau); "softplus": exp(-exp(a_log) softplus(z + bias)).
     ``beta_column``: column of the packed row where one number a head begins whose sigmoid is the delta rule's step (None:
-    no delta rule).  ``silu``: on q, k, v behind the convolution.  ``unit_eps``: q and k become unit vectors (None: not).
+    no delta rule).  ``decay_column``: column where one pre-activation a head begins (one decay a head, ``decay_bias`` then
+    [heads]; None: decays per key channel, whose pre-activations are given apart).  ``silu``: on q, k, v behind the convolution.  ``unit_eps``: q and k become unit vectors (None: not).
     """
 
     def __init__(self, heads: int, kv_heads: int, head_dim: int, v_head_dim: int, q_scale: float = 1.0,
                  decay: str = "logistic", tau: float = 1.0, decay_bias: Optional[torch.Tensor] = None,
                  a_log: Optional[torch.Tensor] = None, beta_column: Optional[int] = None, silu: bool = False,
-                 unit_eps: Optional[float] = None):
+                 unit_eps: Optional[float] = None, decay_column: Optional[int] = None):
         if decay not in ("logistic", "softplus"):
             raise KernelError(f"decay {decay!r} is refused: logistic or softplus")
         _cuda(decay_bias, a_log)
         _contig(decay_bias, a_log)
         _f32(decay_bias, a_log)
-        if (decay_bias is not None and decay_bias.numel() != heads * head_dim) or (a_log is not None and a_log.numel() != heads) \
+        self.head_decay = decay_column is not None
+        if (decay_bias is not None and decay_bias.numel() != (heads if self.head_decay else heads * head_dim)) or (a_log is not None and a_log.numel() != heads) \
                 or (decay == "softplus") != (a_log is not None):
-            raise KernelError("the decay's bias [heads * head_dim] or rates [heads] do not fit")
+            raise KernelError("the decay's bias [heads * head_dim] ([heads] for one decay a head) or rates [heads] do not fit")
         self.heads, self.kv_heads, self.d, self.dv = heads, kv_heads, head_dim, v_head_dim
         self.channels = 2 * kv_heads * head_dim + heads * v_head_dim
         self.delta = beta_column is not None
         self.keep = (decay_bias, a_log)
         self.shape = _LinearStateShape(heads, kv_heads, head_dim, v_head_dim, -1 if beta_column is None else int(beta_column),
                                        int(bool(silu)), float(unit_eps or 0.0), float(q_scale),
-                                       int(decay == "softplus"), 1.0 / float(tau),
+                                       int(decay == "softplus"), -1 if decay_column is None else int(decay_column),
+                                       1.0 / float(tau),
                                        decay_bias.data_ptr() if decay_bias is not None else None,
                                        a_log.data_ptr() if a_log is not None else None)
 
 
-def _state_checks(form: LinearStateForm, x, conv, conv_state, state) -> int:
+def _state_checks(form: LinearStateForm, x, conv, conv_state, state, column: int = 0) -> int:
     _cuda(x, conv, conv_state, state)
     _contig(x, conv, conv_state, state)
     _f32(conv, conv_state, state)
     taps = 0 if conv is None else conv.shape[1]
-    if x.shape[1] < form.channels or (form.delta and form.shape.beta_column + form.heads > x.shape[1]) or \
+    width = x.shape[1] - column                        # (a form's columns count from ``column`` on)
+    if column < 0 or width < form.channels or (form.delta and form.shape.beta_column + form.heads > width) or \
+            (form.head_decay and form.shape.decay_column + form.heads > width) or \
             tuple(state.shape[1:]) != (form.heads, form.d, form.dv) or \
             (conv is not None and conv.shape[0] != form.channels) or \
             (taps > 1 and (conv_state is None or tuple(conv_state.shape[1:]) != (taps - 1, form.channels))):
@@ -1709,65 +1734,71 @@ def _state_checks(form: LinearStateForm, x, conv, conv_state, state) -> int:
 
 
 def state_decode(form: LinearStateForm, x: torch.Tensor, conv: Optional[torch.Tensor], conv_state: Optional[torch.Tensor],
-                 state: torch.Tensor, ctx, a2: torch.Tensor, a_column: int, norm: torch.Tensor, eps: float,
-                 gate_column: int, g2: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+                 state: torch.Tensor, ctx, a2: Optional[torch.Tensor], a_column: int, norm: torch.Tensor, eps: float,
+                 gate_column: int, g2: Optional[torch.Tensor] = None, column: int = 0) -> Optional[torch.Tensor]:
     """A step whose rows all bring one token: the layer between its packed projection ``x`` and its output projection in one
     kernel (convolution, decay, recurrence, per-head norm, gate), [tokens, heads * v_head_dim] in x's dtype; the states are
-    brought up to date.  ``a2`` [heads * d, rank] meets x's columns from ``a_column`` on.  Gate: with ``g2``
+    brought up to date.  ``a2`` [heads * d, rank] meets x's columns from ``a_column`` on (None: the form has one decay a
+    head).  All columns count from ``column`` of x on.  Gate: with ``g2``
     sigmoid(g2 x[gate_column ..]), else silu of the columns from ``gate_column`` on.  None: the step has longer rows or the
     sizes do not fit the kernel; the caller then runs the parts one by one."""
     if not _all_single(ctx):
         return None
-    taps = _state_checks(form, x, conv, conv_state, state)
+    taps = _state_checks(form, x, conv, conv_state, state, column)
+    width = x.shape[1] - column
     _cuda(a2, g2, norm)
     _contig(a2, g2, norm)
     _f32(norm)
-    if a2.dtype != x.dtype or a2.shape[0] != form.heads * form.d or a_column + a2.shape[1] > x.shape[1] or \
-            norm.numel() != form.dv or (g2 is not None and (g2.dtype != x.dtype or g2.shape[0] != form.heads * form.dv)) or \
-            gate_column + (g2.shape[1] if g2 is not None else form.heads * form.dv) > x.shape[1]:
+    if (a2 is None) != form.head_decay or norm.numel() != form.dv or (g2 is not None and (g2.dtype != x.dtype or g2.shape[0] != form.heads * form.dv)) or \
+            gate_column + (g2.shape[1] if g2 is not None else form.heads * form.dv) > width or \
+            (a2 is not None and (a2.dtype != x.dtype or a2.shape[0] != form.heads * form.d or a_column + a2.shape[1] > width)):
         raise KernelError("state_decode: the low-rank products, the norm or the gate do not fit")
     out = torch.empty((x.shape[0], form.heads * form.dv), dtype=x.dtype, device=x.device)
     own = form.heads == form.kv_heads
-    params = _StateDecodeParams(a2.data_ptr(), g2.data_ptr() if g2 is not None else None, int(a_column), a2.shape[1],
+    params = _StateDecodeParams(a2.data_ptr() if a2 is not None else None, g2.data_ptr() if g2 is not None else None,
+                                int(a_column), a2.shape[1] if a2 is not None else 0,
                                 int(gate_column), g2.shape[1] if g2 is not None else 0, int(g2 is None), norm.data_ptr(),
                                 float(eps), int(own), 0)
+    at = ctypes.c_void_p(x.data_ptr() + column * x.element_size())
     rc = _linear_state().b200_state_decode(
-        _p(x), _code(x), x.shape[1], _p(conv), taps, _p(conv_state), _p(ctx.row_of_token), _p(ctx.cu_q), _p(ctx.prefix_len),
+        at, _code(x), x.shape[1], _p(conv), taps, _p(conv_state), _p(ctx.row_of_token), _p(ctx.cu_q), _p(ctx.prefix_len),
         _p(ctx.state_slots), ctypes.byref(form.shape), ctypes.byref(params), _p(out), _p(state), x.shape[0], _stream())
     if rc == -2:
         return None
     _ok(rc, "state_decode")
     if taps > 1 and not own:
-        taps_state_update(x, taps, form.channels, conv_state, ctx)
+        taps_state_update(x, taps, form.channels, conv_state, ctx, column)
     return out
 
 
-def state_recurrence(form: LinearStateForm, x: torch.Tensor, z: torch.Tensor, conv: Optional[torch.Tensor],
-                     conv_state: Optional[torch.Tensor], state: torch.Tensor, ctx) -> torch.Tensor:
+def state_recurrence(form: LinearStateForm, x: torch.Tensor, z: Optional[torch.Tensor], conv: Optional[torch.Tensor],
+                     conv_state: Optional[torch.Tensor], state: torch.Tensor, ctx, column: int = 0) -> torch.Tensor:
     """The recurrence over a step's rows of any length: o [tokens, heads * v_head_dim] float32, the states brought up to
-    date.  ``z`` (float32 [tokens, heads * d]): the decays' pre-activations without bias."""
-    taps = _state_checks(form, x, conv, conv_state, state)
+    date.  ``z`` (float32 [tokens, heads * d]): the decays' pre-activations without bias (None: the form has one decay a
+    head, a column of x).  Columns of x count from ``column`` on."""
+    taps = _state_checks(form, x, conv, conv_state, state, column)
     _cuda(z)
     _contig(z)
     _f32(z)
     tokens, dev = x.shape[0], x.device
-    if tuple(z.shape) != (tokens, form.heads * form.d):
+    if (z is None) != form.head_decay or (z is not None and tuple(z.shape) != (tokens, form.heads * form.d)):
         raise KernelError("state_recurrence: one pre-activation for every head and key channel is needed")
     qf = torch.empty((2, tokens, form.kv_heads * form.d), dtype=torch.float32, device=dev)
     vf = torch.empty((tokens, form.heads * form.dv), dtype=torch.float32, device=dev)
-    gf = torch.empty((tokens, form.heads * form.d), dtype=torch.float32, device=dev)
+    gf = torch.empty((tokens, form.heads * (1 if form.head_decay else form.d)), dtype=torch.float32, device=dev)
     beta = torch.empty((tokens, form.heads), dtype=torch.float32, device=dev) if form.delta else None
     lib = _linear_state()
+    at = ctypes.c_void_p(x.data_ptr() + column * x.element_size())
     rc = lib.b200_state_prepare(
-        _p(x), _code(x), x.shape[1], _p(conv), taps, _p(conv_state), _p(ctx.row_of_token), _p(ctx.cu_q), _p(ctx.prefix_len),
+        at, _code(x), x.shape[1], _p(conv), taps, _p(conv_state), _p(ctx.row_of_token), _p(ctx.cu_q), _p(ctx.prefix_len),
         _p(ctx.state_slots), ctypes.byref(form.shape), _p(z), _p(qf[0]), _p(qf[1]), _p(vf), _p(gf), _p(beta), tokens, _stream())
     _ok(rc, "state_prepare")
     if taps > 1:
-        taps_state_update(x, taps, form.channels, conv_state, ctx)
+        taps_state_update(x, taps, form.channels, conv_state, ctx, column)
     o = torch.empty((tokens, form.heads * form.dv), dtype=torch.float32, device=dev)
-    rc = lib.b200_state_scan(_p(qf[0]), _p(qf[1]), _p(vf), _p(gf), _p(beta), _p(o), _p(state), _p(ctx.cu_q),
+    rc = _state_scan(form).b200_state_scan(_p(qf[0]), _p(qf[1]), _p(vf), _p(gf), _p(beta), _p(o), _p(state), _p(ctx.cu_q),
                              _p(ctx.prefix_len), _p(ctx.state_slots), ctx.num_rows, form.heads, form.kv_heads, form.d,
-                             form.dv, _stream())
+                             form.dv, int(form.head_decay), _stream())
     _ok(rc, "state_scan")
     return o
 
@@ -1959,23 +1990,33 @@ def heads_prepare(x: torch.Tensor, q_out: torch.Tensor, k_cache: torch.Tensor, v
                   head_dim: int, v_head_dim: int, bias: Optional[torch.Tensor] = None,
                   q_weight: Optional[torch.Tensor] = None, k_weight: Optional[torch.Tensor] = None, eps: float = 0.0,
                   inv_freq: Optional[torch.Tensor] = None, rot_dims: int = 0, interleaved: bool = True,
-                  plain_norm: bool = False, norm_after_rotation: bool = False, values_are_keys: bool = False) -> None:
+                  plain_norm: bool = False, norm_after_rotation: bool = False, values_are_keys: bool = False,
+                  maps: int = 1, rot_gain: float = 1.0) -> None:
     """q, k, v are the first columns of ``x``: optional bias (float32, one per column), optional per-head RMS norm
     of q and k (float32 weights over a head; ``plain_norm``: no weights, x / sqrt(mean(x^2) + eps)), optional rotation
     of the first ``rot_dims`` coordinates of every q and k head by position * inv_freq (pairs (2i, 2i+1) if
     ``interleaved`` else (i, i + rot_dims/2)); the norm precedes the rotation unless ``norm_after_rotation``; q to
     ``q_out``, k and v into the paged cache at ``slots`` (None: nothing is stored).  ``values_are_keys``: ``x`` holds
-    no v columns and a token's value is its key as projected (biased, neither normed nor rotated)."""
+    no v columns and a token's value is its key as projected (biased, neither normed nor rotated).  ``rot_gain``
+    multiplies cosines and sines.
+
+    ``maps`` M > 1: ``num_heads`` counts query VECTORS (M a head, side by side in ``x``) and every key head has M key
+    vectors; each is normed and rotated by itself.  A key head's vectors are one row M * head_dim wide of ``k_cache``, and
+    ``q_out`` [tokens, num_heads, M * head_dim] holds every query vector in its own map's columns with zeros beside it:
+    attention over keys of that width serves all maps with one fetch of keys and values."""
     _cuda(x, q_out, k_cache, v_cache, positions, slots, bias, q_weight, k_weight, inv_freq)
     _contig(x, q_out, k_cache, v_cache, positions, slots, bias, q_weight, k_weight, inv_freq)
     _f32(bias, q_weight, k_weight, inv_freq)
     if values_are_keys and v_head_dim != head_dim:
         raise KernelError("values that are the keys are as wide as the keys")
-    c = (num_heads + num_kv_heads) * head_dim + (0 if values_are_keys else num_kv_heads * v_head_dim)
+    c = (num_heads + num_kv_heads * maps) * head_dim + (0 if values_are_keys else num_kv_heads * v_head_dim)
     flags = (1 if plain_norm else 0) | (2 if norm_after_rotation else 0) | (4 if values_are_keys else 0)
     if x.shape[1] < c or q_out.dtype != x.dtype or k_cache.dtype != x.dtype or v_cache.dtype != x.dtype:
         raise KernelError("heads_prepare: the projection is too narrow, or q, cache and projection differ in dtype")
-    if tuple(k_cache.shape[1:]) != (num_kv_heads, k_cache.shape[2], head_dim) or \
+    if maps < 1 or num_heads % maps or (maps > 1 and values_are_keys) or \
+            q_out.numel() != x.shape[0] * num_heads * maps * head_dim:
+        raise KernelError("heads_prepare: q_out or the number of maps does not fit")
+    if tuple(k_cache.shape[1:]) != (num_kv_heads, k_cache.shape[2], maps * head_dim) or \
             tuple(v_cache.shape[1:]) != (num_kv_heads, k_cache.shape[2], v_head_dim):
         raise KernelError("the cache must be [pages + 1, kv_heads, page_size, width]")
     if (bias is not None and bias.numel() != c) or (q_weight is None) != (k_weight is None) or \
@@ -1987,7 +2028,7 @@ def heads_prepare(x: torch.Tensor, q_out: torch.Tensor, k_cache: torch.Tensor, v
     rc = load_cuda_library("attention_prepare.cu").b200_heads_prepare(
         _p(x), _code(x), x.shape[1], _p(bias), _p(q_weight), _p(k_weight), ctypes.c_float(eps), _p(inv_freq),
         int(rot_dims if inv_freq is not None else 0), int(bool(interleaved)), _p(positions), _p(slots), x.shape[0],
-        num_heads, num_kv_heads, head_dim, v_head_dim, flags, page_size,
+        num_heads, num_kv_heads, head_dim, v_head_dim, flags, maps, ctypes.c_float(rot_gain), page_size,
         ctypes.c_longlong(k_cache.shape[0] * page_size), _p(q_out), _p(k_cache), _p(v_cache),
         _p(error_word(x.device)), _stream())
     _ok(rc, "heads_prepare")
@@ -2214,6 +2255,20 @@ def routed_experts(x: torch.Tensor, choice: torch.Tensor, gains: torch.Tensor, g
     return out
 
 
+def head_difference(a: torch.Tensor, heads: int, v_head_dim: int, lam: float, gain: float, eps: float) -> torch.Tensor:
+    """a [tokens, heads * 2 * v_head_dim], a head's two outputs side by side: o = a_1 - lam a_2, every head's o divided by its
+    root mean square (eps inside the root) times ``gain``; [tokens, heads * v_head_dim] in a's dtype."""
+    _cuda(a)
+    _contig(a)
+    if a.shape[1] != heads * 2 * v_head_dim:
+        raise KernelError("head_difference: two outputs a head are needed")
+    out = torch.empty((a.shape[0], heads * v_head_dim), dtype=a.dtype, device=a.device)
+    rc = _gated().b200_head_difference(_p(out), _p(a), ctypes.c_float(lam), ctypes.c_float(gain), ctypes.c_float(eps),
+                                       ctypes.c_longlong(a.shape[0] * heads), v_head_dim, _code(a), _stream())
+    _ok(rc, "head_difference")
+    return out
+
+
 def glu_columns(gate_up: torch.Tensor, glu: str = "silu", limit: float = 0.0, alpha: float = 1.0) -> torch.Tensor:
     """out = glu(gate_up[:, :F], gate_up[:, F:]) with the forms of ``routed_experts`` or "gelu_tanh" (gelu_tanh(g) u);
     computed in float, rounded once."""
@@ -2344,6 +2399,42 @@ def norm_add_pair(x: torch.Tensor, pair: NormedPair, weight: torch.Tensor, eps: 
     if cast_to is None:
         return None
     return out if out is not None else x
+
+
+def residual_sum(x: torch.Tensor, y=None, add: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None,
+                 mult: float = 1.0, weight: Optional[torch.Tensor] = None, eps: float = 0.0,
+                 out_dtype: torch.dtype = torch.float32, rows: Optional[torch.Tensor] = None,
+                 out: Optional[torch.Tensor] = None, column: int = 0, store: bool = True) -> torch.Tensor:
+    """s = x + mult * (y + bias + add) on the float32 stream x [tokens, width], in float and in one kernel with what is
+    made of it: s / sqrt(mean(s^2) + eps) * weight (float32), or s itself without ``weight``, rounded once to
+    ``out_dtype``; of the tokens ``rows`` only, if given.  ``y`` (a mixer's output, or a ``NormedPair``) and ``add`` (a
+    feed-forward's, of the same dtype) may be missing.  ``store``: s becomes the stream.  ``out`` [.., wider] takes the
+    result from ``column`` on (its dtype then counts)."""
+    pair = y if isinstance(y, NormedPair) else None
+    a, b = (pair.a, pair.b) if pair is not None else (y, None)
+    wa, wb = (pair.a_weight, pair.b_weight) if pair is not None else (None, None)
+    _cuda(x, a, b, add, bias, wa, wb, weight, rows, out)
+    _contig(x, a, b, add, bias, wa, wb, weight, rows, out)
+    _f32(x, bias, wa, wb, weight)
+    _i32(rows)
+    tokens, width = x.shape
+    terms = [t for t in (a, b, add) if t is not None]
+    if any(tuple(t.shape) != (tokens, width) or t.dtype != terms[0].dtype for t in terms) or \
+            any(v is not None and v.numel() != width for v in (bias, wa, wb, weight)) or \
+            (bias is not None and (a is None or pair is not None)) or (pair is not None and weight is not None and eps != pair.eps):
+        raise KernelError("residual_sum: the terms, the weights or their eps do not fit the stream")
+    n = tokens if rows is None else rows.numel()
+    if out is None:
+        out = torch.empty((n, width), dtype=out_dtype, device=x.device)
+    elif out.shape[0] != n or column < 0 or column + width > out.shape[1]:
+        raise KernelError("residual_sum: the result's columns do not fit")
+    rc = load_cuda_library("post_norm.cu").b200_residual_sum(
+        _p(x), _p(a), _p(b), _p(add), _code(terms[0]) if terms else F32, _p(bias), _p(wa), _p(wb), ctypes.c_float(mult),
+        _p(weight), ctypes.c_float(pair.eps if pair is not None else eps), _p(rows),
+        ctypes.c_void_p(out.data_ptr() + column * out.element_size()), _code(out), out.shape[1], int(bool(store)), n, width,
+        _stream())
+    _ok(rc, "residual_sum")
+    return out
 
 
 def norm_rows(x: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype: torch.dtype,

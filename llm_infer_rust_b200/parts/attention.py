@@ -175,8 +175,8 @@ class GatedConvAttention(Part):
             raise ValueError(f"{self.taps} taps are refused: the convolution kernels take up to 8")
         name = spec.get("position_encoding")
         self.rope = env.position_encodings[name] if name else None
-        if self.rope is not None and self.rope.rot_dim > self.d:
-            raise ValueError("the rotation is wider than a head")
+        if self.rope is not None and (self.rope.rot_dim > self.d or getattr(self.rope, "gain", 1.0) != 1.0):
+            raise ValueError("the rotation is wider than a head, or it scales")
         self.qkv_channels = (self.nh + self.nkv) * self.d + self.nkv * self.dv
 
     def param_decls(self):
@@ -248,8 +248,8 @@ class GatedConvAttention(Part):
 
 def _masked_attention(part, q, out, ctx, cache, num_heads, num_kv_heads, head_dim, v_head_dim, sinks,
                       shared_values=False):
-    """Attention of a step's rows over the paged cache for a mixer with ``window``, ``chunk`` and ``scale``: prompt
-    portions and single decoded tokens, softmax weights in float.  ``shared_values``: a value is the first
+    """Attention of a step's rows over the paged cache for a mixer with ``window``, ``chunk``, ``scale`` and ``softcap``:
+    prompt portions and single decoded tokens, softmax weights in float.  ``shared_values``: a value is the first
     ``v_head_dim`` columns of its key's row (one KV head)."""
     g = cache.group
     page = ctx.page_sizes[g]
@@ -257,8 +257,8 @@ def _masked_attention(part, q, out, ctx, cache, num_heads, num_kv_heads, head_di
         ops.prefill_attention(q, cache.k, cache.v, out, ctx.block_tables[g], ctx.cu_q, ctx.kv_len,
                               ctx.prefix_len, ctx.prefill_rows, ctx.num_prefill, ctx.max_q_len,
                               num_heads, num_kv_heads, head_dim, page, part.window, part.scale,
-                              v_head_dim=v_head_dim, precise_weights=True, chunk=part.chunk, sinks=sinks,
-                              shared_values=shared_values)
+                              v_head_dim=v_head_dim, softcap=part.softcap, precise_weights=True, chunk=part.chunk,
+                              sinks=sinks, shared_values=shared_values)
     if ctx.num_decode:
         bound = ctx.kv_len_bound
         for limit in (part.window, part.chunk):
@@ -276,8 +276,8 @@ def _masked_attention(part, q, out, ctx, cache, num_heads, num_kv_heads, head_di
         scratch = ctx.scratch(need) if need else None
         ops.decode_attention(q, cache.k, cache.v, out, scratch, ctx.block_tables[g], ctx.cu_q,
                              ctx.kv_len, ctx.decode_rows, ctx.num_decode, num_heads, num_kv_heads, head_dim,
-                             page, part.window, part.scale, splits, v_head_dim=v_head_dim, precise_weights=True,
-                             chunk=part.chunk, sinks=sinks, shared_values=shared_values)
+                             page, part.window, part.scale, splits, v_head_dim=v_head_dim, softcap=part.softcap,
+                             precise_weights=True, chunk=part.chunk, sinks=sinks, shared_values=shared_values)
 
 
 class GroupedAttention(Part):
@@ -298,6 +298,7 @@ class GroupedAttention(Part):
         (the encoding says whether pairs are interleaved or half-split);
       * ``window`` W: a query at position p reads keys p - W < j <= p;  ``chunk`` C: only keys from p - p % C on
         (its own block of C positions, blocks counted from the sequence's start); both masks may be set;
+      * ``softcap``: score <- cap * tanh(score / cap) after ``softmax_scale`` and before the masks;
       * ``sink``: a learned number per head whose exponential joins the softmax's denominator (no key, no value,
         not scaled); "zero": the number is 0 for every head and no parameter (one is added to the denominator);
       * ``own_kv`` False: the layer has no key and value projections (the packed matrix and bias hold q alone) and
@@ -318,6 +319,7 @@ class GroupedAttention(Part):
         self.window = spec.get("window")
         self.chunk = spec.get("chunk")
         self.scale = float(spec.get("softmax_scale", 1.0 / math.sqrt(self.d)))
+        self.softcap = float(spec.get("softcap") or 0.0)
         self.zero_sink = spec.get("sink") == "zero"
         self.sink = bool(spec.get("sink", False)) and not self.zero_sink
         self.gate = bool(spec.get("gate", False))
@@ -350,6 +352,9 @@ class GroupedAttention(Part):
         self.rot_dims = int(spec.get("rot_dims") or (self.rope.rot_dim if self.rope else 0))
         if self.rope is not None and (self.rot_dims != self.rope.rot_dim or self.rot_dims > self.d):
             raise ValueError("the rotation does not fit the head or the encoding")
+        self.rot_gain = float(getattr(self.rope, "gain", 1.0))
+        if self.rot_gain != 1.0 and self.norm_scope == "projection":
+            raise ValueError("a rotation that scales is served with per-head norms or none")
         self.q_channels = self.nh * self.d
         self.qkv_channels = self.q_channels + (self.nkv * (self.d + (0 if self.values_from_keys else self.dv))
                                                if self.own_kv else 0)
@@ -398,7 +403,7 @@ class GroupedAttention(Part):
         if not (self.norm_scope == "head" and not self.bias and not self.gate and self.own_kv and self.dv == self.d
                 and x.dtype == torch.bfloat16 and ops.few_row_route != "chain"):
             return False
-        if self.rope is not None and getattr(self.rope, "pairing", "half_split") != "half_split":
+        if self.rope is not None and (getattr(self.rope, "pairing", "half_split") != "half_split" or self.rot_gain != 1.0):
             return False
         return ops.few_row_takes(tokens, self.params["qkv_proj"], self.env.dtype, ops.EPI_QKV, self.d, norm=False)
 
@@ -441,7 +446,8 @@ class GroupedAttention(Part):
         prepare = ops.joint_heads_prepare if self.norm_scope == "projection" else ops.heads_prepare
         extra = {"has_kv": self.own_kv} if self.norm_scope == "projection" else \
             {"plain_norm": self.qk_eps is not None and not self.norm_weight,
-             "norm_after_rotation": self.norm_order == "after_rotation", "values_are_keys": self.values_from_keys}
+             "norm_after_rotation": self.norm_order == "after_rotation", "values_are_keys": self.values_from_keys,
+             "rot_gain": self.rot_gain}
         prepare(packed, q, cache.k, cache.v, ctx.positions, slots, self.nh, self.nkv, self.d, self.dv,
                 bias=p.get("qkv_bias"), q_weight=p.get("q_norm"), k_weight=p.get("k_norm"),
                 eps=float(self.qk_eps or 0.0), inv_freq=rope.inv_freq if rope else None,
@@ -452,6 +458,99 @@ class GroupedAttention(Part):
                           self.zero_sinks if self.zero_sink else p.get("sink"))
         if self.gate:
             ops.sigmoid_gate_mul(out, packed, self.qkv_channels, per=self.dv if self.gate_per_head else 1)
+        y = ops.linear(out, p["o_proj"])
+        if self.out_bias and not self.bias_deferred:
+            ops.add_row_bias(y, p["o_bias"])
+        return y
+
+
+class DifferentialAttention(Part):
+    """Grouped-query attention whose every head takes the difference of two softmax maps over the same values
+    (differential attention).  q and k of a head are two vectors of ``head_dim`` each, side by side in the packed
+    projection (q rows, k rows, v rows); values are ``v_head_dim`` wide.  With a_1, a_2 the outputs of the two maps:
+
+        o = a_1 - lambda a_2,      lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff     (one number a layer)
+        o <- o / sqrt(mean(o^2) + eps) * (1 - diff)                                    (a head's vector, no weight)
+
+    and the output projection.  ``lambdas`` holds lq1, lk1, lq2 and lk2 one after the other.  ``bias`` / ``out_bias``, ``position_encoding`` / ``rot_dims`` (each of the four vectors is
+    rotated by itself), ``window``, ``softmax_scale``: as in ``grouped_attention``.
+
+    The two keys of a head are one cache row 2 ``head_dim`` wide, and a query vector is a row of that width with zeros
+    beside its own map's columns: to the attention kernels it is grouped-query attention with 2 ``num_heads`` query
+    heads, so keys and values are fetched once for both maps."""
+    category = "mixer"
+
+    def __init__(self, spec, env):
+        super().__init__(spec, env)
+        self.hidden = int(spec["hidden_size"])
+        self.nh = int(spec["num_heads"])
+        self.nkv = int(spec["num_kv_heads"])
+        self.d = int(spec["head_dim"])
+        self.dv = int(spec.get("v_head_dim") or self.d)
+        self.diff = float(spec["diff"])
+        self.eps = float(spec["eps"])
+        self.bias = bool(spec.get("bias", False))
+        self.out_bias = bool(spec.get("out_bias", False))
+        self.window = spec.get("window")
+        self.chunk, self.softcap = None, 0.0
+        self.scale = float(spec.get("softmax_scale", 1.0 / math.sqrt(self.d)))
+        if self.nh % self.nkv:
+            raise ValueError("num_heads must be a multiple of num_kv_heads")
+        if self.dv % 2 or not 2 <= self.dv <= 512 or not 1 <= self.d <= 256:
+            raise ValueError(f"head sizes {self.d} and {self.dv} are refused: the attention kernels take key rows "
+                             f"(two vectors) and even value rows up to 512")
+        name = spec.get("position_encoding")
+        self.rope = env.position_encodings[name] if name else None
+        self.rot_dims = int(spec.get("rot_dims") or (self.rope.rot_dim if self.rope else 0))
+        if self.rope is not None and (self.rot_dims != self.rope.rot_dim or self.rot_dims > self.d):
+            raise ValueError("the rotation does not fit the head or the encoding")
+        self.qkv_channels = (self.nh + self.nkv) * 2 * self.d + self.nkv * self.dv
+        self.bias_deferred = False
+        self._lambda = None
+
+    def param_decls(self):
+        decls = {"qkv_proj": ParamDecl((self.qkv_channels, self.hidden)),
+                 "o_proj": ParamDecl((self.hidden, self.nh * self.dv)), "lambdas": ParamDecl((4 * self.d,), "vector")}
+        if self.bias:
+            decls["qkv_bias"] = ParamDecl((self.qkv_channels,), "vector")
+        if self.out_bias:
+            decls["o_bias"] = ParamDecl((self.hidden,), "vector")
+        return decls
+
+    def bind(self, name, tensor):
+        super().bind(name, tensor)
+        if name in ("qkv_bias", "o_bias", "lambdas"):
+            self.params[name] = tensor.to(torch.float32).contiguous()
+        if name == "lambdas":
+            # one number a layer, fixed with the weights: taken on the host (in double precision), once
+            lq1, lk1, lq2, lk2 = self.params[name].to("cpu", torch.float64).view(4, self.d)
+            self._lambda = float(torch.exp((lq1 * lk1).sum()) - torch.exp((lq2 * lk2).sum()) + self.diff)
+
+    def defer_output_bias(self) -> bool:
+        """See ``grouped_attention``."""
+        self.bias_deferred = self.out_bias
+        return self.bias_deferred
+
+    def cache_spec(self):
+        return PagedKVSpec(self.nkv, 2 * self.d, self.window, self.dv if self.dv != 2 * self.d else None)
+
+    def state_spec(self):
+        return None
+
+    def forward(self, x, ctx, cache):
+        p = self.params
+        packed = ops.linear(x, p["qkv_proj"])
+        tokens = packed.shape[0]
+        rope = self.rope
+        q = torch.empty((tokens, 2 * self.nh * 2 * self.d), dtype=packed.dtype, device=packed.device)
+        ops.heads_prepare(packed, q, cache.k, cache.v, ctx.positions, ctx.slots[cache.group] if cache.writes else None,
+                          2 * self.nh, self.nkv, self.d, self.dv, bias=p.get("qkv_bias"),
+                          inv_freq=rope.inv_freq if rope else None, rot_dims=self.rot_dims if rope else 0,
+                          interleaved=getattr(rope, "pairing", "half_split") == "interleaved", maps=2,
+                          rot_gain=float(getattr(rope, "gain", 1.0)))
+        maps = torch.empty((tokens, 2 * self.nh * self.dv), dtype=packed.dtype, device=packed.device)
+        _masked_attention(self, q, maps, ctx, cache, 2 * self.nh, self.nkv, 2 * self.d, self.dv, None)
+        out = ops.head_difference(maps, self.nh, self.dv, self._lambda, 1.0 - self.diff, self.eps)
         y = ops.linear(out, p["o_proj"])
         if self.out_bias and not self.bias_deferred:
             ops.add_row_bias(y, p["o_bias"])
@@ -489,6 +588,7 @@ class LatentAttention(Part):
         self.eps = float(spec["eps"])
         self.window = spec.get("window")
         self.chunk = spec.get("chunk")
+        self.softcap = 0.0
         self.scale = float(spec.get("softmax_scale", 1.0 / math.sqrt(self.d + self.r)))
         self.sink = bool(spec.get("sink", False))
         self.gate = bool(spec.get("gate", False))
@@ -499,8 +599,9 @@ class LatentAttention(Part):
         name = spec.get("position_encoding")
         self.rope = env.position_encodings[name] if name else None
         self.rot_dims = int(spec.get("rot_dims") or (self.rope.rot_dim if self.rope else 0))
-        if self.rope is not None and (self.rot_dims != self.rope.rot_dim or self.rot_dims > self.r):
-            raise ValueError("the rotation does not fit the rotated part or the encoding")
+        if self.rope is not None and (self.rot_dims != self.rope.rot_dim or self.rot_dims > self.r
+                                      or getattr(self.rope, "gain", 1.0) != 1.0):
+            raise ValueError("the rotation does not fit the rotated part or the encoding, or it scales")
         self.q_channels = self.nh * (self.d + self.r)
         self.down_column = self.q_rank if self.q_rank else self.q_channels
         self.gate_column = self.down_column + self.c + self.r
@@ -565,5 +666,6 @@ class LatentAttention(Part):
 
 register_part("mixer", "gqa_attention", GQAttention)
 register_part("mixer", "grouped_attention", GroupedAttention)
+register_part("mixer", "differential_attention", DifferentialAttention)
 register_part("mixer", "latent_attention", LatentAttention)
 register_part("mixer", "gated_conv_attention", GatedConvAttention)

@@ -24,6 +24,8 @@ Optional, for fusion across parts: a norm may offer ``pending_add(x, residual, .
 returns the add + norm unrun (``ops.PendingNorm``); a mixer, feed-forward or head that offers
 ``takes_pending(tokens) -> bool`` and answers True is then given that object as ``x`` and runs it
 as the prologue of its first product.  Parts without these methods get plain tensors.
+``stream_input``      ``begin(h) -> kept`` of the embedding's output, ``forward(h, residual, kept) -> (h, residual)``
+                      before the run-list entries that name it
 ``block``             built from a ``LayerSpec``; ``forward(h, residual, ctx, cache) -> (h, residual)``
 ``embedding``         ``forward(token_ids) -> h``; one that says ``needs_context`` (it keeps per-request state,
                       ``state_specs()``): ``forward(token_ids, ctx, cache) -> h``

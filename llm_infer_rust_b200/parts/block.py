@@ -5,6 +5,7 @@ import torch
 
 from ..kernels import ops
 from .base import ParamDecl, Part
+from .norm import OwedRMSNorm, OwedSum
 from .registry import build_part, register_part
 
 
@@ -252,6 +253,74 @@ class PostNormStream:
         return h, x
 
 
+class ParallelSublayers:
+    """A layer whose mixer and feed-forward read the SAME normed input, over a float32 stream x:
+
+        h = norm(x);    x <- x + ``residual_mult`` (mixer(h) + feed_forward(h))
+
+    Parts by name: ``input_norm`` (``owed_rms_norm``), ``mixer`` and optionally ``feed_forward``.  The sum is owed
+    (``OwedSum``) to the next read of the stream: the block returns (what is owed, the stream), and the next block's norm,
+    a pass input or the model's last norm takes both in one kernel.  A mixer that has an output bias and offers
+    ``defer_output_bias()`` leaves the bias to that kernel.  A feed-forward that says ``needs_context`` is also given the
+    step's context."""
+    category = "block"
+
+    def __init__(self, layer_spec, env):
+        self.spec = layer_spec
+        self.env = env
+        parts = layer_spec.parts
+        self.mult = float(layer_spec.block.get("residual_mult", 1.0))
+        self.input_norm = build_part("norm", layer_spec["input_norm"], env)
+        self.mixer = build_part("mixer", layer_spec["mixer"], env)
+        self.feed_forward = build_part("feed_forward", parts["feed_forward"], env) if "feed_forward" in parts else None
+        if not hasattr(self.input_norm, "read_raw"):
+            raise ValueError("this block needs a norm that takes an owed sum (owed_rms_norm)")
+        defer = getattr(self.mixer, "defer_output_bias", None)
+        self.mixer_bias_here = bool(defer()) if defer is not None else False
+
+    def children(self):
+        named = {"input_norm": self.input_norm, "mixer": self.mixer, "feed_forward": self.feed_forward}
+        return {name: part for name, part in named.items() if part is not None}
+
+    def forward(self, h, residual, ctx, cache):
+        ops.flush_chain()
+        owed, stream = (None, h) if residual is None else (h, residual)
+        x = self.input_norm.read(owed, stream)
+        y = self.mixer.forward(x, ctx, cache)
+        add = None
+        if self.feed_forward is not None:
+            add = self.feed_forward.forward(x, ctx) if getattr(self.feed_forward, "needs_context", False) \
+                else self.feed_forward.forward(x)
+        return OwedSum(y, add, self.mult, self.mixer.params.get("o_bias") if self.mixer_bias_here else None), stream
+
+
+class ConcatInput(Part):
+    """What a pass through repeated layers begins with: x <- W [x; x0], x0 being the embedding's output and ``weight``
+    [width, 2 width] (x's columns first).  The product reads both rounded once to the engine's dtype and leaves a float32
+    stream."""
+    category = "stream_input"
+
+    def __init__(self, spec, env):
+        super().__init__(spec, env)
+        self.width = int(spec["width"])
+
+    def param_decls(self):
+        return {"weight": ParamDecl((self.width, 2 * self.width))}
+
+    def begin(self, h):
+        """The product's input rows with x0 in place (h: the embedding's output, float32 [tokens, width])."""
+        rows = torch.empty((h.shape[0], 2 * self.width), dtype=self.env.dtype, device=h.device)
+        OwedRMSNorm.read_raw(None, h, rows, self.width)
+        return rows
+
+    def forward(self, h, residual, rows):
+        owed, stream = (None, h) if residual is None else (h, residual)
+        OwedRMSNorm.read_raw(owed, stream, rows, 0)
+        return ops.linear(rows, self.params["weight"], out_dtype=torch.float32), None
+
+
+register_part("stream_input", "concat_input", ConcatInput)
+register_part("block", "parallel_sublayers", ParallelSublayers)
 register_part("stream_mix", "stream_mix", StreamMix)
 register_part("block", "post_norm_stream", PostNormStream)
 register_part("block", "pre_norm_deferred_add", PreNormDeferredAdd)

@@ -91,10 +91,11 @@ class DenseActFF(Part):
 
 
 class GatedActFF(Part):
-    """down(act(gate(x)) * up(x)), no bias, gate and up packed into one matrix (gate rows first); ``activation``:
-    gelu_tanh or silu, computed in float.  The dense models' fused products (few tokens; large portions) serve it too."""
+    """down(glu(gate(x), up(x))), no bias, gate and up packed into one matrix (gate rows first); ``activation``: gelu_tanh or
+    silu (act(g) u), or clamped_swish: g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit), u' = clamp(u, -limit, limit)
+    (``limit``; ``alpha`` 1.702 unless given); computed in float.  The dense models' fused products (few tokens; large portions) serve it too."""
     category = "feed_forward"
-    _GLU = {"gelu_tanh": "gelu_tanh", "silu": "silu"}
+    _GLU = {"gelu_tanh": "gelu_tanh", "silu": "silu", "clamped_swish": "clamped_swish"}
 
     def __init__(self, spec, env):
         super().__init__(spec, env)
@@ -103,6 +104,10 @@ class GatedActFF(Part):
         self.activation = str(spec["activation"])
         if self.activation not in self._GLU:
             raise ValueError(f"activation {self.activation!r} is refused: {sorted(self._GLU)}")
+        self.limit = float(spec.get("limit") or 0.0)
+        self.alpha = float(spec.get("alpha") or 1.702)
+        if self.activation == "clamped_swish" and not self.limit > 0.0:
+            raise ValueError("clamped_swish needs a positive limit")
 
     def param_decls(self):
         return {"gate_up_proj": ParamDecl((2 * self.inter, self.hidden)),
@@ -112,11 +117,11 @@ class GatedActFF(Part):
         w, act = self.params["gate_up_proj"], self._GLU[self.activation]
         if x.dtype == torch.bfloat16 and ops.few_row_route == "single" and \
                 ops.few_row_takes(x.shape[0], w, self.env.dtype, ops.EPI_SWIGLU, norm=False):
-            a = ops.few_row_glu(x, w, act)                       # few tokens: both projections and the activation in one kernel
+            a = ops.few_row_glu(x, w, act, self.limit, self.alpha)       # few tokens: both projections and the activation in one kernel
         elif x.dtype == torch.bfloat16 and ops.gemm_tc_pays(x, w, ops.GEMM_SWIGLU):
-            a = ops.gemm_tc(x, w, ops.GEMM_SWIGLU, glu=act)      # many tokens, large matrices: as the tcgen05 product's epilogue
+            a = ops.gemm_tc(x, w, ops.GEMM_SWIGLU, glu=act, limit=self.limit, alpha=self.alpha)      # many tokens, large matrices: as the tcgen05 product's epilogue
         else:
-            a = ops.glu_columns(ops.linear(x, w), act)
+            a = ops.glu_columns(ops.linear(x, w), act, self.limit, self.alpha)
         return ops.linear(a, self.params["down_proj"])
 
 

@@ -15,7 +15,8 @@ class DecoderModel:
     """Built from a ``ModelSpec`` alone; knows no architecture.
 
     Parameter paths: ``embedding.weight``, ``layers.<i>.<child>.<name>`` (children as
-    the block names them; ``layers.<i>.<child>.<inner>.<name>`` for a part inside a part), ``final_norm.weight``, ``lm_head.weight``.
+    the block names them; ``layers.<i>.<child>.<inner>.<name>`` for a part inside a part), ``final_norm.weight``, ``lm_head.weight``;
+    ``stream_inputs.<name>.<parameter>`` for what run-list entries are fed through before they run.
     """
 
     def __init__(self, spec: ModelSpec, dtype: torch.dtype, device: torch.device):
@@ -29,6 +30,7 @@ class DecoderModel:
         self.position_encodings = env.position_encodings
         self.embedding = build_part("embedding", spec.embedding, env)
         self.blocks = [build_part("block", layer, env) for layer in spec.layers]
+        self.stream_inputs = {name: build_part("stream_input", part, env) for name, part in spec.stream_inputs.items()}
         self.final_norm = build_part("norm", spec.final_norm, env)
         self.lm_head = build_part("head", spec.lm_head, env)
         self.run_list = list(spec.run_list)
@@ -43,6 +45,7 @@ class DecoderModel:
     # ------------------------------------------------------------------ parameters
     def _owners(self) -> Dict[str, Part]:
         owners = {"embedding": self.embedding, "final_norm": self.final_norm, "lm_head": self.lm_head}
+        owners.update({f"stream_inputs.{name}": part for name, part in self.stream_inputs.items()})
         for i, block in enumerate(self.blocks):
             for child, part in block.children().items():
                 self._own(owners, f"layers.{i}.{child}", part)
@@ -92,7 +95,11 @@ class DecoderModel:
         else:
             h = self.embedding.forward(ctx.token_ids)
         residual = None
+        # what the stream inputs keep of the embedding's output, before a layer changes it
+        kept = {name: part.begin(h) for name, part in self.stream_inputs.items()}
         for e, entry in enumerate(self.run_list):
+            if entry.input is not None:
+                h, residual = self.stream_inputs[entry.input].forward(h, residual, kept[entry.input])
             h, residual = self.blocks[entry.layer].forward(h, residual, ctx, caches[e])
         takes = getattr(self.lm_head, "takes_pending", None)
         if not (getattr(self.final_norm, "chainable", False) and getattr(self.lm_head, "chainable", False)):

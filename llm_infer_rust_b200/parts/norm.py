@@ -185,7 +185,52 @@ class OutputLayerNorm(OutputRMSNorm):
     center = True
 
 
+class OwedSum:
+    """What a block still owes to its float32 stream: mult * (y + bias + add), y a mixer's output (or ``ops.NormedPair``) and
+    ``add`` a feed-forward's output of the same input (None: none)."""
+
+    def __init__(self, y, add, mult, bias=None):
+        self.y, self.add, self.mult, self.bias = y, add, mult, bias
+
+
+class OwedRMSNorm(Part):
+    """RMS norm of a float32 stream that is handed the sum it is still owed (``OwedSum``): x <- x + owed, in float, then
+    x / sqrt(mean(x^2) + eps) * weight rounded once to the engine's dtype, one kernel (``read``).  ``read_raw``: the same
+    without the norm, the new x itself rounded into columns of a wider matrix (the stream is not written: whatever is made
+    of those columns takes its place).  ``forward`` / ``forward_add``: a model's last norm, at the chosen rows."""
+    category = "norm"
+
+    def __init__(self, spec, env):
+        super().__init__(spec, env)
+        self.width = int(spec["width"])
+        self.eps = float(spec["eps"])
+
+    def param_decls(self):
+        return {"weight": ParamDecl((self.width,), "vector")}
+
+    def bind(self, name, tensor):
+        super().bind(name, tensor)
+        self.params[name] = tensor.to(torch.float32).contiguous()
+
+    def read(self, owed, stream, rows=None, store=True):
+        terms = {} if owed is None else dict(y=owed.y, add=owed.add, bias=owed.bias, mult=owed.mult)
+        return ops.residual_sum(stream, weight=self.params["weight"], eps=self.eps, out_dtype=self.env.dtype, rows=rows,
+                                store=store and owed is not None, **terms)
+
+    @staticmethod
+    def read_raw(owed, stream, out, column):
+        terms = {} if owed is None else dict(y=owed.y, add=owed.add, bias=owed.bias, mult=owed.mult)
+        return ops.residual_sum(stream, out=out, column=column, store=False, **terms)
+
+    def forward(self, x, out=None, rows=None):
+        return self.read(None, x, rows=rows)
+
+    def forward_add(self, x, residual, out=None, rows=None, write_residual=True):
+        return self.read(x, residual, rows=rows, store=write_residual)
+
+
 register_part("norm", "rms_norm", RMSNorm)
+register_part("norm", "owed_rms_norm", OwedRMSNorm)
 register_part("norm", "output_rms_norm", OutputRMSNorm)
 register_part("norm", "output_layer_norm", OutputLayerNorm)
 register_part("norm", "stream_rms_norm", StreamRMSNorm)

@@ -42,6 +42,10 @@ class RotaryFrequencies(Part):
     ``wavelength_scaling`` {factor, low, high, original} stretches by wavelength l = 2 pi / f instead: f is kept where
     l < original / high, divided by ``factor`` where l > original / low, and in between blended,
     (1 - s) f / factor + s f with s = (original / l - low) / (high - low).
+    ``yarn`` {factor, original, fast, slow} (YaRN) blends by the pair's index i instead: with
+    d(t) = rot_dim ln(original / (2 pi t)) / (2 ln theta), lo = max(floor(d(fast)), 0), hi = min(ceil(d(slow)), rot_dim - 1)
+    and r = clamp((i - lo) / max(hi - lo, 0.001), 0, 1) the frequency is r f / factor + (1 - r) f, and cosines and sines
+    are multiplied by 0.1 ln(factor) + 1 (``gain``; a mixer whose kernel does not take a gain refuses the encoding).
     ``pairing`` says which coordinates frequency i turns: "half_split" (i and i + rot_dim / 2, the default) or
     "interleaved" (2i and 2i + 1); a mixer's kernel reads it, and a mixer that cannot serve a pairing refuses it."""
     category = "position_encoding"
@@ -70,6 +74,23 @@ class RotaryFrequencies(Part):
             # outside the band the blend is exactly 0 or 1, so one expression serves all three ranges
             inv_freq = torch.where(wavelength < original / high, inv_freq,
                                    torch.where(wavelength > original / low, inv_freq / factor, blended))
+        self.gain = 1.0
+        yarn = spec.get("yarn")
+        if yarn:
+            if stretch:
+                raise ValueError("wavelength_scaling and yarn exclude one another")
+            factor, original = float(yarn["factor"]), float(yarn["original"])
+            fast, slow = float(yarn["fast"]), float(yarn["slow"])
+            if factor <= 0.0 or original <= 0.0 or fast <= 0.0 or slow <= 0.0 or self.theta <= 1.0:
+                raise ValueError("yarn needs positive factor, original, fast and slow, and a base above 1")
+
+            def index_of(turns: float) -> float:
+                return self.rot_dim * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(self.theta))
+            lo, hi = max(math.floor(index_of(fast)), 0), min(math.ceil(index_of(slow)), self.rot_dim - 1)
+            index = torch.arange(self.rot_dim // 2, dtype=torch.float64)
+            ramp = torch.clamp((index - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+            inv_freq = inv_freq / factor * ramp + inv_freq * (1.0 - ramp)
+            self.gain = 0.1 * math.log(factor) + 1.0
         self.inv_freq = inv_freq.to(torch.float32).to(env.device).contiguous()
 
 

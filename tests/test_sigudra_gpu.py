@@ -215,7 +215,8 @@ def test_recurrence_with_strong_and_weak_decays(heads, kv, d, dv, delta):
     dev = "cuda"
     state = torch.full((3, heads, d, dv), 5.0, device=dev)
     state[2] = start.to(dev)
-    lib = ops._linear_state()
+    from llm_infer_rust_b200.kernels.build import load_cuda_library
+    lib = load_cuda_library("state_scan.cu")
 
     def scan(lo, hi):
         parts = [t[lo:hi].reshape(hi - lo, -1).to(dev).contiguous() for t in (q, k, v, decay, beta)]
@@ -225,7 +226,7 @@ def test_recurrence_with_strong_and_weak_decays(heads, kv, d, dv, delta):
         rc = lib.b200_state_scan(p[0], p[1], p[2], p[3], p[4] if delta else None, ctypes.c_void_p(out.data_ptr()),
                                  ctypes.c_void_p(state.data_ptr()), ctypes.c_void_p(ctx.cu_q.data_ptr()),
                                  ctypes.c_void_p(ctx.prefix_len.data_ptr()), ctypes.c_void_p(ctx.state_slots.data_ptr()), 1,
-                                 heads, kv, d, dv, ctypes.c_void_p(torch.cuda.current_stream().cuda_stream))
+                                 heads, kv, d, dv, 0, ctypes.c_void_p(torch.cuda.current_stream().cuda_stream))
         assert rc == 0
         torch.cuda.synchronize()
         return out.cpu()
