@@ -456,9 +456,9 @@ def kernel_table(size, peak):
         else:
             from llm_infer_rust_b200.parts.attention import decode_splits
             kvb = rows_dec * ctx_len * nkv * d * 2 * 2
-            for name, kw, plain in (("kefetar.attention_softcap", dict(v_head_dim=d, softcap=50.0, precise_weights=True), True),
-                                    ("qwen3.attention", {}, True)):
-                splits = decode_splits(ops.decode_ctas_per_split(bf, rows_dec, nh, nkv, d, page, plain), ctx_len, 148)
+            for name, kw in (("kefetar.attention_softcap", dict(v_head_dim=d, softcap=50.0, precise_weights=True)),
+                             ("qwen3.attention", {})):
+                splits = decode_splits(ops.decode_ctas_per_split(bf, rows_dec, nh, nkv, d, page), ctx_len, 148)
                 need = ops.decode_scratch_floats(rows_dec, nh, d, splits)
                 scratch = torch.empty(max(need, 1), device=dev)
                 put(f"decode.{name}", timed_alone(lambda: ops.decode_attention(
@@ -615,8 +615,7 @@ def mukenex_kernel_table(size, peak):
                 d ** -0.5), flush), flops=4.0 * nh * d * T * (T + 1) / 2, of="bf16")
         else:
             def decode(name, qq, kk, vv, oo, heads, kvh, dk, dv_, bound, nbytes, **kw):
-                plain = dk == dv_
-                per_split = ops.decode_ctas_per_split(bf, rows_dec, heads, kvh, dk, page, plain)
+                per_split = ops.decode_ctas_per_split(bf, rows_dec, heads, kvh, dk, page, dv_)
                 if kw.get("shared_values"):
                     per_split = rows_dec * (heads // ops.latent_head_group(heads))
                 splits = decode_splits(per_split, bound, 148)
@@ -796,7 +795,7 @@ def torinex_kernel_table(size, peak):
                 d ** -0.5), flush), flops=4.0 * nh * d * T * (T + 1) / 2, of="bf16")
         else:
             def decode(name, bound, nbytes, **kw):
-                per_split = ops.decode_ctas_per_split(bf, rows_dec, nh, nkv, d, page, True)
+                per_split = ops.decode_ctas_per_split(bf, rows_dec, nh, nkv, d, page)
                 splits = decode_splits(per_split, bound, 148)
                 need = ops.decode_scratch_floats(rows_dec, nh, d, splits)
                 scratch = torch.empty(max(need, 1), device=dev)
@@ -1019,8 +1018,7 @@ def lufizen_kernel_table(size, peak):
                 flops=2.0 * nh * (2 * rank + r) * sum(min(p, window - 1) + 1 for p in range(T)), of="bf16")
         else:
             def decode(name, qq, kk, vv, oo, heads, kvh, dk, dv_, bound, nbytes, **kw):
-                plain = dk == dv_
-                per_split = ops.decode_ctas_per_split(bf, rows_dec, heads, kvh, dk, page, plain)
+                per_split = ops.decode_ctas_per_split(bf, rows_dec, heads, kvh, dk, page, dv_)
                 keys = 512
                 if kw.get("shared_values"):
                     per_split = rows_dec * (heads // ops.latent_head_group(heads))
@@ -1278,7 +1276,7 @@ def sigudra_kernel_table(size, peak):
                     q, k_cache, v_cache, o, c.table, c.cu_q, c.kv_len, c.prefix_len, c.rows, 1, T, nh, nkv, d, page, win,
                     d ** -0.5, **more), flush, repeats=few), flops=4.0 * nh * d * seen)
             else:
-                splits = decode_splits(ops.decode_ctas_per_split(bf, rows_dec, nh, nkv, d, page, True), window, 148)
+                splits = decode_splits(ops.decode_ctas_per_split(bf, rows_dec, nh, nkv, d, page), window, 148)
                 scratch = torch.empty(max(ops.decode_scratch_floats(rows_dec, nh, d, splits), 1), device=dev)
                 put(f"decode.{name}", timed_alone(lambda: ops.decode_attention(
                     q, k_cache, v_cache, o, scratch, c.table, c.cu_q, c.kv_len, c.rows, rows_dec, nh, nkv, d, page, win,

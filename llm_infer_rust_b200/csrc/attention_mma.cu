@@ -41,27 +41,41 @@
 // row (from column ScoreForm::v_col0 on), so a block's tile is fetched once and serves both products.  The output
 // goes to columns out_col0 .. out_col0 + V_DIM of rows out_width wide: values wider than 256 columns take several
 // launches, each with the scores computed again.
+//
+// Values of another width than keys take a build with -DV_DIM=<multiple of 16, at most 256> (a block's tile then holds
+// key boxes and value boxes of different counts).
+//
+// A build with -DDIFF=1 hands on the difference of a head's two maps (differential attention): the query vectors of a KV
+// head are pairs, rows 2j and 2j + 1 the two maps of one head, and what is stored for the pair is
+//     o / sqrt(mean(o^2) + diff_eps) * diff_gain,   o = a_(2j) - diff_lambda a_(2j + 1),
+// in float from the softmax on and rounded once; an output row is half as many heads wide.
 #ifndef V_SHARED
 #define V_SHARED 0
 #endif
 #ifndef V_DIM
 #define V_DIM HEAD_DIM
 #endif
+#ifndef DIFF
+#define DIFF 0
+#endif
 static_assert(HEAD_DIM % 16 == 0 && HEAD_DIM >= 16 && HEAD_DIM <= (V_SHARED ? 512 : 256),
               "the tensor-core kernels take head sizes 16..256 in steps of 16 (keys of a shared row: up to 512)");
-static_assert(V_DIM % 16 == 0 && V_DIM >= 16 && V_DIM <= 256 && V_DIM <= HEAD_DIM && (V_SHARED || V_DIM == HEAD_DIM),
-              "values are as wide as keys, or 16..256 columns of the keys' own rows");
+static_assert(V_DIM % 16 == 0 && V_DIM >= 16 && V_DIM <= 256 && (!V_SHARED || (V_DIM <= HEAD_DIM && !DIFF)),
+              "values are 16..256 columns wide (of a shared row: some of the keys' own columns)");
 
 typedef __nv_bfloat16 bf16;
 namespace cg = cooperative_groups;
 constexpr int D = HEAD_DIM;
 constexpr int DV = V_DIM;          // columns of a value and of an output tile
 constexpr bool kShared = V_SHARED != 0;
+constexpr bool kDiff = DIFF != 0;
 constexpr int LD = D + 8;          // padded row of the query tile (16 bytes of padding): conflict-free ldmatrix
 constexpr int KB = 32;             // keys per block
 constexpr int NB = (D + 63) / 64;  // 64-dim (128-byte) column boxes per row
 constexpr int HALF_BYTES = KB * 128;              // one column box of a block: 32 rows x 128 bytes
-constexpr int TILE_BYTES = (kShared ? 1 : 2) * NB * HALF_BYTES;   // keys then values of one block (one tile for both)
+constexpr int NBV = kShared ? 0 : (DV + 63) / 64;                 // column boxes of a value row with a tile of its own
+constexpr int TILE_BYTES = (NB + NBV) * HALF_BYTES;               // keys then values of one block (one tile for both)
+constexpr int VALUE_CHUNKS = (kShared ? NB : NBV) * 8;            // 16-byte chunks of a row that holds values
 constexpr int V_OFFSET = kShared ? 0 : NB * HALF_BYTES;           // where a block's values begin in its tile
 constexpr int QROWS = 16;          // rows of the A operand: query heads of one KV head
 
@@ -98,6 +112,7 @@ struct ScoreForm {
   const float* sinks;
   int v_col0;                  // shared rows: first column of the values
   int out_width, out_col0;     // an output row's width and the first column that this launch writes
+  float diff_lambda, diff_gain, diff_eps;      // DIFF
 };
 // The sum of a row's weights with the sink's term (the row's maximum m is in log2 units).
 __device__ __forceinline__ float with_sink(const ScoreForm& sf, int head, float m, float l) {
@@ -146,7 +161,7 @@ __device__ __forceinline__ void fetch_block(unsigned char* tile, const CUtensorM
                                             int kv_end, uint64_t* bar, int lane) {
   const int n_sub = (min(KB, kv_end - first_key) + box_rows - 1) / box_rows;
   asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");   // earlier reads and writes of the tile come first
-  if (lane == 0) mbar_expect_tx(bar, static_cast<uint32_t>(n_sub) * (kShared ? 1u : 2u) * NB * box_rows * 128u);
+  if (lane == 0) mbar_expect_tx(bar, static_cast<uint32_t>(n_sub) * (NB + NBV) * box_rows * 128u);
   __syncwarp();
   if (lane < n_sub) {
     const int key0 = first_key + lane * box_rows;
@@ -155,8 +170,11 @@ __device__ __forceinline__ void fetch_block(unsigned char* tile, const CUtensorM
 #pragma unroll
     for (int h = 0; h < NB; ++h) {
       tma_load_2d(tile + h * HALF_BYTES + lane * box_rows * 128, kmap, h * 64, y, bar);
-      if constexpr (!kShared) tma_load_2d(tile + (NB + h) * HALF_BYTES + lane * box_rows * 128, vmap, h * 64, y, bar);
+      if (h < NBV) tma_load_2d(tile + (NB + h) * HALF_BYTES + lane * box_rows * 128, vmap, h * 64, y, bar);
     }
+#pragma unroll
+    for (int h = NB; h < NBV; ++h)
+      tma_load_2d(tile + (NB + h) * HALF_BYTES + lane * box_rows * 128, vmap, h * 64, y, bar);
   }
 }
 
@@ -378,7 +396,7 @@ decode_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_constan
       // Value rows beyond the sequence: whatever the page holds there must not reach P.V.
       const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
 #pragma unroll
-      for (int c = 0; c < NB * 8; ++c) *reinterpret_cast<uint4*>(t + V_OFFSET + (c >> 3) * HALF_BYTES + lane * 128 + (c & 7) * 16) = zero;
+      for (int c = 0; c < VALUE_CHUNKS; ++c) *reinterpret_cast<uint4*>(t + V_OFFSET + (c >> 3) * HALF_BYTES + lane * 128 + (c & 7) * 16) = zero;
     }
     __syncwarp();
     if (first_key + KB <= kv_end && (window <= 0 || first_key > qp - window) &&
@@ -395,8 +413,24 @@ decode_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_constan
   // Merge the warps through shared memory: [WARPS][group][D + 2] floats over the tile area.
   float* merge = reinterpret_cast<float*>(tiles);     // all copies have landed and been used
   constexpr int MS = DV + 2;
-  const int ow = kShared ? sf.out_width : D, oc = kShared ? sf.out_col0 : 0;     // an output row and this launch's columns
+  const int ow = kShared ? sf.out_width : DV, oc = kShared ? sf.out_col0 : 0;     // an output row and this launch's columns
   float* mine = merge + WARPS * QROWS * MS;           // [group][MS]: the CTA's own combined part
+  // DIFF: the pairs of finished outputs [group][MS] in shared memory become the stored heads, a warp a head
+  auto store_differences = [&](const float* done) {
+    __syncthreads();
+    for (int j = warp; j < group / 2; j += WARPS) {
+      const float* a = done + 2 * j * MS;
+      const float* b = a + MS;
+      float ss = 0.0f;
+      for (int dim = lane; dim < DV; dim += 32) {
+        const float o = fmaf(-sf.diff_lambda, b[dim], a[dim]);
+        ss = fmaf(o, o, ss);
+      }
+      const float f = sf.diff_gain / sqrtf(warp_sum(ss) / static_cast<float>(DV) + sf.diff_eps);
+      bf16* dst = out + (static_cast<size_t>(tok) * (nh / 2) + head0 / 2 + j) * DV;
+      for (int dim = lane; dim < DV; dim += 32) dst[dim] = __float2bfloat16_rn(fmaf(-sf.diff_lambda, b[dim], a[dim]) * f);
+    }
+  };
   const int t2 = (lane & 3) * 2;
 #pragma unroll
   for (int half = 0; half < 2; ++half) {
@@ -430,7 +464,9 @@ decode_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_constan
     const int head = head0 + r;
     if (splits == 1) {
       l = with_sink(sf, head, m, l);
-      out[(static_cast<size_t>(tok) * nh + head) * ow + oc + dim] = __float2bfloat16_rn(l > 0.0f ? o / l : 0.0f);
+      const float y = l > 0.0f ? o / l : 0.0f;
+      if constexpr (kDiff) mine[r * MS + dim] = y;
+      else out[(static_cast<size_t>(tok) * nh + head) * ow + oc + dim] = __float2bfloat16_rn(y);
     } else if (cluster_merge) {
       mine[r * MS + dim] = o;                          // this CTA's part, for the cluster's first CTA to read
       if (dim == 0) { mine[r * MS + DV] = m; mine[r * MS + DV + 1] = l; }
@@ -439,6 +475,9 @@ decode_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_constan
       part_acc[slot * DV + dim] = o;
       if (dim == 0) { part_ml[slot * 2] = m; part_ml[slot * 2 + 1] = l; }
     }
+  }
+  if constexpr (kDiff) {
+    if (splits == 1) store_differences(mine);
   }
   if (!cluster_merge) return;
   // The splits of a (row, KV head) pair are the CTAs of one cluster: the first combines all parts out of the others'
@@ -460,10 +499,55 @@ decode_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_constan
         }
         l = with_sink(sf, head0 + r, m, l);
       }
-      out[(static_cast<size_t>(tok) * nh + head0 + r) * ow + oc + dim] = __float2bfloat16_rn(l > 0.0f ? o / l : 0.0f);
+      const float y = l > 0.0f ? o / l : 0.0f;
+      if constexpr (kDiff) merge[r * MS + dim] = y;      // (the warps' parts there have been used)
+      else out[(static_cast<size_t>(tok) * nh + head0 + r) * ow + oc + dim] = __float2bfloat16_rn(y);
     }
+    if constexpr (kDiff) store_differences(merge);
   }
   cluster.sync();                                      // nobody leaves while its shared memory may still be read
+}
+
+// DIFF.  grid (decode rows, nh / 2): combines the splits of a head's two maps and stores their difference.
+__global__ void decode_mma_merge_diff_kernel(bf16* __restrict__ out, const float* __restrict__ part_acc,
+                                             const float* __restrict__ part_ml, const int* __restrict__ cu_q,
+                                             const int* __restrict__ rows, int nh, int splits, float lambda, float gain,
+                                             float eps) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float scratch[33];
+  constexpr int PER = (DV + 63) / 64;                   // columns of a thread (the launcher gives at least 64 threads)
+  const int tok = cu_q[rows[blockIdx.x]];
+  float y[PER] = {};
+  for (int map = 0; map < 2; ++map) {
+    const size_t base = (static_cast<size_t>(blockIdx.x) * nh + 2 * blockIdx.y + map) * splits;
+    float m = -INFINITY;
+    for (int s = 0; s < splits; ++s) m = fmaxf(m, part_ml[(base + s) * 2]);
+    if (m == -INFINITY) continue;
+    float l = 0.0f, o[PER] = {};
+    for (int s = 0; s < splits; ++s) {
+      const float f = exp2f(part_ml[(base + s) * 2] - m);
+      l += part_ml[(base + s) * 2 + 1] * f;
+#pragma unroll
+      for (int i = 0; i < PER; ++i) {
+        const int dim = threadIdx.x + i * blockDim.x;
+        if (dim < DV) o[i] += part_acc[(base + s) * DV + dim] * f;
+      }
+    }
+    const float w = (map == 0 ? 1.0f : -lambda) / l;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) y[i] = fmaf(w, o[i], y[i]);
+  }
+  float ss = 0.0f;
+#pragma unroll
+  for (int i = 0; i < PER; ++i) ss = fmaf(y[i], y[i], ss);
+  const float f = gain / sqrtf(block_sum(ss, scratch) / static_cast<float>(DV) + eps);
+  bf16* dst = out + (static_cast<size_t>(tok) * (nh / 2) + blockIdx.y) * DV;
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int dim = threadIdx.x + i * blockDim.x;
+    if (dim < DV) dst[dim] = __float2bfloat16_rn(y[i] * f);
+  }
 }
 
 // grid (decode rows, nh): combines the splits of one head (maxima are in log2 units).
@@ -501,7 +585,7 @@ __global__ void decode_mma_merge_kernel(bf16* __restrict__ out, const float* __r
 // window) is applied per row of the score tile.
 constexpr int PF_WARPS = 4;
 // Three CTAs share an SM for heads up to 128 wide (the register budget that this leaves is 170 a thread).
-constexpr int PF_MIN_CTAS = D <= 128 ? 3 : 1;
+constexpr int PF_MIN_CTAS = D <= 128 && DV <= 128 ? 3 : 1;
 constexpr int PF_ROWS = PF_WARPS * 16;
 
 __device__ __forceinline__ void mbar_arrive(uint64_t* bar) {
@@ -612,7 +696,7 @@ prefill_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_consta
       // masked for every query of the tile): keep them out of P.V.
       const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
 #pragma unroll
-      for (int c = 0; c < NB * 8; ++c) *reinterpret_cast<uint4*>(t + V_OFFSET + (c >> 3) * HALF_BYTES + lane * 128 + (c & 7) * 16) = zero;
+      for (int c = 0; c < VALUE_CHUNKS; ++c) *reinterpret_cast<uint4*>(t + V_OFFSET + (c >> 3) * HALF_BYTES + lane * 128 + (c & 7) * 16) = zero;
     }
     __syncwarp();
     if (w_tok_hi >= w_tok_lo && first_key <= w_p_hi && first_key + KB > w_first_key) {
@@ -636,11 +720,40 @@ prefill_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_consta
   st.l[0] += __shfl_xor_sync(0xffffffffu, st.l[0], 1); st.l[0] += __shfl_xor_sync(0xffffffffu, st.l[0], 2);
   st.l[1] += __shfl_xor_sync(0xffffffffu, st.l[1], 1); st.l[1] += __shfl_xor_sync(0xffffffffu, st.l[1], 2);
   const int t2 = (lane & 3) * 2;
+  if constexpr (kDiff) {
+    // a head's two maps are neighbouring rows of the tile: rows g and g ^ 1, that is lanes 4 apart
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const float inv = st.l[h] > 0.0f ? 1.0f / st.l[h] : 0.0f;
+      const float w = (g & 1) ? -sf.diff_lambda * inv : inv;
+      float ss = 0.0f;
+#pragma unroll
+      for (int dn = 0; dn < DV / 8; ++dn) {
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const float mine = st.o[dn][2 * h + e] * w;
+          const float o = mine + __shfl_xor_sync(0xffffffffu, mine, 4);
+          st.o[dn][2 * h + e] = o;
+          ss = fmaf(o, o, ss);
+        }
+      }
+      ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+      ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+      if (tok_of[h] < 0 || (g & 1)) continue;
+      const float f = sf.diff_gain / sqrtf(ss / static_cast<float>(DV) + sf.diff_eps);
+      const int head = (head0 + (g + 8 * h) % group) / 2;
+      bf16* dst = out + (static_cast<size_t>(q_begin + tok0 + tok_of[h]) * (nh / 2) + head) * DV;
+#pragma unroll
+      for (int dn = 0; dn < DV / 8; ++dn)
+        *reinterpret_cast<uint32_t*>(dst + dn * 8 + t2) = pack_bf16(st.o[dn][2 * h] * f, st.o[dn][2 * h + 1] * f);
+    }
+    return;
+  }
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
     if (tok_of[h] < 0) continue;
     const int head = head0 + (g + 8 * h) % group;
-    bf16* dst = out + (static_cast<size_t>(q_begin + tok0 + tok_of[h]) * nh + head) * (kShared ? sf.out_width : D) +
+    bf16* dst = out + (static_cast<size_t>(q_begin + tok0 + tok_of[h]) * nh + head) * (kShared ? sf.out_width : DV) +
                 (kShared ? sf.out_col0 : 0);
     const float l = with_sink(sf, head, st.m[h], st.l[h]);
     const float inv = l > 0.0f ? 1.0f / l : 0.0f;
@@ -670,11 +783,11 @@ typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t,
                                   const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
                                   CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
 
-// Writes into `out_map` (128 bytes) the TMA descriptor of one cache tensor [pages + 1, kv_heads, page_size, D]
-// seen as a matrix of `rows` = (pages + 1) * kv_heads * page_size rows of D bfloat16, fetched in boxes of
-// `box_rows` rows x 64 columns with the 128-byte swizzle.  Columns beyond D read as zeros.
-B200_EXPORT int b200_kv_tensor_map(void* out_map, const void* cache, long long rows, int box_rows) {
-  if (rows <= 0 || box_rows <= 0 || box_rows > 256) return B200_BAD_SIZE;
+// Writes into `out_map` (128 bytes) the TMA descriptor of one cache tensor [pages + 1, kv_heads, page_size, width]
+// seen as a matrix of `rows` = (pages + 1) * kv_heads * page_size rows of `width` bfloat16, fetched in boxes of
+// `box_rows` rows x 64 columns with the 128-byte swizzle.  Columns beyond the width read as zeros.
+B200_EXPORT int b200_kv_tensor_map(void* out_map, const void* cache, long long rows, int width, int box_rows) {
+  if (width <= 0 || width % 8 != 0 || rows <= 0 || box_rows <= 0 || box_rows > 256) return B200_BAD_SIZE;
   if (reinterpret_cast<uintptr_t>(cache) % 16 != 0) return B200_BAD_ALIGN;
   static EncodeTiledFn encode = nullptr;
   if (encode == nullptr) {
@@ -686,8 +799,8 @@ B200_EXPORT int b200_kv_tensor_map(void* out_map, const void* cache, long long r
     encode = reinterpret_cast<EncodeTiledFn>(fn);
   }
   CUtensorMap map;
-  const cuuint64_t dims[2] = {static_cast<cuuint64_t>(D), static_cast<cuuint64_t>(rows)};
-  const cuuint64_t strides[1] = {static_cast<cuuint64_t>(D) * sizeof(bf16)};
+  const cuuint64_t dims[2] = {static_cast<cuuint64_t>(width), static_cast<cuuint64_t>(rows)};
+  const cuuint64_t strides[1] = {static_cast<cuuint64_t>(width) * sizeof(bf16)};
   const cuuint32_t box[2] = {64u, static_cast<cuuint32_t>(box_rows)};
   const cuuint32_t elem_strides[2] = {1u, 1u};
   CUresult r = encode(&map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(cache), dims, strides, box, elem_strides,
@@ -698,8 +811,8 @@ B200_EXPORT int b200_kv_tensor_map(void* out_map, const void* cache, long long r
   return 0;
 }
 
-static ScoreForm score_form(float scale, float softcap, int split_p, int chunk, const float* sinks, int v_col0 = 0,
-                            int out_width = D, int out_col0 = 0) {
+static ScoreForm score_form(float scale, float softcap, int split_p, int chunk, const float* sinks, int v_col0,
+                            int out_width, int out_col0, const float* diff) {
   ScoreForm sf;
   sf.scale_log2 = scale * 1.4426950408889634f;
   sf.tanh_in = softcap > 0.0f ? scale / softcap : 0.0f;
@@ -710,6 +823,9 @@ static ScoreForm score_form(float scale, float softcap, int split_p, int chunk, 
   sf.v_col0 = v_col0;
   sf.out_width = out_width;
   sf.out_col0 = out_col0;
+  sf.diff_lambda = diff != nullptr ? diff[0] : 0.0f;
+  sf.diff_gain = diff != nullptr ? diff[1] : 0.0f;
+  sf.diff_eps = diff != nullptr ? diff[2] : 0.0f;
   return sf;
 }
 
@@ -721,8 +837,10 @@ B200_EXPORT int b200_decode_attention_mma(const void* q, const void* k_map, cons
                                           const int* cu_q, const int* kv_len, const int* rows, int n_rows, int nh,
                                           int nkv, int page_size, int window, float scale, int splits,
                                           float softcap, int split_p, int chunk, const float* sinks, int v_col0,
-                                          int out_width, int out_col0, int* err, cudaStream_t stream) {
+                                          int out_width, int out_col0, const float* diff, int* err,
+                                          cudaStream_t stream) {
   if (n_rows <= 0) return 0;
+  if (kDiff && (diff == nullptr || sinks != nullptr || (nkv > 0 && (nh / nkv) % 2 != 0))) return B200_BAD_SIZE;
   if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || nh / nkv > QROWS || page_size <= 0 || splits <= 0) return B200_BAD_SIZE;
   if ((page_size & (page_size - 1)) != 0) return B200_BAD_SIZE;
   const int box_rows = page_size < KB ? page_size : KB;
@@ -758,17 +876,23 @@ B200_EXPORT int b200_decode_attention_mma(const void* q, const void* k_map, cons
   int rc = b200_launch(kernel, grid, dim3(kWarps * 32), smem, stream, cluster_merge ? splits : 0,
                        kmap, vmap, static_cast<const bf16*>(q), static_cast<bf16*>(out), part_acc, part_ml, block_table,
                        table_stride, cu_q, kv_len, rows, nh, nkv, page_size, box_rows, window,
-                       score_form(scale, softcap, split_p, chunk, sinks, v_col0, kShared ? out_width : D, kShared ? out_col0 : 0), cluster_merge ? 1 : 0, err);
+                       score_form(scale, softcap, split_p, chunk, sinks, v_col0, kShared ? out_width : DV, kShared ? out_col0 : 0, diff),
+                       cluster_merge ? 1 : 0, err);
   if (rc != 0 || splits == 1 || cluster_merge) return rc;
+  if constexpr (kDiff) {
+    return b200_launch(decode_mma_merge_diff_kernel, dim3(n_rows, nh / 2), dim3(DV >= 128 ? 128 : 64), 0, stream, 0,
+                       static_cast<bf16*>(out), static_cast<const float*>(part_acc), static_cast<const float*>(part_ml), cu_q,
+                       rows, nh, splits, diff[0], diff[1], diff[2]);
+  }
   dim3 mgrid(n_rows, nh);
-  return b200_launch(decode_mma_merge_kernel, mgrid, dim3(D >= 128 ? 128 : 64), 0, stream, 0, static_cast<bf16*>(out),
+  return b200_launch(decode_mma_merge_kernel, mgrid, dim3(DV >= 128 ? 128 : 64), 0, stream, 0, static_cast<bf16*>(out),
                      static_cast<const float*>(part_acc), static_cast<const float*>(part_ml), cu_q, rows, nh, splits, sinks,
-                     kShared ? out_width : D, kShared ? out_col0 : 0);
+                     kShared ? out_width : DV, kShared ? out_col0 : 0);
 }
 
 constexpr size_t kPfQBytes = PF_ROWS * LD * sizeof(bf16);
 constexpr size_t kPfFixed = 1024 + kPfQBytes + kBarBytes;
-constexpr int kPfStages = D <= 128 ? 3 : kPfFixed + 4 * TILE_BYTES <= kSmemLimit ? 4 : (kPfFixed + 3 * TILE_BYTES <= kSmemLimit ? 3 : 2);
+constexpr int kPfStages = D <= 128 && DV <= 128 ? 3 : kPfFixed + 4 * TILE_BYTES <= kSmemLimit ? 4 : (kPfFixed + 3 * TILE_BYTES <= kSmemLimit ? 3 : 2);
 static_assert(kPfFixed + kPfStages * TILE_BYTES <= kSmemLimit, "the key blocks must fit shared memory");
 
 // Portions of prompts over a bfloat16 cache; arguments as b200_prefill_attention of attention.cu, with the
@@ -778,8 +902,10 @@ B200_EXPORT int b200_prefill_attention_mma(const void* q, const void* k_map, con
                                            const int* kv_len, const int* prefix_len, const int* rows, int n_rows,
                                            int max_q_len, int nh, int nkv, int page_size, int window, float scale,
                                            float softcap, int split_p, int chunk, const float* sinks, int v_col0,
-                                          int out_width, int out_col0, int* err, cudaStream_t stream) {
+                                           int out_width, int out_col0, const float* diff, int* err,
+                                           cudaStream_t stream) {
   if (n_rows <= 0 || max_q_len <= 0) return 0;
+  if (kDiff && (diff == nullptr || sinks != nullptr || (nkv > 0 && (nh / nkv) % 2 != 0))) return B200_BAD_SIZE;
   if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || nh / nkv > QROWS || page_size <= 0) return B200_BAD_SIZE;
   if ((page_size & (page_size - 1)) != 0) return B200_BAD_SIZE;
   const int box_rows = page_size < KB ? page_size : KB;
@@ -801,6 +927,7 @@ B200_EXPORT int b200_prefill_attention_mma(const void* q, const void* k_map, con
   dim3 grid(nkv, n_rows, n_tiles);
   kernel<<<grid, PF_WARPS * 32, smem, stream>>>(
       kmap, vmap, static_cast<const bf16*>(q), static_cast<bf16*>(out), block_table, table_stride, cu_q, kv_len,
-      prefix_len, rows, nh, nkv, page_size, box_rows, window, score_form(scale, softcap, split_p, chunk, sinks, v_col0, kShared ? out_width : D, kShared ? out_col0 : 0), err);
+      prefix_len, rows, nh, nkv, page_size, box_rows, window, score_form(scale, softcap, split_p, chunk, sinks, v_col0, kShared ? out_width : DV, kShared ? out_col0 : 0, diff),
+      err);
   return b200_check_launch();
 }

@@ -13,7 +13,7 @@ import ctypes
 import gc
 import os
 import sys
-from typing import Optional
+from typing import Optional, Tuple
 
 import torch
 
@@ -323,20 +323,27 @@ def prefill_attention(q, k_cache, v_cache, out, block_table, cu_q, kv_len, prefi
                       max_q_len, num_heads, num_kv_heads, head_dim, page_size, window, scale,
                       tiles_per_cta: int = 0, v_head_dim: Optional[int] = None, softcap: float = 0.0,
                       precise_weights: bool = False, chunk: Optional[int] = None,
-                      sinks: Optional[torch.Tensor] = None, shared_values: bool = False) -> None:
+                      sinks: Optional[torch.Tensor] = None, shared_values: bool = False,
+                      difference: Optional[Tuple[float, float, float]] = None) -> None:
     """Causal attention of prompt portions over the paged cache (rows: which batch rows).
 
     ``v_head_dim``: the width of a value (and of an output) vector where it differs from a key's;
     ``softcap`` > 0: a score becomes cap * tanh(score / cap) before the mask; ``precise_weights``: the softmax
-    weights enter the product with the values as two bfloat16 terms (about 16 bits) instead of one.  Values of
-    another width than keys take the all-sizes kernel, whose weights are floats; a soft-cap or precise weights take
-    the mma.sync kernel, not the tcgen05 one (whose weights are single bfloat16 numbers in tensor memory).
+    weights enter the product with the values as two bfloat16 terms (about 16 bits) instead of one.  A soft-cap, precise
+    weights and values of another width than keys take the mma.sync kernel (see ``decode_uses_tensor_cores``), not the
+    tcgen05 one (whose weights are single bfloat16 numbers in tensor memory); what that does not take goes to the
+    all-sizes kernel, whose weights are floats.
 
     ``chunk`` C: a query at position p sees only keys from p - p % C on (its own block of C positions, counted from
     the sequence's start); ``sinks`` (float32, one per query head): exp(sink) joins the softmax's denominator.  Both
     are served by the mma.sync and the all-sizes kernels, not by the tcgen05 one.  ``shared_values``: one KV head
     whose values are the first ``v_head_dim`` columns of the key rows (``v_cache`` is not read and may be None): the
     mma.sync kernels fetch a block's rows once for both products and take the values in column tiles.
+
+    ``difference`` (lambda, gain, eps): query heads come in pairs, the two maps of one head, and ``out`` [tokens,
+    num_heads / 2 * v_head_dim] receives a_1 - lambda a_2, every head's vector divided by its root mean square (eps inside
+    the root), times gain.  Only where ``fuses_difference`` says so; else the pairs' outputs are taken from here and
+    ``head_difference`` makes the rest.
 
     ``tiles_per_cta`` (head size 128 on the tcgen05 kernel only): 1 or 2 tiles of 128 query vectors per
     CTA, 0 lets the kernel's launcher choose by the size of the grid."""
@@ -355,23 +362,23 @@ def prefill_attention(q, k_cache, v_cache, out, block_table, cu_q, kv_len, prefi
             raise KernelError("values that are columns of the key rows need one KV head")
         if latent_uses_tensor_cores(q.dtype, num_heads, head_dim, dv, page_size):
             tile, group = shared_value_tile(dv), latent_head_group(num_heads)
-            lib = _attention_mma(head_dim, tile)
+            lib = _attention_mma(head_dim, shared_tile=tile)
             kmap = kv_tensor_map(k_cache, min(page_size, 32), lib)
             for col0 in range(0, dv, tile):
                 rc = lib.b200_prefill_attention_mma(
                     _p(q), kmap, kmap, _p(out), _p(block_table), block_table.shape[-1], _p(cu_q), _p(kv_len),
                     _p(prefix_len), _p(rows), n_rows, max_q_len, num_heads, num_heads // group, page_size,
                     int(window or 0), ctypes.c_float(scale), ctypes.c_float(cap), int(bool(precise_weights)),
-                    int(chunk or 0), _p(sinks), col0, dv, col0, _p(error_word(q.device)), _stream())
+                    int(chunk or 0), _p(sinks), col0, dv, col0, None, _p(error_word(q.device)), _stream())
                 _ok(rc, "prefill_attention_mma_shared")
             return
         v_cache = k_cache
-    if not shared_values and dv == head_dim and decode_uses_tensor_cores(q.dtype, num_heads, num_kv_heads, head_dim, page_size):
-        if k_cache.shape[1] != num_kv_heads or k_cache.shape[2] != page_size:
-            raise KernelError("the cache must be [pages + 1, kv_heads, page_size, head_dim]")
+    if not shared_values and decode_uses_tensor_cores(q.dtype, num_heads, num_kv_heads, head_dim, page_size, dv):
+        _check_cache(k_cache, v_cache, num_kv_heads, page_size, head_dim, dv)
+        _check_difference(difference, q, out, num_heads, num_kv_heads, dv, sinks)
         box_rows = min(page_size, 32)
         group = num_heads // num_kv_heads
-        if head_dim == 128 and 128 % group == 0 and max_q_len * group >= 128 and not cap > 0.0 and not precise_weights \
+        if head_dim == 128 and dv == 128 and difference is None and 128 % group == 0 and max_q_len * group >= 128 and not cap > 0.0 and not precise_weights \
                 and plain_mask:
             # head size 128 and at least one full tile of 128 query vectors: the tcgen05 kernel
             rc = load_cuda_library("attention_tcgen05.cu").b200_prefill_attention_tcgen05(
@@ -381,19 +388,40 @@ def prefill_attention(q, k_cache, v_cache, out, block_table, cu_q, kv_len, prefi
                 _p(error_word(q.device)), _stream())
             _ok(rc, "prefill_attention_tcgen05")
             return
-        rc = _attention_mma(head_dim).b200_prefill_attention_mma(
+        rc = _attention_mma(head_dim, dv, difference is not None).b200_prefill_attention_mma(
             _p(q), kv_tensor_map(k_cache, box_rows), kv_tensor_map(v_cache, box_rows), _p(out), _p(block_table),
             block_table.shape[-1], _p(cu_q), _p(kv_len), _p(prefix_len), _p(rows), n_rows, max_q_len, num_heads,
             num_kv_heads, page_size, int(window or 0), ctypes.c_float(scale), ctypes.c_float(cap),
-            int(bool(precise_weights)), int(chunk or 0), _p(sinks), 0, 0, 0, _p(error_word(q.device)), _stream())
+            int(bool(precise_weights)), int(chunk or 0), _p(sinks), 0, 0, 0, _floats(difference),
+            _p(error_word(q.device)), _stream())
         _ok(rc, "prefill_attention_mma")
         return
+    if difference is not None:
+        raise KernelError("the all-sizes attention kernel leaves the difference of two maps to head_difference")
     rc = _attention(max(head_dim, dv)).b200_prefill_attention(
         _p(q), _p(k_cache), _p(v_cache), _p(out), _p(block_table), block_table.shape[-1], _p(cu_q),
         _p(kv_len), _p(prefix_len), _p(rows), n_rows, max_q_len, num_heads, num_kv_heads, page_size,
         int(window or 0), ctypes.c_float(scale), _code(q), head_dim, dv, ctypes.c_float(cap), int(chunk or 0),
         _p(sinks), head_dim if shared_values else 0, _stream())
     _ok(rc, "prefill_attention")
+
+
+def _check_cache(k_cache, v_cache, num_kv_heads, page_size, head_dim, v_head_dim) -> None:
+    for cache, width in ((k_cache, head_dim), (v_cache, v_head_dim)):
+        if tuple(cache.shape[1:]) != (num_kv_heads, page_size, width):
+            raise KernelError("the cache must be [pages + 1, kv_heads, page_size, width]")
+
+
+def _check_difference(difference, q, out, num_heads, num_kv_heads, v_head_dim, sinks) -> None:
+    if difference is None:
+        return
+    if (num_heads // num_kv_heads) % 2 or sinks is not None or out.shape[-1] * 2 != num_heads * v_head_dim:
+        raise KernelError("a difference of maps needs pairs of query heads, no sinks and an output half as many heads wide")
+
+
+def _floats(values):
+    """A few floats as a C array (None: a null pointer)."""
+    return None if values is None else (ctypes.c_float * len(values))(*[float(v) for v in values])
 
 
 def _check_sinks(sinks: Optional[torch.Tensor], num_heads: int) -> None:
@@ -405,12 +433,19 @@ MMA_MAX_GROUP = 16
 MMA_MAX_HEAD_DIM = 256
 
 
-def _attention_mma(head_dim: int, shared_value_tile: Optional[int] = None):
-    """The tensor-core attention library for a head size; ``shared_value_tile``: the form whose values are a range of
-    that many columns of the key rows."""
-    if shared_value_tile:
-        return load_cuda_library("attention_mma.cu", {"HEAD_DIM": head_dim, "V_DIM": shared_value_tile, "V_SHARED": 1})
-    return load_cuda_library("attention_mma.cu", {"HEAD_DIM": head_dim})
+def _attention_mma(head_dim: int, v_head_dim: Optional[int] = None, difference: bool = False,
+                   shared_tile: Optional[int] = None):
+    """The tensor-core attention library for a key width and a value width (None: the same); ``shared_tile``: the form
+    whose values are a range of that many columns of the key rows; ``difference``: the form that stores the difference of
+    two maps."""
+    defines = {"HEAD_DIM": head_dim}
+    if shared_tile:
+        defines.update(V_DIM=shared_tile, V_SHARED=1)
+    elif v_head_dim is not None and v_head_dim != head_dim:
+        defines["V_DIM"] = v_head_dim
+    if difference:
+        defines["DIFF"] = 1
+    return load_cuda_library("attention_mma.cu", defines)
 
 
 def shared_value_tile(value_dim: int) -> int:
@@ -432,12 +467,18 @@ def latent_uses_tensor_cores(dtype: torch.dtype, num_heads: int, key_dim: int, v
 
 
 def decode_uses_tensor_cores(dtype: torch.dtype, num_heads: int, num_kv_heads: int, head_dim: int,
-                             page_size: int) -> bool:
-    """bfloat16 caches with at most 16 query heads per KV head, heads up to 256 wide and a page size
-    that is a power of two take the TMA / tensor-core kernel; everything else the all-sizes kernel."""
+                             page_size: int, v_head_dim: Optional[int] = None) -> bool:
+    """bfloat16 caches with at most 16 query heads per KV head, keys and values up to 256 wide (multiples of 16) and a
+    page size that is a power of two take the TMA / tensor-core kernel; everything else the all-sizes kernel."""
     return (dtype == torch.bfloat16 and num_heads // num_kv_heads <= MMA_MAX_GROUP
-            and head_dim <= MMA_MAX_HEAD_DIM and head_dim % 16 == 0
+            and all(0 < w <= MMA_MAX_HEAD_DIM and w % 16 == 0 for w in (head_dim, v_head_dim or head_dim))
             and page_size > 0 and page_size & (page_size - 1) == 0)
+
+
+def fuses_difference(dtype: torch.dtype, num_heads: int, num_kv_heads: int, head_dim: int, page_size: int,
+                     v_head_dim: int) -> bool:
+    """Whether attention itself stores the difference of a head's two maps (``num_heads`` counts query vectors)."""
+    return decode_uses_tensor_cores(dtype, num_heads, num_kv_heads, head_dim, page_size, v_head_dim)
 
 
 _kv_maps = {}
@@ -452,7 +493,8 @@ def kv_tensor_map(cache: torch.Tensor, box_rows: int, lib=None):
             raise KernelError("a TMA descriptor needs a contiguous bfloat16 cache [pages + 1, kv_heads, page_size, head_dim]")
         buf = ctypes.create_string_buffer(128)
         rows = cache.shape[0] * cache.shape[1] * cache.shape[2]
-        rc = (lib or _attention_mma(cache.shape[3])).b200_kv_tensor_map(buf, _p(cache), ctypes.c_longlong(rows), box_rows)
+        rc = (lib or _attention_mma(cache.shape[3])).b200_kv_tensor_map(buf, _p(cache), ctypes.c_longlong(rows),
+                                                                        cache.shape[3], box_rows)
         if rc != 0:
             raise KernelError(f"the TMA descriptor of a cache tensor could not be made (code {rc})")
         if len(_kv_maps) > 4096:
@@ -462,10 +504,10 @@ def kv_tensor_map(cache: torch.Tensor, box_rows: int, lib=None):
 
 
 def decode_ctas_per_split(dtype: torch.dtype, n_rows: int, num_heads: int, num_kv_heads: int, head_dim: int,
-                          page_size: int, plain: bool = True) -> int:
-    """CTAs that the decode kernel launches for each split of the keys (``plain``: values as wide as keys, the
-    case the tensor-core kernel takes)."""
-    if plain and decode_uses_tensor_cores(dtype, num_heads, num_kv_heads, head_dim, page_size):
+                          page_size: int, v_head_dim: Optional[int] = None) -> int:
+    """CTAs that the decode kernel launches for each split of the keys (``v_head_dim``: the width of a value where it
+    differs from a key's)."""
+    if decode_uses_tensor_cores(dtype, num_heads, num_kv_heads, head_dim, page_size, v_head_dim):
         return n_rows * num_kv_heads
     return n_rows * num_kv_heads * ((num_heads // num_kv_heads + 3) // 4)
 
@@ -479,9 +521,10 @@ def decode_attention(q, k_cache, v_cache, out, scratch, block_table, cu_q, kv_le
                      num_heads, num_kv_heads, head_dim, page_size, window, scale, splits,
                      v_head_dim: Optional[int] = None, softcap: float = 0.0, precise_weights: bool = False,
                      chunk: Optional[int] = None, sinks: Optional[torch.Tensor] = None,
-                     shared_values: bool = False) -> None:
+                     shared_values: bool = False, difference: Optional[Tuple[float, float, float]] = None) -> None:
     """Attention of single decoded tokens, the keys split over ``splits`` blocks per row (``v_head_dim``,
-    ``softcap``, ``precise_weights``, ``chunk``, ``sinks``, ``shared_values``: see ``prefill_attention``)."""
+    ``softcap``, ``precise_weights``, ``chunk``, ``sinks``, ``shared_values``, ``difference``: see
+    ``prefill_attention``)."""
     _cuda(q, k_cache, v_cache, out, scratch, block_table, cu_q, kv_len, rows, sinks)
     _contig(q, k_cache, v_cache, out, block_table, scratch, sinks)
     _check_sinks(sinks, num_heads)
@@ -490,7 +533,6 @@ def decode_attention(q, k_cache, v_cache, out, scratch, block_table, cu_q, kv_le
     if k_cache.dtype != q.dtype or out.dtype != q.dtype:
         raise KernelError("q, cache and output must share a dtype")
     dv = int(v_head_dim or head_dim)
-    plain = dv == head_dim and not shared_values
     need = decode_scratch_floats(n_rows, num_heads, max(head_dim, dv), splits)
     if need and (scratch is None or scratch.dtype != torch.float32 or scratch.numel() < need):
         raise KernelError(f"decode attention needs {need} floats of scratch")
@@ -499,7 +541,7 @@ def decode_attention(q, k_cache, v_cache, out, scratch, block_table, cu_q, kv_le
             raise KernelError("values that are columns of the key rows need one KV head")
         if latent_uses_tensor_cores(q.dtype, num_heads, head_dim, dv, page_size):
             tile, group = shared_value_tile(dv), latent_head_group(num_heads)
-            lib = _attention_mma(head_dim, tile)
+            lib = _attention_mma(head_dim, shared_tile=tile)
             kmap = kv_tensor_map(k_cache, min(page_size, 32), lib)
             groups = num_heads // group
             in_kernel = splits == 1 or (splits in (2, 4, 8) and splits * groups * n_rows <= _sm_count(q.device))
@@ -508,22 +550,24 @@ def decode_attention(q, k_cache, v_cache, out, scratch, block_table, cu_q, kv_le
                     _p(q), kmap, kmap, _p(out), _p(scratch), _p(block_table), block_table.shape[-1], _p(cu_q),
                     _p(kv_len), _p(rows), n_rows, num_heads, groups, page_size, int(window or 0),
                     ctypes.c_float(scale), splits, ctypes.c_float(softcap or 0.0), int(bool(precise_weights)),
-                    int(chunk or 0), _p(sinks), col0, dv, col0, _p(error_word(q.device)), _stream())
+                    int(chunk or 0), _p(sinks), col0, dv, col0, None, _p(error_word(q.device)), _stream())
                 _ok(rc, "decode_attention_mma_shared", 1 if in_kernel else 2)
             return
         v_cache = k_cache
-    if plain and decode_uses_tensor_cores(q.dtype, num_heads, num_kv_heads, head_dim, page_size):
-        if k_cache.shape[1] != num_kv_heads or k_cache.shape[2] != page_size:
-            raise KernelError("the cache must be [pages + 1, kv_heads, page_size, head_dim]")
+    if not shared_values and decode_uses_tensor_cores(q.dtype, num_heads, num_kv_heads, head_dim, page_size, dv):
+        _check_cache(k_cache, v_cache, num_kv_heads, page_size, head_dim, dv)
+        _check_difference(difference, q, out, num_heads, num_kv_heads, dv, sinks)
         box_rows = min(page_size, 32)
-        rc = _attention_mma(head_dim).b200_decode_attention_mma(
+        rc = _attention_mma(head_dim, dv, difference is not None).b200_decode_attention_mma(
             _p(q), kv_tensor_map(k_cache, box_rows), kv_tensor_map(v_cache, box_rows), _p(out), _p(scratch), _p(block_table), block_table.shape[-1],
             _p(cu_q), _p(kv_len), _p(rows), n_rows, num_heads, num_kv_heads, page_size, int(window or 0),
             ctypes.c_float(scale), splits, ctypes.c_float(softcap or 0.0), int(bool(precise_weights)),
-            int(chunk or 0), _p(sinks), 0, 0, 0, _p(error_word(q.device)), _stream())
+            int(chunk or 0), _p(sinks), 0, 0, 0, _floats(difference), _p(error_word(q.device)), _stream())
         in_kernel = splits == 1 or (splits in (2, 4, 8) and splits * num_kv_heads * n_rows <= _sm_count(q.device))
         _ok(rc, "decode_attention_mma", 1 if in_kernel else 2)      # (a cluster of 2, 4 or 8 splits combines them itself)
         return
+    if difference is not None:
+        raise KernelError("the all-sizes attention kernel leaves the difference of two maps to head_difference")
     rc = _attention(max(head_dim, dv)).b200_decode_attention(
         _p(q), _p(k_cache), _p(v_cache), _p(out), _p(scratch), _p(block_table), block_table.shape[-1],
         _p(cu_q), _p(kv_len), _p(rows), n_rows, num_heads, num_kv_heads, page_size, int(window or 0),

@@ -232,8 +232,7 @@ class GatedConvAttention(Part):
                                   v_head_dim=self.dv, softcap=self.softcap, precise_weights=True)
         if ctx.num_decode:
             bound = min(ctx.kv_len_bound, self.window) if self.window else ctx.kv_len_bound
-            plain = self.dv == self.d
-            per_split = ops.decode_ctas_per_split(q.dtype, ctx.num_decode, self.nh, self.nkv, self.d, page, plain)
+            per_split = ops.decode_ctas_per_split(q.dtype, ctx.num_decode, self.nh, self.nkv, self.d, page, self.dv)
             splits = decode_splits(per_split, bound, ctx.sm_count)
             need = ops.decode_scratch_floats(ctx.num_decode, self.nh, max(self.d, self.dv), splits)
             scratch = ctx.scratch(need) if need else None
@@ -247,10 +246,11 @@ class GatedConvAttention(Part):
 
 
 def _masked_attention(part, q, out, ctx, cache, num_heads, num_kv_heads, head_dim, v_head_dim, sinks,
-                      shared_values=False):
+                      shared_values=False, difference=None):
     """Attention of a step's rows over the paged cache for a mixer with ``window``, ``chunk``, ``scale`` and ``softcap``:
     prompt portions and single decoded tokens, softmax weights in float.  ``shared_values``: a value is the first
-    ``v_head_dim`` columns of its key's row (one KV head)."""
+    ``v_head_dim`` columns of its key's row (one KV head).  ``difference``: query heads are pairs of maps and ``out`` holds
+    their differences (see ``ops.prefill_attention``)."""
     g = cache.group
     page = ctx.page_sizes[g]
     if ctx.num_prefill:
@@ -258,26 +258,26 @@ def _masked_attention(part, q, out, ctx, cache, num_heads, num_kv_heads, head_di
                               ctx.prefix_len, ctx.prefill_rows, ctx.num_prefill, ctx.max_q_len,
                               num_heads, num_kv_heads, head_dim, page, part.window, part.scale,
                               v_head_dim=v_head_dim, softcap=part.softcap, precise_weights=True, chunk=part.chunk,
-                              sinks=sinks, shared_values=shared_values)
+                              sinks=sinks, shared_values=shared_values, difference=difference)
     if ctx.num_decode:
         bound = ctx.kv_len_bound
         for limit in (part.window, part.chunk):
             if limit:
                 bound = min(bound, limit)
-        plain = v_head_dim == head_dim
         keys_per_cta = _KEYS_PER_CTA_AT_LEAST
         if shared_values and ops.latent_uses_tensor_cores(q.dtype, num_heads, head_dim, v_head_dim, page):
             per_split = ctx.num_decode * (num_heads // ops.latent_head_group(num_heads))
             keys_per_cta = _LATENT_KEYS_PER_CTA_AT_LEAST
         else:
-            per_split = ops.decode_ctas_per_split(q.dtype, ctx.num_decode, num_heads, num_kv_heads, head_dim, page, plain)
+            per_split = ops.decode_ctas_per_split(q.dtype, ctx.num_decode, num_heads, num_kv_heads, head_dim, page, v_head_dim)
         splits = decode_splits(per_split, bound, ctx.sm_count, keys_per_cta)
         need = ops.decode_scratch_floats(ctx.num_decode, num_heads, max(head_dim, v_head_dim), splits)
         scratch = ctx.scratch(need) if need else None
         ops.decode_attention(q, cache.k, cache.v, out, scratch, ctx.block_tables[g], ctx.cu_q,
                              ctx.kv_len, ctx.decode_rows, ctx.num_decode, num_heads, num_kv_heads, head_dim,
                              page, part.window, part.scale, splits, v_head_dim=v_head_dim, softcap=part.softcap,
-                             precise_weights=True, chunk=part.chunk, sinks=sinks, shared_values=shared_values)
+                             precise_weights=True, chunk=part.chunk, sinks=sinks, shared_values=shared_values,
+                             difference=difference)
 
 
 class GroupedAttention(Part):
@@ -477,7 +477,8 @@ class DifferentialAttention(Part):
 
     The two keys of a head are one cache row 2 ``head_dim`` wide, and a query vector is a row of that width with zeros
     beside its own map's columns: to the attention kernels it is grouped-query attention with 2 ``num_heads`` query
-    heads, so keys and values are fetched once for both maps."""
+    heads, so keys and values are fetched once for both maps; where they take the size, they store the normed difference
+    themselves (``ops.fuses_difference``)."""
     category = "mixer"
 
     def __init__(self, spec, env):
@@ -548,9 +549,15 @@ class DifferentialAttention(Part):
                           inv_freq=rope.inv_freq if rope else None, rot_dims=self.rot_dims if rope else 0,
                           interleaved=getattr(rope, "pairing", "half_split") == "interleaved", maps=2,
                           rot_gain=float(getattr(rope, "gain", 1.0)))
-        maps = torch.empty((tokens, 2 * self.nh * self.dv), dtype=packed.dtype, device=packed.device)
-        _masked_attention(self, q, maps, ctx, cache, 2 * self.nh, self.nkv, 2 * self.d, self.dv, None)
-        out = ops.head_difference(maps, self.nh, self.dv, self._lambda, 1.0 - self.diff, self.eps)
+        sizes = (2 * self.nh, self.nkv, 2 * self.d)
+        if ops.fuses_difference(q.dtype, *sizes, ctx.page_sizes[cache.group], self.dv):
+            out = torch.empty((tokens, self.nh * self.dv), dtype=packed.dtype, device=packed.device)
+            _masked_attention(self, q, out, ctx, cache, *sizes, self.dv, None,
+                              difference=(self._lambda, 1.0 - self.diff, self.eps))
+        else:
+            maps = torch.empty((tokens, 2 * self.nh * self.dv), dtype=packed.dtype, device=packed.device)
+            _masked_attention(self, q, maps, ctx, cache, *sizes, self.dv, None)
+            out = ops.head_difference(maps, self.nh, self.dv, self._lambda, 1.0 - self.diff, self.eps)
         y = ops.linear(out, p["o_proj"])
         if self.out_bias and not self.bias_deferred:
             ops.add_row_bias(y, p["o_bias"])

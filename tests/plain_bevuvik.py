@@ -72,6 +72,12 @@ def yarn(dims: int, base: float, scaling: Optional[dict]):
     return torch.tensor(out, dtype=torch.float64), 0.1 * math.log(factor) + 1.0
 
 
+def rotation(m: dict):
+    """(frequencies, gain) of a mixer's rotation (none: no coordinate is turned)."""
+    r = m.get("rot")
+    return yarn(r["dims"], r["base"], r.get("scaling")) if r else (torch.zeros(0, dtype=torch.float64), 1.0)
+
+
 def rotate(x: torch.Tensor, freq: torch.Tensor, gain: float, interleaved: bool) -> torch.Tensor:
     """x [T, heads, d] at positions 0..T-1: the first 2 len(freq) coordinates of every head are turned."""
     T, n = x.shape[0], len(freq)
@@ -119,7 +125,7 @@ def differential_attention(h: torch.Tensor, w: Dict[str, torch.Tensor], p: str, 
     q = (h @ w[p + "q"].T + w[p + "q.b"]).reshape(T, H, 2, d)
     k = (h @ w[p + "k"].T + w[p + "k.b"]).reshape(T, G, 2, d)
     v = (h @ w[p + "v"].T + w[p + "v.b"]).reshape(T, G, dv)
-    freq, gain = yarn(m["rot"]["dims"], m["rot"]["base"], m["rot"].get("scaling"))
+    freq, gain = rotation(m)
     mask = window_mask(T, m["mask"]["size"] if m.get("mask") else None)
     a = [softmax_attention(rotate(q[:, :, i], freq, gain, True), rotate(k[:, :, i], freq, gain, True), v, m["scale"], mask)
          for i in range(2)]
@@ -130,11 +136,11 @@ def differential_attention(h: torch.Tensor, w: Dict[str, torch.Tensor], p: str, 
 def capped_attention(h: torch.Tensor, w: Dict[str, torch.Tensor], p: str, m: dict) -> torch.Tensor:
     T = h.shape[0]
     H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
-    freq = frequencies(m["rot"]["dims"], m["rot"]["base"])
+    freq, _ = rotation(m)
     q = rotate((h @ w[p + "q"].T).reshape(T, H, d), freq, 1.0, False)
     k = rotate((h @ w[p + "k"].T).reshape(T, G, d), freq, 1.0, False)
     v = (h @ w[p + "v"].T).reshape(T, G, dv)
-    a = softmax_attention(q, k, v, m["scale"], window_mask(T, None), m["softcap"])
+    a = softmax_attention(q, k, v, m["scale"], window_mask(T, None), m.get("softcap"))
     return a.reshape(T, H * dv) @ w[p + "o"].T
 
 
