@@ -48,6 +48,10 @@ closest earlier design, and Qwen3.
 attention over a window beside a gated linear recurrent unit, experts weighted on their input, layer norms on the
 outputs), beside Kefetar, the closest earlier design, and Qwen3; its kernels also stand beside Torinex's.
 
+``--design bevuvik`` does the same for Bevuvik (differences of two attention maps over a window, soft-capped attention
+beside a delta rule with one decay a head, one norm for mixer and feed-forward, looped layers), beside Sigudra, the
+closest earlier design, and Qwen3; its kernels also stand beside Kefetar's, Lufizen's and Torinex's.
+
 Peaks come from MEASURED_PEAKS.json beside this file when it is there.  Weights are random
 (drawn on the device), token ids are synthetic.  One GPU only.
 """
@@ -1311,11 +1315,183 @@ def sigudra_kernel_table(size, peak):
     return out
 
 
+# ----------------------------------------------------------------------------- --design bevuvik
+def bevuvik_config(size, layers):
+    """Pairs (soft-capped attention beside a delta rule as many heads wide) and differential attention over a window in
+    turn, one pair to three; a head's two maps are half a head wide each, so that keys and values have the sizes of the
+    others.  The feed-forwards are as wide as Qwen3's.  Two of the layers are looped once more in place of two further ones:
+    as many layer runs as the others have layers."""
+    z = DESIGN_SIZES[size]
+    d, I = z["head_dim"], z["inter"]
+
+    def layer(i):
+        mlp = {"kind": "dense", "ff": I, "limit": 7.0}
+        if i % 4 == 0:
+            return {"type": "parallel", "mlp": mlp, "mixer": {
+                "left": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": d, "vdim": d, "scale": d ** -0.5, "softcap": 50.0,
+                         "rot": {"base": 1e6, "dims": d // 2}},
+                "right": {"heads": z["heads"], "kv_heads": z["heads"] // 2, "dim": d, "vdim": d, "conv": 4}}}
+        return {"type": "attention", "mlp": mlp, "mixer": {
+            "heads": z["heads"], "kv_heads": z["kv_heads"], "dim": d // 2, "vdim": d, "scale": (d // 2) ** -0.5, "diff": 0.4,
+            "rot": {"base": 1e6, "dims": d // 2, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}},
+            "mask": {"size": 1024}}}
+
+    raw = {"architecture": "Bevuvik", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5}, "residual_mult": 0.3}
+    if layers < 5:
+        return dict(raw, layers=[layer(i) for i in range(layers)])
+    return dict(raw, layers=[layer(i) for i in range(layers - 2)], loop={"start": 1, "stop": 3, "times": 2})
+
+
+def bevuvik_kernel_table(size, peak):
+    """Every kernel of Bevuvik alone, beside the like kernel of the closest designs (Sigudra's recurrence, norms and window
+    attention, Kefetar's soft-capped attention and per-head norm, Lufizen's prepare kernel, Sigudra's and Qwen3's
+    feed-forwards, Qwen3's projections), at one layer's sizes: a prompt portion of 2,048 tokens and a decode step of 8 rows
+    at 2,048 tokens.  ``frac`` as in ``kernel_table``; FLOPs of the delta rule: 8 d dv a token and head; of a difference of
+    maps: each map's scores and values once (2 d + 2 dv a pair and map), whatever the kernel does beside them."""
+    import types
+    import torch
+    from llm_infer_rust_b200.config.spec import PartSpec
+    from llm_infer_rust_b200.kernels import ops
+    from llm_infer_rust_b200.parts import BuildEnv, build_part
+    from llm_infer_rust_b200.parts.attention import decode_splits
+    z = DESIGN_SIZES[size]
+    W, nh, nkv, d, I = z["width"], z["heads"], z["kv_heads"], z["head_dim"], z["inter"]
+    window, taps, rank, rkv = 1024, 4, z["head_dim"], z["heads"] // 2
+    dev, bf = torch.device("cuda"), torch.bfloat16
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    page, ctx_len, rows_dec = 16, 2048, 8
+    out = {}
+
+    def put(name, us, nbytes=None, flops=None, of="bf16"):
+        rec = {"us": round(us, 2)}
+        if nbytes is not None:
+            rec["gb_s"] = round(nbytes / us / 1e3, 1)
+            rec["frac"] = round(nbytes / us / 1e3 / peak["hbm_gbs"], 3)
+        if flops is not None:
+            rec["tflops"] = round(flops / us / 1e6, 2)
+            rec["frac"] = round(flops / us / 1e6 / {"bf16": peak["bf16_tflops"], "fp32": peak["fp32_tflops"]}[of], 3)
+            rec["of"] = of
+        out[name] = rec
+
+    def step(rows):
+        cu, row_of, pos = [0], [], []
+        for i, (prefix, n) in enumerate(rows):
+            cu.append(cu[-1] + n)
+            row_of += [i] * n
+            pos += list(range(prefix, prefix + n))
+        R = len(rows)
+        width = -(-max(p + n for p, n in rows) // page)
+        table = torch.arange(1, R * width + 1, dtype=torch.int32, device=dev).view(R, width).contiguous()
+        slots = [int(table[i, (p + j) // page]) * page + (p + j) % page for i, (p, n) in enumerate(rows) for j in range(n)]
+        return types.SimpleNamespace(
+            num_rows=R, row_of_token=i32(row_of), cu_q=i32(cu), positions=i32(pos), prefix_len=i32([p for p, _ in rows]),
+            kv_len=i32([p + n for p, n in rows]), state_slots=i32(list(range(1, R + 1))), slots=i32(slots), table=table,
+            rows=i32(list(range(R))), tokens=cu[-1], pages=R * width + 1, max_q_len=max(n for _, n in rows),
+            num_prefill=sum(n > 1 for _, n in rows))
+
+    for phase, c in (("prefill", step([(0, ctx_len)])), ("decode", step([(ctx_len - 1, 1)] * rows_dec))):
+        T = c.tokens
+        rnd = lambda *shape, f=1.0: (torch.randn(*shape, device=dev) * f).to(bf)
+        few = 3 if phase == "prefill" else 7
+        # --- the owed sum and the norm behind it; a pass's first product
+        stream, y, y2, f, wn = torch.randn(T, W, device=dev), rnd(T, W), rnd(T, W), rnd(T, W), torch.ones(W, device=dev)
+        pair = ops.NormedPair(y, y2, wn, wn, 1e-5)
+        put(f"{phase}.bevuvik.residual_sum", timed_alone(lambda: ops.residual_sum(
+            stream, y=y, add=f, bias=wn, mult=0.3, weight=wn, eps=1e-5, out_dtype=bf), flush), T * W * 14)
+        put(f"{phase}.bevuvik.residual_sum_pair", timed_alone(lambda: ops.residual_sum(
+            stream, y=pair, add=f, mult=0.3, weight=wn, eps=1e-5, out_dtype=bf), flush), T * W * 16)
+        put(f"{phase}.torinex.norm_add", timed_alone(lambda: ops.norm_add(stream, y, wn, 1e-5, bias=wn, cast_to=bf), flush), T * W * 12)
+        put(f"{phase}.sigudra.layer_norm_add_pair", timed_alone(
+            lambda: ops.norm_add_pair(stream, pair, wn, 1e-5, cast_to=bf, center=True), flush), T * W * 14)
+        both, win = rnd(T, 2 * W), rnd(W, 2 * W, f=W ** -0.5)
+        put(f"{phase}.bevuvik.pass_rows", timed_alone(lambda: ops.residual_sum(
+            stream, y=y, add=f, bias=wn, mult=0.3, out=both, column=0, store=False), flush), T * W * 10)
+        for name, dtype in (("bevuvik.pass_product", torch.float32), ("qwen3.projection", bf)):
+            us = timed_alone(lambda: ops.linear(both, win, out_dtype=dtype), flush)
+            put(f"{phase}.{name}", us, flops=4.0 * T * W * W) if phase == "prefill" else put(f"{phase}.{name}", us, 4 * W * W)
+        # --- the delta rule with one decay a head beside the one with a decay a key channel
+        for name, kv, per_head in (("bevuvik", rkv, True), ("sigudra", nh, False)):
+            channels = 2 * kv * d + nh * d
+            a_col, g_col, beta = (channels + nh * d, channels, channels + nh * d + nh) if per_head else \
+                (channels, channels + rank, channels + 2 * rank)
+            packed = rnd(T, beta + nh, f=0.5)
+            packed = torch.nn.functional.pad(packed, (0, -packed.shape[1] % 8)).contiguous()
+            form = ops.LinearStateForm(nh, kv, d, d, q_scale=d ** -0.5, decay="softplus",
+                                       decay_bias=torch.full((nh if per_head else nh * d,), -3.0, device=dev),
+                                       a_log=torch.zeros(nh, device=dev), beta_column=beta, silu=True, unit_eps=1e-6,
+                                       decay_column=a_col if per_head else None)
+            conv = torch.randn(channels, taps, device=dev) * 0.3
+            cstate, state = torch.zeros(rows_dec + 1, taps - 1, channels, device=dev), torch.zeros(rows_dec + 1, nh, d, d, device=dev)
+            a2, g2 = (None, None) if per_head else (rnd(nh * d, rank, f=rank ** -0.5), rnd(nh * d, rank, f=rank ** -0.5))
+            hw = torch.ones(d, device=dev)
+            if phase == "prefill":
+                zf = None if per_head else ops.linear_columns(packed, a_col, a2, out_dtype=torch.float32)
+                us = timed_alone(lambda: ops.state_recurrence(form, packed, zf, conv, cstate, state, c), flush, repeats=few)
+                put(f"prefill.{name}.delta_recurrence", us, flops=8.0 * T * nh * d * d, of="fp32")
+                o = torch.randn(T, nh * d, device=dev)
+                gz = packed if per_head else ops.linear_columns(packed, g_col, g2)
+                put(f"prefill.{name}.head_norm_gate", timed_alone(lambda: ops.head_unit_norm_gate(
+                    o, gz, g_col if per_head else 0, nh, d, 1e-5, weight=hw, gate="silu" if per_head else "sigmoid"), flush),
+                    T * nh * d * 8)
+            else:
+                put(f"decode.{name}.state_decode", timed_alone(lambda: ops.state_decode(
+                    form, packed, conv, cstate, state, c, a2, a_col, hw, 1e-5, g_col, g2), flush), rows_dec * nh * d * d * 8)
+        # --- attention: a head's two maps over a window, and soft-capped scores over everything
+        h2, cols = d // 2, (nh + nkv) * d + nkv * d
+        packed, bias = rnd(T, cols, f=0.5), torch.zeros(cols, device=dev)
+        k_cache, v_cache = (torch.zeros(c.pages, nkv, page, d, dtype=bf, device=dev).normal_() for _ in range(2))
+        q, qm = torch.empty(T, nh * d, dtype=bf, device=dev).normal_(), torch.empty(T, 2 * nh * d, dtype=bf, device=dev)
+        o, om = torch.empty(T, nh * d, dtype=bf, device=dev), torch.empty(T, 2 * nh * d, dtype=bf, device=dev)
+        freq = torch.pow(torch.tensor(1e6), -torch.arange(0, h2, 2) / h2).to(dev)
+        put(f"{phase}.bevuvik.heads_prepare_maps", timed_alone(lambda: ops.heads_prepare(
+            packed, qm, k_cache, v_cache, c.positions, c.slots, 2 * nh, nkv, h2, d, bias=bias, inv_freq=freq, rot_dims=h2,
+            interleaved=True, maps=2, rot_gain=1.1), flush), T * (cols + 2 * nh * d + 2 * nkv * d) * 2)
+        put(f"{phase}.bevuvik.heads_prepare", timed_alone(lambda: ops.heads_prepare(
+            packed, q, k_cache, v_cache, c.positions, c.slots, nh, nkv, d, d, inv_freq=freq, rot_dims=h2, interleaved=False),
+            flush), T * cols * 4)
+        put(f"{phase}.lufizen.heads_prepare", timed_alone(lambda: ops.heads_prepare(
+            packed, q, k_cache, v_cache, c.positions, c.slots, nh, nkv, d, d, inv_freq=freq, rot_dims=h2, interleaved=False,
+            plain_norm=True, norm_after_rotation=True, eps=1e-5), flush), T * cols * 4)
+        put(f"{phase}.bevuvik.head_difference", timed_alone(lambda: ops.head_difference(om, nh, d, 0.5, 0.6, 1e-5), flush), T * nh * d * 6)
+        arms = (("bevuvik.difference_window", qm, o, 2 * nh, window, dict(difference=(0.5, 0.6, 1e-5)), 2.0 * 2 * nh * (h2 + d)),
+                ("sigudra.attention_window", q, o, nh, window, {}, 4.0 * nh * d),
+                ("bevuvik.attention_softcap", q, o, nh, None, dict(softcap=50.0), 4.0 * nh * d),
+                ("kefetar.attention_softcap", q, o, nh, None, dict(softcap=50.0), 4.0 * nh * d))
+        for name, qq, oo, heads, win_, more, per_pair in arms:
+            more = dict(v_head_dim=d, precise_weights=True, **more)
+            if phase == "prefill":
+                seen = sum(min(p + 1, win_ or T) for p in range(T))
+                put(f"prefill.{name}", timed_alone(lambda: ops.prefill_attention(
+                    qq, k_cache, v_cache, oo, c.table, c.cu_q, c.kv_len, c.prefix_len, c.rows, 1, T, heads, nkv, d, page, win_,
+                    d ** -0.5, **more), flush, repeats=few), flops=per_pair * seen)
+            else:
+                seen = min(win_ or ctx_len, ctx_len)
+                splits = decode_splits(ops.decode_ctas_per_split(bf, rows_dec, heads, nkv, d, page), seen, 148)
+                scratch = torch.empty(max(ops.decode_scratch_floats(rows_dec, heads, d, splits), 1), device=dev)
+                put(f"decode.{name}", timed_alone(lambda: ops.decode_attention(
+                    qq, k_cache, v_cache, oo, scratch, c.table, c.cu_q, c.kv_len, c.rows, rows_dec, heads, nkv, d, page, win_,
+                    d ** -0.5, splits, **more), flush), rows_dec * seen * nkv * d * 4)
+        # --- feed-forwards
+        xe = rnd(T, W)
+        wgu, wdn = rnd(2 * I, W, f=W ** -0.5), rnd(W, I, f=I ** -0.5)
+        for name, kind, extra in (("bevuvik.clamped_feed_forward", "gated_act", {"activation": "clamped_swish", "limit": 7.0}),
+                                  ("sigudra.gelu_feed_forward", "gated_act", {"activation": "gelu_tanh"}),
+                                  ("qwen3.feed_forward", "swiglu", {})):
+            ff = build_part("feed_forward", PartSpec(kind, dict(hidden_size=W, intermediate_size=I, **extra)), BuildEnv(bf, dev, {}))
+            ff.bind("gate_up_proj", wgu)
+            ff.bind("down_proj", wdn)
+            us = timed_alone(lambda: (ff.forward(xe), ops.flush_chain()), flush)
+            put(f"prefill.{name}", us, flops=6.0 * T * W * I) if phase == "prefill" else put(f"decode.{name}", us, 3 * W * I * 2)
+    return out
+
+
 DESIGNS = {"kefetar": (kefetar_config, kernel_table), "mukenex": (mukenex_config, mukenex_kernel_table),
            "torinex": (torinex_config, torinex_kernel_table), "lufizen": (lufizen_config, lufizen_kernel_table),
-           "sigudra": (sigudra_config, sigudra_kernel_table)}
+           "sigudra": (sigudra_config, sigudra_kernel_table), "bevuvik": (bevuvik_config, bevuvik_kernel_table)}
 # The closest earlier design, which stands beside the new one and Qwen3 at equal sizes.
-BESIDE = {"lufizen": ("torinex", torinex_config), "sigudra": ("kefetar", kefetar_config)}
+BESIDE = {"lufizen": ("torinex", torinex_config), "sigudra": ("kefetar", kefetar_config),
+          "bevuvik": ("sigudra", sigudra_config)}
 
 
 def design_main(args) -> int:
@@ -1371,8 +1547,8 @@ def main() -> int:
                     help="other shapes measured into `points` (decode at batch 1 / 8 / 64, prefill), comma separated")
     ap.add_argument("--only", choices=["decode", "prefill"], default=None,
                     help="run one phase alone and print a short line (for profiling)")
-    ap.add_argument("--design", choices=["qwen3", "kefetar", "mukenex", "torinex", "lufizen", "sigudra"], default="qwen3",
-                    help="kefetar, mukenex, torinex, lufizen, sigudra: that design beside Qwen3 at equal sizes, and its kernels alone (another line)")
+    ap.add_argument("--design", choices=["qwen3", "kefetar", "mukenex", "torinex", "lufizen", "sigudra", "bevuvik"], default="qwen3",
+                    help="kefetar, mukenex, torinex, lufizen, sigudra, bevuvik: that design beside Qwen3 at equal sizes, and its kernels alone (another line)")
     ap.add_argument("--design-sizes", default="1k,4k", help="layer sizes of the other designs, comma separated")
     ap.add_argument("--no-kernels", action="store_true", help="--design ... without the table of single kernels")
     args = ap.parse_args()

@@ -1298,6 +1298,53 @@ def flush_chain() -> None:
             _ok(rc, "linear_chain")
 
 
+# --------------------------------------------------------------------------- independent work side by side
+# Parts of a layer that read the same input and do not read one another (a mixer and a feed-forward behind one norm, two
+# mixers side by side) may run on streams of their own.  Off: everything on one stream, in the order of the calls.
+run_beside = os.environ.get("LLM_INFER_B200_BESIDE", "1") != "0"
+_side_streams = {}
+
+
+def side_by_side(device: torch.device, first, *others):
+    """The results of ``first()`` and of every function of ``others``: pieces of work that do not read one another's
+    results.  ``first`` runs on the current stream, each of the others on a stream of its own, behind what the current
+    stream holds now; what the current stream gets next waits for all of them.  Inside a graph capture they become
+    parallel branches.  May be nested (an inner call takes other streams).
+
+    Memory: what a side stream allocates goes back to that stream's pool, and its next use there lies behind a later fork of
+    the current stream, that is behind whatever read it.  The persistent chain of few-row products, whose CTAs wait for one
+    another, must have the GPU to itself: on that route everything stays on one stream."""
+    if not run_beside or few_row_route == "chain" or device.type != "cuda":
+        return tuple([first()] + [f() for f in others])
+    flush_chain()
+    main = torch.cuda.current_stream(device)
+    pool = _side_streams.setdefault(device.index or 0, [])
+    fork = main.record_event()
+    depth = _side_depth[0]
+    _side_depth[0] += len(others)
+    while len(pool) < depth + len(others):
+        pool.append(torch.cuda.Stream(device))
+    try:
+        results, joins = [None] * len(others), []
+        for i, f in enumerate(others):
+            side = pool[depth + i]
+            with torch.cuda.stream(side):
+                side.wait_event(fork)
+                results[i] = f()
+                flush_chain()
+                joins.append(side.record_event())
+        head = first()
+        flush_chain()
+        for event in joins:
+            main.wait_event(event)
+    finally:
+        _side_depth[0] = depth
+    return tuple([head] + results)
+
+
+_side_depth = [0]          # side streams that the calls around the current one have taken
+
+
 # --------------------------------------------------------------------------- many-row products on tcgen05
 GEMM_PLAIN, GEMM_SWIGLU = 0, 1
 _gemm_maps = {}
