@@ -138,6 +138,115 @@ heads_prepare_kernel(const T* __restrict__ x, int in_stride, const float* __rest
   for (int i = lane; i < width; i += 32) dst[i] = from_f32<T>(row[i]);
 }
 
+// (1) without norms, for rows of whole 16-byte pieces: a block takes a token (in a step of few tokens a part of one), its
+// angles once for all heads, eight neighbouring columns a thread (in the half-split form together with the eight that they
+// turn with).  grid (tokens, parts).
+constexpr int VEC_THREADS = 256;
+
+template <typename T>
+__device__ __forceinline__ void store_piece(T* p, const float (&v)[8]) {
+  if constexpr (sizeof(T) == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+  } else {
+    __nv_bfloat162 h[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) h[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+    *reinterpret_cast<uint4*>(p) = *reinterpret_cast<const uint4*>(h);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(VEC_THREADS)
+heads_prepare_vec_kernel(const T* __restrict__ x, int in_stride, const float* __restrict__ bias,
+                         const float* __restrict__ inv_freq, int rot_dims, int interleaved,
+                         const int* __restrict__ positions, const int* __restrict__ slots, int nh, int nkv, int d, int dv,
+                         int maps, float rot_gain, int page_size, long long cache_slots, T* __restrict__ q_out,
+                         T* __restrict__ k_cache, T* __restrict__ v_cache, int* err) {
+  pdl_launch_dependents();                          // the kernel after this one may be scheduled; it waits before it reads
+  extern __shared__ float angles[];                  // cosines, then sines, of the token's rot_dims / 2 angles
+  const int t = blockIdx.x, half = rot_dims >> 1;
+  const float pos = static_cast<float>(positions[t]);          // (uploaded before the step's first kernel)
+  for (int i = threadIdx.x; i < half; i += VEC_THREADS) {
+    float sn, cs;
+    sincosf(pos * inv_freq[i], &sn, &cs);
+    angles[i] = cs * rot_gain;
+    angles[half + i] = sn * rot_gain;
+  }
+  int slot = slots != nullptr ? slots[t] : 0;
+  if (slot < 0 || slot >= cache_slots) {
+    if (slots != nullptr && threadIdx.x == 0 && blockIdx.y == 0) atomicOr(err, B200_ERR_SLOT_RANGE);
+    slot = 0;
+  }
+  pdl_wait();                                        // the packed projection comes from the kernel before
+  __syncthreads();
+  const int page = slot / page_size, offset = slot - page * page_size;
+  const T* row = x + static_cast<size_t>(t) * in_stride;
+  const int per = d >> 3, per_v = dv >> 3, nk = nkv * maps;
+  const int turned = (nh + nk) * per, pieces = turned + nkv * per_v;
+  auto load = [&](int col, float (&v)[8]) {
+    load_floats<T, 8>(row + col, v);
+    if (bias != nullptr) {
+      float b[8];
+      load_floats<float, 8>(bias + col, b);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) v[i] += b[i];
+    }
+  };
+  for (int p = blockIdx.y * VEC_THREADS + threadIdx.x; p < pieces; p += gridDim.y * VEC_THREADS) {
+    float v[8];
+    if (p >= turned) {                               // a value
+      if (slot == 0) continue;
+      const int kvh = (p - turned) / per_v, c = (p - turned - kvh * per_v) << 3;
+      load((nh + nk) * d + kvh * dv + c, v);
+      store_piece<T>(v_cache + ((static_cast<size_t>(page) * nkv + kvh) * page_size + offset) * dv + c, v);
+      continue;
+    }
+    const int h = p / per, c = (p - h * per) << 3;   // which vector of q and k, and the first of its columns
+    const bool is_q = h < nh;
+    const int vec = is_q ? h : h - nh, map = vec % maps;
+    T* dst;
+    if (is_q) {
+      T* base = q_out + (static_cast<size_t>(t) * nh + vec) * maps * d;
+      dst = base + map * d;
+      for (int m = 0; m < maps; ++m) {
+        const float zero[8] = {};
+        if (m != map) store_piece<T>(base + m * d + c, zero);
+      }
+    } else {
+      if (slot == 0) continue;
+      const int kvh = vec / maps;
+      dst = k_cache + ((static_cast<size_t>(page) * nkv + kvh) * page_size + offset) * (maps * d) + map * d;
+    }
+    if (!interleaved && c >= half && c < rot_dims) continue;      // the thread of the other eight has them
+    load(h * d + c, v);
+    if (c < rot_dims) {
+      if (interleaved) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          if (c + 2 * i < rot_dims) {
+            const int a = (c >> 1) + i;
+            const float cs = angles[a], sn = angles[half + a], u = v[2 * i], w = v[2 * i + 1];
+            v[2 * i] = u * cs - w * sn;
+            v[2 * i + 1] = w * cs + u * sn;
+          }
+        }
+      } else {
+        float w[8];
+        load(h * d + c + half, w);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          const float cs = angles[c + i], sn = angles[half + c + i], u = v[i];
+          v[i] = u * cs - w[i] * sn;
+          w[i] = w[i] * cs + u * sn;
+        }
+        store_piece<T>(dst + c + half, w);
+      }
+    }
+    store_piece<T>(dst + c, v);
+  }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(WARPS * 32)
 latent_prepare_kernel(const T* __restrict__ x, int in_stride, const T* __restrict__ down, int down_stride,
@@ -338,6 +447,24 @@ B200_EXPORT int b200_heads_prepare(const void* x, int dtype, int in_stride, cons
       (rot_dims & 1) || page_size <= 0 || ((flags & PREP_VALUES_ARE_KEYS) && (dv != d || maps != 1)) || maps < 1 ||
       nh % maps != 0)
     return B200_BAD_SIZE;
+  if (inv_freq == nullptr) rot_dims = 0;
+  const int item = dtype == B200_F32 ? 4 : 2;
+  const bool whole = d % 8 == 0 && dv % 8 == 0 && in_stride * item % 16 == 0 && (interleaved || rot_dims % 16 == 0) &&
+                     ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(bias) | reinterpret_cast<uintptr_t>(q_out) |
+                       reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache)) % 16) == 0;
+  if (q_w == nullptr && k_w == nullptr && flags == 0 && whole) {
+    const long long pieces = (static_cast<long long>(nh + nkv * maps) * d + static_cast<long long>(nkv) * dv) / 8;
+    const dim3 grid(tokens, tokens <= 64 ? static_cast<unsigned>((pieces + VEC_THREADS - 1) / VEC_THREADS) : 1u);
+#define B200_PREPARE_VEC(T)                                                                                            \
+  return b200_launch(heads_prepare_vec_kernel<T>, grid, dim3(VEC_THREADS), rot_dims * sizeof(float), stream, 0, \
+                     static_cast<const T*>(x), in_stride, bias, inv_freq, rot_dims, interleaved, positions, slots, nh, \
+                     nkv, d, dv, maps, rot_gain, page_size, cache_slots, static_cast<T*>(q_out),                       \
+                     static_cast<T*>(k_cache), static_cast<T*>(v_cache), err)
+    if (dtype == B200_F32) B200_PREPARE_VEC(float);
+    if (dtype == B200_BF16) B200_PREPARE_VEC(__nv_bfloat16);
+#undef B200_PREPARE_VEC
+    return B200_BAD_DTYPE;
+  }
   const long long work = static_cast<long long>(tokens) * (nh + nkv * maps + nkv);
   const unsigned blocks = static_cast<unsigned>((work + WARPS - 1) / WARPS);
   if (dtype == B200_F32)

@@ -1302,47 +1302,45 @@ def flush_chain() -> None:
 # Parts of a layer that read the same input and do not read one another (a mixer and a feed-forward behind one norm, two
 # mixers side by side) may run on streams of their own.  Off: everything on one stream, in the order of the calls.
 run_beside = os.environ.get("LLM_INFER_B200_BESIDE", "1") != "0"
-_side_streams = {}
+# Steps of up to so many tokens are made of kernels that leave much of the GPU idle (a decode step of Bevuvik at width 1,024,
+# batch 1: 0.477 -> 0.374 ms).  In a prompt portion of thousands of tokens they fill it: measured, a recurrence's scan beside
+# attention and products takes as much longer as it would have waited.
+BESIDE_FEW = 64
+_side_streams = {}         # device -> streams
+_side_depth = [0]          # side streams that the calls around the current one have taken
 
 
-def side_by_side(device: torch.device, first, *others):
-    """The results of ``first()`` and of every function of ``others``: pieces of work that do not read one another's
-    results.  ``first`` runs on the current stream, each of the others on a stream of its own, behind what the current
-    stream holds now; what the current stream gets next waits for all of them.  Inside a graph capture they become
-    parallel branches.  May be nested (an inner call takes other streams).
+def side_by_side(tokens: int, device: torch.device, here, aside):
+    """(``here()``, ``aside()``): two pieces of a step's work that do not read one another's results.  In a step of few
+    tokens ``here`` runs on the current stream and ``aside`` on a stream of its own, behind what the current stream holds
+    now; what the current stream gets next waits for both.  Inside a graph capture they become parallel branches.  May be
+    nested (an inner call takes another stream).
 
     Memory: what a side stream allocates goes back to that stream's pool, and its next use there lies behind a later fork of
     the current stream, that is behind whatever read it.  The persistent chain of few-row products, whose CTAs wait for one
     another, must have the GPU to itself: on that route everything stays on one stream."""
-    if not run_beside or few_row_route == "chain" or device.type != "cuda":
-        return tuple([first()] + [f() for f in others])
+    if not run_beside or tokens > BESIDE_FEW or few_row_route == "chain" or device.type != "cuda":
+        return here(), aside()
     flush_chain()
     main = torch.cuda.current_stream(device)
-    pool = _side_streams.setdefault(device.index or 0, [])
     fork = main.record_event()
     depth = _side_depth[0]
-    _side_depth[0] += len(others)
-    while len(pool) < depth + len(others):
+    pool = _side_streams.setdefault(device.index or 0, [])
+    while len(pool) <= depth:
         pool.append(torch.cuda.Stream(device))
+    _side_depth[0] = depth + 1
     try:
-        results, joins = [None] * len(others), []
-        for i, f in enumerate(others):
-            side = pool[depth + i]
-            with torch.cuda.stream(side):
-                side.wait_event(fork)
-                results[i] = f()
-                flush_chain()
-                joins.append(side.record_event())
-        head = first()
+        with torch.cuda.stream(pool[depth]):
+            pool[depth].wait_event(fork)
+            there = aside()
+            flush_chain()
+            done = pool[depth].record_event()
+        mine = here()
         flush_chain()
-        for event in joins:
-            main.wait_event(event)
+        main.wait_event(done)
     finally:
         _side_depth[0] = depth
-    return tuple([head] + results)
-
-
-_side_depth = [0]          # side streams that the calls around the current one have taken
+    return mine, there
 
 
 # --------------------------------------------------------------------------- many-row products on tcgen05

@@ -260,8 +260,8 @@ class ParallelSublayers:
 
     Parts by name: ``input_norm`` (``owed_rms_norm``), ``mixer`` and optionally ``feed_forward``.  The sum is owed
     (``OwedSum``) to the next read of the stream: the block returns (what is owed, the stream), and the next block's norm,
-    a pass input or the model's last norm takes both in one kernel.  Neither sublayer reads the other's result: they run
-    side by side, on streams of their own (``ops.side_by_side``).  A mixer that has an output bias and offers
+    a pass input or the model's last norm takes both in one kernel.  Neither sublayer reads the other's result: in a
+    step of few tokens they run side by side (``ops.side_by_side``).  A mixer that has an output bias and offers
     ``defer_output_bias()`` leaves the bias to that kernel.  A feed-forward that says ``needs_context`` is also given the
     step's context."""
     category = "block"
@@ -291,8 +291,12 @@ class ParallelSublayers:
         if ff is None:
             y = self.mixer.forward(x, ctx, cache)
         else:
-            y, add = ops.side_by_side(x.device, lambda: self.mixer.forward(x, ctx, cache),
-                                      lambda: ff.forward(x, ctx) if getattr(ff, "needs_context", False) else ff.forward(x))
+            def mix():
+                return self.mixer.forward(x, ctx, cache)
+
+            def feed():
+                return ff.forward(x, ctx) if getattr(ff, "needs_context", False) else ff.forward(x)
+            y, add = ops.side_by_side(x.shape[0], x.device, mix, feed)
         return OwedSum(y, add, self.mult, self.mixer.params.get("o_bias") if self.mixer_bias_here else None), stream
 
 

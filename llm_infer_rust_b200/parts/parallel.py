@@ -12,7 +12,8 @@ class ParallelMixers(Part):
     """(R(left(h); left_out) + R(right(h); right_out)) / 2, R the RMS norm over the model's width (``eps``) with a branch's
     own weights.  ``left`` and ``right`` are part specifications; at most one of them keeps keys and values in pages, both
     may keep state.  Branches that can start from a packed projection (``in_proj_name`` and ``forward_packed``) share ONE
-    product for their projections; from there on they run side by side (``ops.side_by_side``).  The mean is handed on unformed (``ops.NormedPair``): the norm that adds the mixer's
+    product for their projections; from there on, in a step of few tokens, they run side
+    by side (``ops.side_by_side``).  The mean is handed on unformed (``ops.NormedPair``): the norm that adds the mixer's
     output into the stream takes it in its own kernel."""
     category = "mixer"
 
@@ -70,10 +71,11 @@ class ParallelMixers(Part):
         if all(hasattr(m, "forward_packed") for m in (self.left, self.right)):
             weight, column = self._joint_projection()
             packed = ops.linear(x, weight)
-            a, b = ops.side_by_side(x.device, lambda: self.left.forward_packed(packed, 0, ctx, left),
+            a, b = ops.side_by_side(x.shape[0], x.device, lambda: self.left.forward_packed(packed, 0, ctx, left),
                                     lambda: self.right.forward_packed(packed, column, ctx, right))
         else:
-            a, b = ops.side_by_side(x.device, lambda: self.left.forward(x, ctx, left), lambda: self.right.forward(x, ctx, right))
+            a, b = ops.side_by_side(x.shape[0], x.device, lambda: self.left.forward(x, ctx, left),
+                                    lambda: self.right.forward(x, ctx, right))
         return ops.NormedPair(a, b, self.params["left_out"], self.params["right_out"], self.eps)
 
 

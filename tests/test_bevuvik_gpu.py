@@ -89,19 +89,21 @@ def test_the_owed_sum_and_the_norm_behind_it(width, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("H,G,d,dv,dims,maps,interleaved", [(4, 2, 12, 20, 8, 2, True), (3, 1, 32, 16, 32, 2, True),
-                                                           (2, 2, 9, 6, 2, 2, False), (5, 5, 16, 16, 6, 1, False)])
-def test_heads_before_attention(H, G, d, dv, dims, maps, interleaved, dtype):
+@pytest.mark.parametrize("whole_rows", [False, True])
+@pytest.mark.parametrize("H,G,d,dv,dims,maps,interleaved", [
+    (4, 2, 12, 20, 8, 2, True), (3, 1, 32, 16, 32, 2, True), (4, 2, 24, 16, 12, 2, True), (2, 2, 9, 6, 2, 2, False),
+    (5, 5, 16, 16, 6, 1, False), (3, 3, 40, 8, 32, 1, False), (2, 1, 16, 32, 16, 2, False), (2, 1, 8, 8, 0, 2, True)])
+def test_heads_before_attention(H, G, d, dv, dims, maps, interleaved, whole_rows, dtype):
     """Biases, scaled frequencies with a gain, both pairings, and two maps a head: keys of both in one cache row, query
-    vectors zero outside their own map's columns."""
+    vectors zero outside their own map's columns; rows of whole 16-byte pieces (eight columns a thread) and others."""
     from llm_infer_rust_b200.kernels import ops
     dev = torch.device("cuda")
     g = torch.Generator().manual_seed(d)
     T, page = 11, 4
     n = (H + G) * maps * d + G * dv
-    packed = K.bf16_values(torch.randn(T, n + 5, generator=g))
+    packed = K.bf16_values(torch.randn(T, n + (8 - n % 8 if whole_rows else 5), generator=g))
     bias = torch.randn(n, generator=g)
-    freq, gain = P.yarn(dims, 1000.0, {"factor": 4.0, "original": 32, "fast": 8.0, "slow": 0.5})
+    freq, gain = P.yarn(dims, 1000.0, {"factor": 4.0, "original": 32, "fast": 8.0, "slow": 0.5}) if dims else P.rotation({})
     q = torch.full((T, H * maps * maps * d), 9.0, device=dev, dtype=dtype)
     k_cache = torch.full((6, G, page, maps * d), 9.0, device=dev, dtype=dtype)
     v_cache = torch.full((6, G, page, dv), 9.0, device=dev, dtype=dtype)
@@ -109,7 +111,7 @@ def test_heads_before_attention(H, G, d, dv, dims, maps, interleaved, dtype):
     slots = [order[t // page] * page + t % page for t in range(T)]
     slots[7] = 0                                             # a padding row stores nothing
     ops.heads_prepare(packed.to(dev, dtype), q, k_cache, v_cache, _i32(list(range(T))), _i32(slots), H * maps, G, d, dv,
-                      bias=bias.to(dev), inv_freq=freq.float().to(dev), rot_dims=dims, interleaved=interleaved, maps=maps,
+                      bias=bias.to(dev), inv_freq=freq.float().to(dev) if dims else None, rot_dims=dims, interleaved=interleaved, maps=maps,
                       rot_gain=gain)
     x = packed[:, :n].double() + bias.double()
     wq = P.rotate(x[:, :H * maps * d].reshape(T, H * maps, d), freq, gain, interleaved)
